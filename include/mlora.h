@@ -51,6 +51,8 @@ extern "C" {
                                8), then the index of each adapter's first slice.  The expand then reads exactly
                                rank * out * 2 bytes per row, in whole 16-byte units per output feature, whatever the
                                widest rank of the stack is */
+#define MLORA_ACT_RELU2 256 /* y = relu(y)^2, on the fp32 accumulator (projections without adapters) */
+#define MLORA_ACT_GELU 512  /* y = gelu(y) with the exact erf, likewise */
 #define MLORA_SHARE_LORA_KERNEL 32 /* hint for a call WITHOUT LoRA operands that sits between calls with them
                                (gate/up/down when only q/k/v/o carry adapters): run the kernel variant the LoRA
                                calls use, so one code footprint stays hot in the instruction caches for the whole
@@ -430,6 +432,84 @@ int mlora_decode_step_begin(const int32_t* d_live, const int32_t* d_seq_slot, co
 int mlora_decode_step_end(const int32_t* d_row_src, const int32_t* d_next_tok, int32_t n_rows, int32_t* d_live,
                           int32_t* d_last_tok, int32_t* d_gen_count, const int32_t* d_max_gen,
                           int32_t* d_out_tokens, int64_t ld_out, int32_t eos_id, int32_t* d_n_live, void* stream);
+
+/* ---- grouped projections ---------------------------------------------------------------------------------
+ * Several weights of one shape [out, in] in one launch of the tensor-core projection, each over its own rows or its own
+ * column slice: the experts of a mixture (rows listed per expert, on the device) or the heads of an attention layer.
+ *   d_Wp: n_groups matrices in the layout of mlora_pack_weight, one after the other
+ *   d_tiles == NULL: every group has the rows 0 .. T-1; group g reads the columns [g * x_cols, g * x_cols + in) of x (x_cols
+ *     a multiple of 64; 0: all groups read the same columns) and writes the columns from g * y_cols
+ *   d_tiles (int32, 16-byte aligned): [0] the number of row tiles, then from [4] on per tile (group, first row, rows <=
+ *     tile_rows, 0), as written by mlora_moe_plan.  Row r of the table reads x row d_gather[r] (NULL: row r) and writes y
+ *     row r.  x_rows = rows of x.
+ *   tile_rows: 16, 32, 64, 128 or 256 rows per tile.  flags: MLORA_OUT_F32, one of MLORA_ACT_*
+ *   d_gate (bf16, NULL: none): output row t of group g is multiplied by sigmoid(d_gate[t * ld_gate + g])
+ *   d_work: mlora_grouped_linear_workspace(tile_rows) bytes with the zero-fill rule and status word of mlora_linear's. */
+size_t mlora_grouped_linear_workspace(int32_t tile_rows);
+int mlora_grouped_linear(const void* d_x, int64_t ldx, int32_t x_rows, int32_t x_cols, const int32_t* d_gather,
+                         const void* d_Wp, void* d_y, int64_t ldy, int32_t y_cols, const int32_t* d_tiles,
+                         int32_t n_groups, int32_t T, int32_t tile_rows, int32_t in, int32_t out, int32_t flags,
+                         const void* d_gate, int64_t ld_gate, void* d_work, size_t work_bytes, void* stream);
+/* The same in true 32-bit on the CUDA cores (x, W, y, gate fp32; W row-major [n_groups, out, in]); n_groups = 1 without a
+ * table is a plain projection.  Row tiles of 64: a table must have been made with tile_rows = 64; max_tiles bounds its
+ * length.  flags: one of MLORA_ACT_*. */
+int mlora_linear_f32(const float* d_x, int64_t ldx, int32_t x_cols, const int32_t* d_gather, const float* d_W, float* d_y,
+                     int64_t ldy, int32_t y_cols, const int32_t* d_tiles, int32_t max_tiles, int32_t n_groups, int32_t T,
+                     int32_t in, int32_t out, int32_t flags, const float* d_gate, int64_t ld_gate, void* stream);
+
+/* ---- mixture of experts: routing and grouping ---------------------------------------------------------------
+ * Per token the `top` largest of its E router logits (logits[t * ld + e] + bias[e], fp32; lower index first among equals)
+ * and the softmax over exactly those; then the T * top (token, expert) pairs grouped by expert, in token order inside one.
+ *   d_expert, d_weight [T, top]; d_pos [T, top]: row of the pair in expert order; d_rows [T * top]: token of a row;
+ *   d_tiles: the table of mlora_grouped_linear for tiles of tile_rows rows, room for 1 + T * top / tile_rows + min(E, T * top)
+ *   entries of 16 bytes.  E <= 1024.  d_work: mlora_moe_plan_workspace(T, E, top) bytes (0 for decode sizes, one launch). */
+size_t mlora_moe_plan_workspace(int32_t T, int32_t E, int32_t top);
+int mlora_moe_plan(const float* d_logits, int64_t ld, const float* d_bias, int32_t T, int32_t E, int32_t top, int32_t tile_rows,
+                   int32_t* d_expert, float* d_weight, int32_t* d_pos, int32_t* d_rows, int32_t* d_tiles, void* d_work,
+                   size_t work_bytes, void* stream);
+
+/* ---- residual add + dynamic tanh norm ----------------------------------------------------------------------
+ *   res[t] += delta[t] + sum_k weight[t, k] * expert_rows[pos[t, k]];   out[i] = tanh(alpha * res[r]) * w + b
+ * with r = i, or d_rows[i] when given (then only those rows are updated and written; they must be distinct if anything is
+ * added).  delta and expert_rows may be NULL.  delta, expert_rows and out are bf16, or fp32 with f32 != 0; w, b [H] and the
+ * scalar alpha are bf16 on the device; res is fp32. */
+int mlora_residual_dyt(const void* d_delta, const void* d_expert_rows, const int32_t* d_pos, const float* d_weight, int32_t top,
+                       float* d_res, const int32_t* d_rows, const void* d_w, const void* d_b, const void* d_alpha, void* d_out,
+                       int32_t T, int32_t H, int32_t f32, void* stream);
+
+/* ---- latent attention ----------------------------------------------------------------------------------------
+ * The cache holds one vector of R = kv_rank values per token (pages [n_pages, page_size, pitch], bf16 or fp32); keys and
+ * values of all heads are linear maps of it.
+ * mlora_latent_append: c = x / sqrt(mean(x^2) + eps) * w into the row's place (rows with row_pos < 0 are skipped).
+ * mlora_latent_gather: segments int32 [n][4] = (cache slot, first output row (a multiple of page_size), tokens, 0): the
+ *   pages of the sequence as consecutive rows (bf16), for callers that expand keys and values of a whole context.
+ * mlora_prefill_attention_dense: causal attention of prompt rows on the tensor cores over expanded keys and values; row of
+ *   d_kv = [head 0's key, ..., head H-1's key, (from v_col) head 0's value, ...]; tiles as for mlora_prefill_attention with
+ *   the row of the sequence's first key instead of the cache slot; head sizes 64 or 128, scale > 0.  d_gate as for
+ *   mlora_grouped_linear, by head.
+ * mlora_latent_attention: queries already mapped into latent space (qa [T, H, q_pitch], q_pitch = R rounded up to 128,
+ *   zero columns past R); out[t, h] = sum_j softmax_j(scale * qa[t, h] . c_j) c_j over the positions j <= row_pos[t], bf16,
+ *   tensor cores, R <= 512.  n_splits CTAs share a row's keys (mlora_latent_attention_splits proposes a number).
+ * mlora_latent_attention_simt: the same on the CUDA cores, bf16 or fp32, q_pitch >= R up to 2048. */
+int mlora_latent_append(const void* d_x, int64_t ld, int32_t R, const void* d_w, float eps, void* d_pages, int32_t pitch,
+                        int32_t page_size, const int32_t* d_block_table, int32_t max_pages, const int32_t* d_row_slot,
+                        const int32_t* d_row_pos, int32_t T, int32_t f32, void* stream);
+int mlora_latent_gather(const void* d_pages, int32_t pitch, int32_t page_size, const int32_t* d_block_table, int32_t max_pages,
+                        const int32_t* d_segs, int32_t n_segs, int32_t max_tokens, void* d_out, void* stream);
+int mlora_prefill_attention_dense(const void* d_q, int64_t ld, const void* d_kv, int64_t ld_kv, int32_t kv_rows, int32_t v_col,
+                                  const int32_t* d_tiles, int32_t n_tiles, int32_t H, int32_t Dk, int32_t Dv, float scale,
+                                  const void* d_gate, int64_t ld_gate, int32_t T, void* d_out, int64_t ld_out,
+                                  int32_t* d_status, void* stream);
+uint32_t mlora_latent_attention_splits(int32_t T, int32_t H, int32_t max_keys);
+size_t mlora_latent_attention_workspace(int32_t T, int32_t H, int32_t q_pitch, int32_t n_splits);
+int mlora_latent_attention(const void* d_qa, int64_t q_pitch, const void* d_pages, int32_t n_pages_total, int32_t R, int32_t pitch,
+                           int32_t page_size, const int32_t* d_block_table, int32_t max_pages, const int32_t* d_row_slot,
+                           const int32_t* d_row_pos, int32_t T, int32_t H, float scale, int32_t n_splits, void* d_out,
+                           void* d_work, size_t work_bytes, int32_t* d_status, void* stream);
+int mlora_latent_attention_simt(const void* d_qa, int64_t q_pitch, const void* d_pages, int32_t R, int32_t pitch, int32_t page_size,
+                                const int32_t* d_block_table, int32_t max_pages, const int32_t* d_row_slot,
+                                const int32_t* d_row_pos, int32_t T, int32_t H, float scale, void* d_out, int32_t f32,
+                                void* stream);
 
 #ifdef __cplusplus
 }

@@ -72,6 +72,25 @@ PROTOTYPES = {
     "mlora_tp_reset": (C.c_int, [_vp]),
     "mlora_tp_destroy": (C.c_int, [_vp]),
     "mlora_tp_allreduce_rmsnorm": (C.c_int, [_vp, _vp, _vp, _vp, _f32, _vp, _i32, _i32, _vp]),
+    "mlora_grouped_linear_workspace": (_sz, [_i32]),
+    "mlora_grouped_linear": (C.c_int, [_vp, _i64, _i32, _i32, _vp, _vp, _vp, _i64, _i32, _vp, _i32, _i32, _i32, _i32,
+                                       _i32, _i32, _vp, _i64, _vp, _sz, _vp]),
+    "mlora_linear_f32": (C.c_int, [_vp, _i64, _i32, _vp, _vp, _vp, _i64, _i32, _vp, _i32, _i32, _i32, _i32, _i32,
+                                   _i32, _vp, _i64, _vp]),
+    "mlora_moe_plan_workspace": (_sz, [_i32, _i32, _i32]),
+    "mlora_moe_plan": (C.c_int, [_vp, _i64, _vp, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
+    "mlora_residual_dyt": (C.c_int, [_vp, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _vp]),
+    "mlora_latent_append": (C.c_int, [_vp, _i64, _i32, _vp, _f32, _vp, _i32, _i32, _vp, _i32, _vp, _vp, _i32, _i32,
+                                      _vp]),
+    "mlora_latent_gather": (C.c_int, [_vp, _i32, _i32, _vp, _i32, _vp, _i32, _i32, _vp, _vp]),
+    "mlora_prefill_attention_dense": (C.c_int, [_vp, _i64, _vp, _i64, _i32, _i32, _vp, _i32, _i32, _i32, _i32, _f32,
+                                                _vp, _i64, _i32, _vp, _i64, _vp, _vp]),
+    "mlora_latent_attention_splits": (C.c_uint32, [_i32, _i32, _i32]),
+    "mlora_latent_attention_workspace": (_sz, [_i32, _i32, _i32, _i32]),
+    "mlora_latent_attention": (C.c_int, [_vp, _i64, _vp, _i32, _i32, _i32, _i32, _vp, _i32, _vp, _vp, _i32, _i32,
+                                         _f32, _i32, _vp, _vp, _sz, _vp, _vp]),
+    "mlora_latent_attention_simt": (C.c_int, [_vp, _i64, _vp, _i32, _i32, _i32, _vp, _i32, _vp, _vp, _i32, _i32,
+                                              _f32, _vp, _i32, _vp]),
     "mlora_decode_step_begin": (C.c_int, [_vp, _vp, _vp, _vp, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),
     "mlora_decode_step_end": (C.c_int, [_vp, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _vp, _vp]),
 }

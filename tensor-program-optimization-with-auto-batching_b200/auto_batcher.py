@@ -29,9 +29,9 @@ import torch
 
 from . import adapter_contract
 from . import adapters as adapter_files
+from . import checkpoint, registry
 from . import vm as mvm
 from .adapter_contract import LoraConfig  # same fields as tvm/llama_auto_batcher/lora.py:5-8
-from .model import PackedLlama
 from .seq_info import LlamaSeqInfo
 
 
@@ -267,6 +267,7 @@ class LlamaAutoBatcherClass:
         self.device = torch.device("cuda", 0)
         self.model_config = None
         self.weights = None
+        self.dtype = torch.bfloat16
         self.adapter_dir = None
         self.adapter_targets = ("q_proj", "v_proj")
         self.tokenizer = None
@@ -285,6 +286,13 @@ class LlamaAutoBatcherClass:
     def set_weights(self, state_dict):
         """HF-named state dict of the base model (stands in for the cache_dir + from_pretrained)."""
         self.weights = state_dict
+
+    def set_model_dir(self, model_dir, dtype=torch.bfloat16):
+        """A folder with ``config.json`` and ``model.safetensors`` of any registered design."""
+        cfg = checkpoint.read_config(model_dir)
+        if dtype not in registry.design_of(cfg).dtypes:
+            raise registry.UnsupportedPrecision(f"{registry.design_of(cfg).name} does not run in {dtype}")
+        self.model_config, self.weights, self.dtype = cfg, checkpoint.read_tensors(model_dir), dtype
 
     def set_cache_dir(self, cache_dir):
         """Directory holding ``lora_adapters/r{rank}_a{id}.safetensors`` (compile_tvm.py:302)."""
@@ -343,7 +351,7 @@ class LlamaAutoBatcherClass:
                 lowered, scale = adapter_contract.lower_adapter_file(adapter_files.load_adapter(path), cfg, self.model_config)
                 adapters.append(lowered)
                 scales.append(scale)
-        model = PackedLlama(self.model_config, self.weights, adapters, scales, device=self.device)
+        model = registry.build_model(self.model_config, self.weights, adapters, scales, device=self.device, dtype=self.dtype)
         self.vm = mvm.B200VM(model, type_slot_base=base or [0])
         self.graph.set_exec_vars(self.vm, self.device, self.vm.params, self.tokenizer, self.seq_info, self.exec_config)
 

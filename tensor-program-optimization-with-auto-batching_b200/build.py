@@ -28,16 +28,17 @@ def sources():
     return sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cu"))
 
 
-def _stale() -> bool:
-    if not os.path.exists(LIB):
-        return True
-    t = os.path.getmtime(LIB)
-    deps = [os.path.join(CSRC, f) for f in os.listdir(CSRC)] + [os.path.join(INCLUDE, "mlora.h"), __file__]
-    return any(os.path.getmtime(d) > t for d in deps)
+def _headers():
+    return [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cuh")] + [os.path.join(INCLUDE, "mlora.h"), __file__]
+
+
+def _newer(target, deps) -> bool:
+    return os.path.exists(target) and all(os.path.getmtime(d) <= os.path.getmtime(target) for d in deps)
 
 
 def build(force: bool = False, verbose: bool = False) -> str:
-    if not force and not _stale():
+    """Compiles what is out of date (an object is, when its source or any header is newer) and links."""
+    if not force and _newer(LIB, sources() + _headers()):
         return LIB
     nvcc = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
     if not os.path.exists(nvcc):
@@ -49,16 +50,21 @@ def build(force: bool = False, verbose: bool = False) -> str:
     for src in sources():
         obj = os.path.join(objdir, os.path.basename(src)[:-3] + ".o")
         objs.append(obj)
+        if not force and _newer(obj, [src] + _headers()):
+            continue
         cmd = [nvcc, *NVCC_FLAGS, "-I", INCLUDE, "-c", src, "-o", obj]
         if verbose:
             cmd.insert(1, "-Xptxas=-v")
-        procs.append((src, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
+        procs.append((src, obj, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
     failed = False
-    for src, p in procs:
+    for src, obj, p in procs:
         out, _ = p.communicate()
         if p.returncode != 0 or verbose:
             sys.stderr.write(f"== {os.path.basename(src)}\n{out}\n")
-        failed |= p.returncode != 0
+        if p.returncode != 0:
+            failed = True
+            if os.path.exists(obj):
+                os.remove(obj)
     if failed:
         raise RuntimeError("nvcc failed")
     tmp = LIB + ".tmp"

@@ -15,6 +15,8 @@
 // (96 KB of shared memory and 256 TMEM columns each) and fill each other's gaps.  The point of this kernel is to take
 // prompt attention off the CUDA cores -- the single-query kernel it replaces re-reads every key for every row and
 // reduces every score with shuffles.  Every wait is bounded; a CTA that gives up writes zeros.
+#include <math.h>
+
 #include <atomic>
 
 #include "common.cuh"
@@ -23,7 +25,7 @@
 namespace mlora {
 namespace {
 
-constexpr int kD = 128;            // head dimension
+constexpr int kD = 128;            // head dimension of the paged form
 constexpr int kPS = 16;            // page size
 constexpr int kTile = 128;         // query rows per CTA = keys per block
 constexpr int kPfThreads = 160;    // warps 0..3: one thread per query row; warp 4: TMA + MMA issue
@@ -49,22 +51,31 @@ __device__ __forceinline__ uint64_t make_smem_desc_mn(uint32_t saddr, uint32_t l
 }
 
 struct PfArgs {
-  const int32_t* block_table;
+  const int32_t* block_table;  // paged form
   int max_pages;
-  const int32_t* tiles;  // [n_tiles][4]: cache slot, first row (index into qkv / out), rows, position of the first row
+  const int32_t* tiles;  // [n_tiles][4]: cache slot (dense form: row of the sequence's key 0), first row (index into qkv /
+                         // out), rows, position of the first row
   int Hq, Hkv;
   bf16* out;
   int64_t ld_out;
   int32_t* status;  // optional: set to 1 when a wait expired
+  float scale;      // of the scores
+  const bf16* gate; // dense form: a head's result of row t is multiplied by sigmoid(gate[t * ld_gate + head]); NULL: no gate
+  int64_t ld_gate;
+  int v_col;        // dense form: column of head 0's values in a row of keys and values
 };
 
+// NK, NV: query/key and value size of a head in 64s.  PAGED: keys and values of 128-wide heads come page by page through
+// the block table; else they are consecutive rows [key][head 0's key, head 1's key, ..., head 0's value, ...], one TMA
+// box per 128 keys.
+template <int NK, int NV, bool PAGED>
 __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                          const __grid_constant__ CUtensorMap map_k,
                                                                          const __grid_constant__ CUtensorMap map_v,
                                                                          PfArgs a) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* sq = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-  uint8_t* sk = sq + 2 * kSub;   // K block   [128 keys][128 d]   as two d-halves
+  uint8_t* sk = sq + NK * kSub;  // K block   [128 keys][128 d]   as two d-halves
   uint8_t* sv = sk + 2 * kSub;   // V block   [128 keys][128 d]   as two d-halves, exactly as the pages hold it
   uint8_t* sp = sk;              // P block   [128 q][128 keys]   as two key-halves: over K, which S = Q K^T has consumed by then
   __shared__ uint64_t kbar, sbar, obar;
@@ -75,7 +86,8 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
   const int tile = blockIdx.x, h = blockIdx.y;
   const int rep = a.Hq / a.Hkv, kvh = h / rep;
   const int slot = a.tiles[tile * 4 + 0], row0 = a.tiles[tile * 4 + 1], rows = a.tiles[tile * 4 + 2], pos0 = a.tiles[tile * 4 + 3];
-  const int32_t* bt = a.block_table + (size_t)slot * a.max_pages;
+  const int32_t* bt = PAGED ? a.block_table + (size_t)slot * a.max_pages : nullptr;
+  constexpr int kDv = NV * 64;
   const int n_keys = pos0 + rows;                       // keys any row of the tile may see
   const int n_blocks = (n_keys + kTile - 1) / kTile;
   const int n_pages = (n_keys + kPS - 1) / kPS;
@@ -96,39 +108,46 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
   tc_fence_after();
   const uint32_t tmem_base = tmem_slot;
   constexpr uint32_t idesc = make_idesc(kTile, kTile);
-  constexpr uint32_t idesc_pv = idesc | (1u << 16);  // B operand MN-major
+  constexpr uint32_t idesc_pv = make_idesc(kTile, kDv) | (1u << 16);  // B operand MN-major
 
   // per-row state (threads 0..127)
-  float o_reg[kD];
+  float o_reg[kDv];
 #pragma unroll
-  for (int i = 0; i < kD; ++i) o_reg[i] = 0.f;
+  for (int i = 0; i < kDv; ++i) o_reg[i] = 0.f;
   float m_run = -INFINITY, l_run = 0.f;
   const int q_pos = pos0 + tid;  // position of this thread's query row
-  const float scale = rsqrtf((float)kD) * kLog2e;
+  const float scale = a.scale * kLog2e;
   bool ok = true;
 
   // Block-table entries are read one block ahead (lane p of warp 4 keeps page p of the block's eight), so that no block
   // starts with a dependent chain of two global round trips.
   auto page_of = [&](int pg) { return pg < n_pages ? bt[pg] : -1; };
-  int page_next = (warp == 4 && lane < kTile / kPS) ? page_of(lane) : -1;
+  int page_next = (PAGED && warp == 4 && lane < kTile / kPS) ? page_of(lane) : -1;
 
   for (int kb = 0; kb < n_blocks; ++kb) {
     const uint32_t par = kb & 1;
     const int page0 = kb * (kTile / kPS);
     const int page_cur = page_next;
     const int valid = min(kTile / kPS, n_pages - page0);
-    if (kb + 1 < n_blocks && warp == 4 && lane < kTile / kPS) page_next = page_of(page0 + kTile / kPS + lane);
+    if (PAGED && kb + 1 < n_blocks && warp == 4 && lane < kTile / kPS) page_next = page_of(page0 + kTile / kPS + lane);
     // ---- loads: K and V pages (and Q once) by TMA -----------------------------------------------------------------------------
     if (warp == 4) {
       if (lane == 0) {
-        mbar_expect_tx(&kbar, (uint32_t)valid * 4 * (kPS * 128) + (kb == 0 ? 2 * kSub : 0));
+        mbar_expect_tx(&kbar, (PAGED ? (uint32_t)valid * 4 * (kPS * 128) : (uint32_t)(NK + NV) * kSub) + (kb == 0 ? NK * kSub : 0));
         if (kb == 0) {
-          tma_load_2d(sq, &map_q, h * kD, row0, &kbar);
-          tma_load_2d(sq + kSub, &map_q, h * kD + 64, row0, &kbar);
+#pragma unroll
+          for (int j = 0; j < NK; ++j) tma_load_2d(sq + j * kSub, &map_q, h * NK * 64 + j * 64, row0, &kbar);
+        }
+        if constexpr (!PAGED) {  // rows past the sequence's last key belong to the next one (or are zeros): masked
+#pragma unroll
+          for (int j = 0; j < NK; ++j) tma_load_2d(sk + j * kSub, &map_k, h * NK * 64 + j * 64, slot + kb * kTile, &kbar);
+#pragma unroll
+          for (int j = 0; j < NV; ++j)
+            tma_load_2d(sv + j * kSub, &map_v, a.v_col + h * NV * 64 + j * 64, slot + kb * kTile, &kbar);
         }
       }
       __syncwarp();
-      if (lane < valid) {  // one page per lane, both 64-column halves of K and of V (a missing table entry reads as rows before 0: zeros)
+      if (PAGED && lane < valid) {  // one page per lane, both 64-column halves of K and of V (a missing table entry reads as rows before 0: zeros)
         const int r = (page_cur * a.Hkv + kvh) * kPS;
         tma_load_2d(sk + lane * (kPS * 128), &map_k, 0, r, &kbar);
         tma_load_2d(sk + kSub + lane * (kPS * 128), &map_k, 64, r, &kbar);
@@ -142,7 +161,7 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
       if (!mbar_wait(&kbar, par, &s_abort)) s_abort = 1;
       if (tid >= n_keys - kb * kTile) {
 #pragma unroll
-        for (int half = 0; half < 2; ++half)
+        for (int half = 0; half < NV; ++half)
 #pragma unroll
           for (int c = 0; c < 8; ++c) reinterpret_cast<uint4*>(sv + half * kSub + tid * 128)[c] = make_uint4(0u, 0u, 0u, 0u);
       }
@@ -155,7 +174,7 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
       tc_fence_after();
       if (!s_abort) {
 #pragma unroll
-        for (int j = 0; j < 2; ++j) {
+        for (int j = 0; j < NK; ++j) {
           const uint64_t adesc = make_smem_desc(smem_u32(sq + j * kSub));
           const uint64_t bdesc = make_smem_desc(smem_u32(sk + j * kSub));
 #pragma unroll
@@ -252,7 +271,7 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
       tc_fence_after();
       const uint32_t t_addr = tmem_base + ((uint32_t)(warp * 32) << 16) + kTile;
 #pragma unroll
-      for (int c0 = 0; c0 < kD; c0 += 32) {
+      for (int c0 = 0; c0 < kDv; c0 += 32) {
         float blk[32];
         tmem_ld32(t_addr + c0, blk);
 #pragma unroll
@@ -275,10 +294,12 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
 
   // ---- write ------------------------------------------------------------------------------------------------------------------
   if (tid < kTile && tid < rows) {
-    const float inv = (ok && l_run > 0.f) ? 1.f / l_run : 0.f;
-    uint4* dst = reinterpret_cast<uint4*>(a.out + (size_t)(row0 + tid) * a.ld_out + (size_t)h * kD);
+    float inv = (ok && l_run > 0.f) ? 1.f / l_run : 0.f;
+    if constexpr (!PAGED)
+      if (a.gate) inv /= 1.f + __expf(-__bfloat162float(a.gate[(size_t)(row0 + tid) * a.ld_gate + h]));
+    uint4* dst = reinterpret_cast<uint4*>(a.out + (size_t)(row0 + tid) * a.ld_out + (size_t)h * kDv);
 #pragma unroll
-    for (int c = 0; c < 16; ++c) {
+    for (int c = 0; c < kDv / 8; ++c) {
       float f[8];
 #pragma unroll
       for (int i = 0; i < 8; ++i) f[i] = o_reg[c * 8 + i] * inv;
@@ -289,6 +310,23 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
   tc_fence_before();
   __syncthreads();
   if (warp == 4) tmem_dealloc(tmem_base, 256);
+}
+
+template <int NK, int NV, bool PAGED>
+int launch_prefill(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const PfArgs& a, int n_tiles, cudaStream_t st) {
+  constexpr int smem = (NK + 2 + NV) * kSub + 1024;  // Q, K (= P), V
+  static std::atomic<unsigned long long> attr_done{0};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!((attr_done.load(std::memory_order_acquire) >> (dev & 63)) & 1ull)) {
+    cudaError_t e = cudaFuncSetAttribute(prefill_attn_tc_kernel<NK, NV, PAGED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return fail(MLORA_ECUDA, "prefill_attention: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
+    attr_done.fetch_or(1ull << (dev & 63), std::memory_order_release);
+  }
+  prefill_attn_tc_kernel<NK, NV, PAGED><<<dim3(n_tiles, a.Hq), kPfThreads, smem, st>>>(mq, mk, mv, a);
+  count_launch();
+  MLORA_CHECK_LAUNCH("prefill_attn_tc_kernel");
+  return MLORA_OK;
 }
 
 }  // namespace
@@ -317,18 +355,32 @@ extern "C" int mlora_prefill_attention(const void* d_qkv, int64_t ld, const void
   if (rc) return rc;
   rc = make_map(&mv, d_v_pages, (long long)n_pages_total * Hkv * kPS, kD, kD, kPS, 64);
   if (rc) return rc;
-  constexpr int smem = 6 * kSub + 1024;  // Q, K (= P), V^T
-  static std::atomic<unsigned long long> attr_done{0};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (!((attr_done.load(std::memory_order_acquire) >> (dev & 63)) & 1ull)) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return fail(MLORA_ECUDA, "prefill_attention: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
-    attr_done.fetch_or(1ull << (dev & 63), std::memory_order_release);
-  }
-  PfArgs a{d_block_table, max_pages, d_tiles, Hq, Hkv, (bf16*)d_out, ld_out, d_status};
-  prefill_attn_tc_kernel<<<dim3(n_tiles, Hq), kPfThreads, smem, (cudaStream_t)stream>>>(mq, mk, mv, a);
-  count_launch();
-  MLORA_CHECK_LAUNCH("prefill_attn_tc_kernel");
-  return MLORA_OK;
+  PfArgs a{d_block_table, max_pages, d_tiles, Hq, Hkv, (bf16*)d_out, ld_out, d_status, 1.f / sqrtf((float)kD), nullptr, 0, 0};
+  return launch_prefill<2, 2, true>(mq, mk, mv, a, n_tiles, (cudaStream_t)stream);
+}
+
+extern "C" int mlora_prefill_attention_dense(const void* d_q, int64_t ld, const void* d_kv, int64_t ld_kv, int32_t kv_rows,
+                                             int32_t v_col, const int32_t* d_tiles, int32_t n_tiles, int32_t H, int32_t Dk,
+                                             int32_t Dv, float scale, const void* d_gate, int64_t ld_gate, int32_t T, void* d_out,
+                                             int64_t ld_out, int32_t* d_status, void* stream) {
+  MLORA_REQUIRE((Dk == 64 || Dk == 128) && (Dv == 64 || Dv == 128), "prefill_attention_dense: head sizes 64 and 128 (got %d, %d)", Dk, Dv);
+  MLORA_REQUIRE(scale > 0.f, "prefill_attention_dense: the scale must be positive");
+  MLORA_REQUIRE(n_tiles >= 0 && T >= 0 && H > 0 && H <= 65535 && kv_rows > 0 && v_col >= H * Dk && v_col % 64 == 0 &&
+                    ld_kv >= (int64_t)v_col + (int64_t)H * Dv && ld >= (int64_t)H * Dk && ld_out >= (int64_t)H * Dv,
+                "prefill_attention_dense: bad sizes");
+  MLORA_REQUIRE(d_q && d_kv && d_tiles && d_out, "prefill_attention_dense: null pointer");
+  MLORA_REQUIRE(aligned16(d_q) && aligned16(d_kv) && aligned16(d_out) && (ld * 2) % 16 == 0 && (ld_kv * 2) % 16 == 0 && (ld_out * 2) % 16 == 0,
+                "prefill_attention_dense: 16-byte alignment of tensors and row pitches");
+  if (n_tiles == 0 || T == 0) return MLORA_OK;
+  CUtensorMap mq, mkv;
+  int rc = make_map(&mq, d_q, T, H * Dk, ld, kTile, 64);
+  if (rc) return rc;
+  rc = make_map(&mkv, d_kv, kv_rows, v_col + H * Dv, ld_kv, kTile, 64);
+  if (rc) return rc;
+  PfArgs a{nullptr, 0, d_tiles, H, H, (bf16*)d_out, ld_out, d_status, scale, (const bf16*)d_gate, ld_gate, v_col};
+  cudaStream_t st = (cudaStream_t)stream;
+  if (Dk == 64 && Dv == 64) return launch_prefill<1, 1, false>(mq, mkv, mkv, a, n_tiles, st);
+  if (Dk == 64) return launch_prefill<1, 2, false>(mq, mkv, mkv, a, n_tiles, st);
+  if (Dv == 64) return launch_prefill<2, 1, false>(mq, mkv, mkv, a, n_tiles, st);
+  return launch_prefill<2, 2, false>(mq, mkv, mkv, a, n_tiles, st);
 }

@@ -32,6 +32,10 @@ static int linear_impl(const void* d_x, int64_t ldx, const void* d_W, void* d_y,
                 (long long)ldx);
   MLORA_REQUIRE(d_x && d_W && d_y, "linear: null pointer");
   MLORA_REQUIRE(aligned16(d_x) && aligned16(d_W), "linear: x and W must be 16-byte aligned");
+  if (flags & (MLORA_ACT_RELU2 | MLORA_ACT_GELU))
+    MLORA_REQUIRE(!d_u && !nf && !(flags & (MLORA_SILU_MUL | MLORA_SHARE_LORA_KERNEL)) &&
+                      (flags & (MLORA_ACT_RELU2 | MLORA_ACT_GELU)) != (MLORA_ACT_RELU2 | MLORA_ACT_GELU),
+                  "linear: one activation, on a projection without adapters");
   if (flags & MLORA_SILU_MUL) MLORA_REQUIRE(out % 16 == 0, "linear: SILU_MUL needs out %% 16 == 0 (out=%d)", out);
   LinearArgs a{};
   a.x = (const bf16*)d_x;

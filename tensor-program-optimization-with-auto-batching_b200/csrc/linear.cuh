@@ -77,6 +77,26 @@ __device__ __forceinline__ float lora_expand(const LinearArgs& a, int t, int o) 
 // runs once per tile, from cold instruction caches)
 __device__ __forceinline__ float silu_mul(float g, float up) { return __fdividef(g, 1.f + __expf(-g)) * up; }
 
+// Activations of plain feed-forward layers, applied to the fp32 accumulator: relu(z)^2, or gelu(z) with the exact erf.
+__device__ __forceinline__ float act_one(float z, int act) {
+  if (act == MLORA_ACT_RELU2) {
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+  }
+  if (act == MLORA_ACT_GELU) return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
+  return z;
+}
+template <int N>
+__device__ __forceinline__ void apply_act(float (&v)[32], int act) {
+  if (act == MLORA_ACT_RELU2) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = act_one(v[i], MLORA_ACT_RELU2);
+  } else if (act == MLORA_ACT_GELU) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = act_one(v[i], MLORA_ACT_GELU);
+  }
+}
+
 __device__ __forceinline__ void store_out(const LinearArgs& a, int t, int col, float v) {
   if (a.flags & MLORA_OUT_F32)
     reinterpret_cast<float*>(a.y)[(size_t)t * a.ldy + col] = v;
@@ -86,6 +106,17 @@ __device__ __forceinline__ void store_out(const LinearArgs& a, int t, int col, f
 
 int launch_linear_simt(const LinearArgs& a, cudaStream_t st);
 // Tensor-core (tcgen05) weight-streaming kernel; returns MLORA_OK or an error.
+// Grouped form of the tensor-core kernel: see mlora_grouped_linear.
+struct GroupedArgs {
+  LinearArgs a;            // x, ldx, W (packed, all groups), y, ldy, T (rows per group without a table), in, out, flags
+  const int32_t* table;    // see mlora_grouped_linear
+  const int32_t* gather;
+  int x_rows, n_groups, tile_rows, x_cols, y_cols;
+  const bf16* gate;
+  int64_t ld_gate;
+};
+size_t grouped_tc_workspace(int tile_rows);
+int launch_grouped_tc(const GroupedArgs& g, void* work, size_t work_bytes, cudaStream_t st);
 bool linear_tc_supported(const LinearArgs& a);
 size_t linear_tc_workspace(int T, int in, int out);
 void linear_tc_plan(int T, int in, int out, int32_t* v12);

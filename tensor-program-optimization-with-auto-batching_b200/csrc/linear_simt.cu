@@ -105,7 +105,7 @@ __global__ void __launch_bounds__(256) linear_simt_kernel(LinearArgs a) {
     if (lane < TT && t < a.T) {
       v0 += lora_expand(a, t, row0);
       if (SILU) v1 += lora_expand(a, t, row1);
-      store_out(a, t, SILU ? unit : row0, SILU ? silu_mul(v0, v1) : v0);
+      store_out(a, t, SILU ? unit : row0, SILU ? silu_mul(v0, v1) : act_one(v0, a.flags & (MLORA_ACT_RELU2 | MLORA_ACT_GELU)));
     }
   }
 }

@@ -1,12 +1,11 @@
-"""Paged KV cache: device pages + block tables, host-side page allocator.
+"""Paged caches: device pages + block tables, host-side page allocator.
 
 Stands in for the object ``vm["create_paged_kv_cache"]`` returns and for the
 ``vm.builtin.kv_state_*`` functions the reference executor calls
 (``tvm/llama_auto_batcher/llama_exec_graph.py:38-46,66,75-79,85,121-127``;
 cache parameters ``tvm/llama_auto_batcher/llama_for_causal_lm.py:148-174``).
 
-Layout in HBM: one tensor ``[n_layers, 2, n_pages, Hkv, page_size, D]`` bf16
-(K pages then V pages of a layer), a block table ``[max_batch, max_pages]``
+:class:`PagedCache` is the bookkeeping, shared by all kinds of cache: a block table ``[max_batch, max_pages]``
 int32 and ``seq_lens [max_batch]`` int32.  Page ids are handed out by a host
 free list; the device tables are refreshed with small async copies when they
 change.  A decode step captured in a CUDA graph advances ``seq_lens`` on the
@@ -21,12 +20,12 @@ import torch
 from . import ops
 
 
-class PagedKVCache:
-    def __init__(self, n_layers, n_kv_heads, head_dim, max_batch, max_total_seq_len, prefill_chunk_size,
-                 page_size, device, max_seq_len=None):
+class PagedCache:
+    """Sequences, slots, page ids and block table; what a page holds is up to the subclass."""
+
+    def __init__(self, max_batch, max_total_seq_len, prefill_chunk_size, page_size, device, max_seq_len=None):
         if page_size not in (16, 32):
             raise ValueError("page_size must be 16 or 32")
-        self.n_layers, self.Hkv, self.D = n_layers, n_kv_heads, head_dim
         self.max_batch, self.page_size = int(max_batch), int(page_size)
         self.prefill_chunk_size = int(prefill_chunk_size)
         self.device = torch.device(device)
@@ -35,8 +34,6 @@ class PagedKVCache:
         self.n_pages = (int(max_total_seq_len) + ps - 1) // ps + self.max_batch
         per_seq = int(max_seq_len) if max_seq_len else int(max_total_seq_len)
         self.max_pages = min((per_seq + ps - 1) // ps + 1, self.n_pages)
-        self.pages = torch.zeros(n_layers, 2, self.n_pages, n_kv_heads, ps, head_dim, dtype=torch.bfloat16,
-                                 device=self.device)
         self.block_table = torch.zeros(self.max_batch, self.max_pages, dtype=torch.int32, device=self.device)
         self.seq_lens = torch.zeros(self.max_batch, dtype=torch.int32, device=self.device)
         # host mirrors; device refreshes go through a fresh pinned staging tensor per copy, so a
@@ -48,13 +45,6 @@ class PagedKVCache:
         self._free_slots = list(range(self.max_batch - 1, -1, -1))
         self._n_pages_of = {}        # sid -> pages held
         self._pending = None
-
-    # -- layer views -----------------------------------------------------------------------------
-    def k_pages(self, layer):
-        return self.pages[layer, 0]
-
-    def v_pages(self, layer):
-        return self.pages[layer, 1]
 
     # -- sequences -----------------------------------------------------------------------------
     def add_sequence(self, sid):
@@ -138,29 +128,67 @@ class PagedKVCache:
             self._len_host[self._slot_of[int(sid)]] += n_steps
 
     # -- checks used by tests ---------------------------------------------------------------------
-    def gather(self, sid, layer):
-        """(K, V) of a sequence as dense [n, Hkv, D] tensors (block-table gather)."""
+    def _gather_pages(self, pages, sid):
+        """The first ``length(sid)`` rows of a sequence out of ``pages`` [n_pages, page_size, ...]."""
         slot = self._slot_of[sid]
         n = int(self._len_host[slot])
-        ps = self.page_size
-        n_pg = (n + ps - 1) // ps
+        n_pg = (n + self.page_size - 1) // self.page_size
         idx = torch.from_numpy(self._bt_host[slot, :n_pg].astype(np.int64)).to(self.device)
-        out = []
-        for kv in (0, 1):
-            g = self.pages[layer, kv][idx].permute(0, 2, 1, 3).reshape(n_pg * ps, self.Hkv, self.D)
-            out.append(g[:n])
-        return out
+        return pages[idx].flatten(0, 1)[:n]
+
+
+class PagedKVCache(PagedCache):
+    """Keys and values per layer and head: ``[n_layers, 2, n_pages, Hkv, page_size, D]`` bf16."""
+
+    def __init__(self, n_layers, n_kv_heads, head_dim, max_batch, max_total_seq_len, prefill_chunk_size,
+                 page_size, device, max_seq_len=None):
+        super().__init__(max_batch, max_total_seq_len, prefill_chunk_size, page_size, device, max_seq_len)
+        self.n_layers, self.Hkv, self.D = n_layers, n_kv_heads, head_dim
+        self.pages = torch.zeros(n_layers, 2, self.n_pages, n_kv_heads, self.page_size, head_dim, dtype=torch.bfloat16,
+                                 device=self.device)
+
+    # -- layer views -----------------------------------------------------------------------------
+    def k_pages(self, layer):
+        return self.pages[layer, 0]
+
+    def v_pages(self, layer):
+        return self.pages[layer, 1]
+
+    def gather(self, sid, layer):
+        """(K, V) of a sequence as dense [n, Hkv, D] tensors (block-table gather)."""
+        return [self._gather_pages(self.pages[layer, kv].transpose(1, 2), sid) for kv in (0, 1)]
+
+
+class PagedLatentCache(PagedCache):
+    """One latent vector per token for every layer that computes latents: ``[n_pages, page_size, pitch]`` per such
+    layer.  Layers that attend to another layer's latents hold nothing and read that layer's pages.
+
+    ``ranks``: layer -> kv_rank of the layers that own latents (the pitch is the rank rounded up to 8)."""
+
+    def __init__(self, ranks, max_batch, max_total_seq_len, prefill_chunk_size, page_size, device, max_seq_len=None,
+                 dtype=torch.bfloat16):
+        super().__init__(max_batch, max_total_seq_len, prefill_chunk_size, page_size, device, max_seq_len)
+        self.ranks = dict(ranks)
+        self.pages = {l: torch.zeros(self.n_pages, self.page_size, -(-r // 8) * 8, dtype=dtype, device=self.device)
+                      for l, r in self.ranks.items()}
+
+    def latent_pages(self, layer):
+        return self.pages[layer]
+
+    def gather(self, sid, layer):
+        """Latents of a sequence, dense [n, kv_rank]."""
+        return self._gather_pages(self.pages[layer], sid)[:, :self.ranks[layer]]
 
 
 # The three global functions of the reference's runtime, same names and argument order.
-def kv_state_add_sequence(kv: PagedKVCache, sid):
+def kv_state_add_sequence(kv: PagedCache, sid):
     kv.add_sequence(int(sid))
 
 
-def kv_state_begin_forward(kv: PagedKVCache, seq_ids, append_lens):
+def kv_state_begin_forward(kv: PagedCache, seq_ids, append_lens):
     kv._rows = kv.begin_forward(list(seq_ids), list(append_lens))
 
 
-def kv_state_end_forward(kv: PagedKVCache):
+def kv_state_end_forward(kv: PagedCache):
     kv.end_forward()
     kv._rows = None

@@ -27,6 +27,7 @@ import numpy as np
 import torch
 
 from . import ops
+from .engine import DecodeGraph, DecodeSession, EngineBase  # noqa: F401  (also reached as model.DecodeSession)
 from .kv_cache import PagedKVCache
 from .ops import LoraStack, LORA_PER_ROW, OUT_F32, SHARE_LORA_KERNEL, SILU_MUL
 
@@ -243,6 +244,14 @@ class PackedLlama:
         self.ranks_host[slot] = 0
         self._free_slots.append(slot)
 
+    # -- what the model is served with ------------------------------------------------------------------------
+    def new_cache(self, max_batch, max_total_seq_len, prefill_chunk, page_size=16, max_seq_len=None):
+        return PagedKVCache(self.L, self.Hkv, self.D, max_batch, max_total_seq_len, prefill_chunk, page_size, self.device,
+                            max_seq_len=max_seq_len)
+
+    def new_engine(self, kv, max_rows):
+        return Engine(self, kv, max_rows)
+
     def weight_bytes(self):
         """Bytes of base weights one decode step streams (all layers + final norm + lm_head)."""
         n = self.norm.numel() + self.lm_head.numel()
@@ -258,7 +267,7 @@ class PackedLlama:
         return n
 
 
-class Engine:
+class Engine(EngineBase):
     """Runs prefill / decode forwards of a :class:`PackedLlama` over a :class:`PagedKVCache`.
 
     All activations live in buffers sized for ``max_rows`` rows, allocated once, so a forward does
@@ -267,7 +276,7 @@ class Engine:
     def __init__(self, model: PackedLlama, kv: PagedKVCache, max_rows: int, collective=None):
         """``collective`` (tensor parallelism only): object with ``all_reduce_sum(t)`` (in place) and
         ``all_gather(t) -> [G, *t.shape]``; see ``sharding.DistCollective``."""
-        self.m, self.kv, self.max_rows = model, kv, int(max_rows)
+        super().__init__(model, kv, max_rows)
         self.coll = collective
         if model.tp_size > 1 and collective is None:
             raise ValueError("a tensor-parallel model needs a collective")
@@ -283,14 +292,6 @@ class Engine:
         self.y = torch.zeros(T, m.H, **bf)
         self.act = torch.zeros(T, m.I, **bf)
         self.u = torch.zeros(T, max(3 * m.r_max, 8), **f32)
-        self.logits = torch.zeros(T, m.V, **f32)
-        self.next_tok = torch.zeros(T, dtype=torch.int32, device=dev)
-        self.tokens = torch.zeros(T, dtype=torch.int32, device=dev)
-        self.slots = torch.full((T,), -1, dtype=torch.int32, device=dev)
-        self.row_slot = torch.zeros(T, dtype=torch.int32, device=dev)
-        self.row_pos = torch.zeros(T, dtype=torch.int32, device=dev)
-        self.last_rows = torch.zeros(T, dtype=torch.int32, device=dev)
-        self.iota = torch.arange(T, dtype=torch.int32, device=dev)
         self.xn_last = torch.zeros(T, m.H, **bf)
         # scratch sized for the largest projection of this model at max_rows
         lib = ops._lib.lib()
@@ -313,7 +314,6 @@ class Engine:
         self.pf_status = torch.zeros(1, dtype=torch.int32, device=dev)
         self._n_pf_tiles = 0
         self._graphs = {}
-        self.n_distinct = 0  # distinct adapters among the rows staged for the next pass (set with self.slots)
         self.fuse_norm_shrink = os.environ.get("MLORA_FUSE_NORM_SHRINK", "1") != "0"
         # decode passes of <= 32 rows: the residual add + RMSNorm between the o projection and gate|up folded into the two
         # projections' epilogues (mlora_linear_norm) -- one launch fewer per layer.  Measured on the benchmark's step: the
@@ -326,21 +326,6 @@ class Engine:
         self.use_chain = os.environ.get("MLORA_CHAIN", "0") == "1"
         # "2": only gate|up -> down (two projections with nothing between them) as one launch
         self.chain_mlp = os.environ.get("MLORA_CHAIN", "0") == "2"
-
-    # ------------------------------------------------------------------------------------------
-    def status_word(self) -> int:
-        """Status word of the projection kernels' scratch (synchronises): non-zero after a bounded wait expired
-        somewhere since the buffer was last cleared; the outputs since then are undefined."""
-        return ops.status_word(self.ws_linear)
-
-    def check_status(self):
-        """Raises if a projection kernel gave up a bounded wait, after re-zeroing the scratch (arrival counters of
-        split tiles may be stale after such a failure) so that the engine stays usable."""
-        st = self.status_word()
-        if st:
-            self.ws_linear.zero_()
-            raise RuntimeError(f"mlora: a projection kernel gave up a bounded wait (status bits {st:#x}); "
-                               "the results of this pass are undefined")
 
     @staticmethod
     def _full_rank(stack):
@@ -468,6 +453,23 @@ class Engine:
         ops.argmax(self.logits[:T], out=self.next_tok[:T])
         return self.logits[:T], self.next_tok[:T]
 
+    def _begin_prompt_pass(self, chunk):
+        # tiles of the tensor-core prompt attention: <= 128 consecutive rows of one sequence each
+        tiles = [(self.kv.slot(sid), r0 + off, min(128, n - off), p0 + off)
+                 for sid, r0, n, p0 in chunk for off in range(0, n, 128)]
+        self._n_pf_tiles = 0
+        if self.tc_prefill and len(tiles) <= self.pf_tiles.shape[0]:
+            self._stage(self.pf_tiles.view(-1), np.asarray(tiles, dtype=np.int32).reshape(-1), torch.int32)
+            self._n_pf_tiles = len(tiles)
+
+    def _end_prompt_pass(self):
+        self._n_pf_tiles = 0
+
+    def _check_prompt_status(self):
+        if int(self.pf_status.item()):
+            self.pf_status.zero_()
+            raise RuntimeError("mlora: the prompt attention kernel gave up a bounded wait; this pass's results are undefined")
+
     def forward(self, T: int, fused_append: bool, use_lora: bool = True, lm_rows=None, n_lm=None, hidden=None):
         """One pass over the T rows staged in self.tokens / self.slots / self.row_slot /
         self.row_pos.  Logits (fp32) land in self.logits[:n_lm], greedy tokens in self.next_tok.
@@ -561,232 +563,3 @@ class Engine:
             tk.copy_(allp[win, torch.arange(n_lm, device=lg.device), 1].int())
         return self.logits[:n_lm], self.next_tok[:n_lm]
 
-    # ------------------------------------------------------------------------------------------
-    def _stage(self, dst, values, dtype):
-        t = torch.as_tensor(np.asarray(values), dtype=dtype)
-        dst[: t.numel()].copy_(t.pin_memory(), non_blocking=True)
-
-    def prefill(self, seq_ids, prompts, adapter_slots, use_lora=True):
-        """Prefill whole prompts (lists of token ids) of already-added sequences, chunked to
-        max_rows rows per pass.  Returns (logits [n_seq,V] fp32, next tokens [n_seq] int32)."""
-        kv = self.kv
-        out_logits = torch.empty(len(seq_ids), self.m.V, dtype=torch.float32, device=self.m.device)
-        out_tok = torch.empty(len(seq_ids), dtype=torch.int32, device=self.m.device)
-        # rows: (seq index, position) in sequence order, cut into chunks
-        pending = [(i, 0) for i in range(len(seq_ids))]
-        while pending:
-            rows_left = self.max_rows
-            chunk = []  # (seq index, start, n)
-            nxt = []
-            for i, start in pending:
-                n_total = len(prompts[i])
-                if rows_left == 0:
-                    nxt.append((i, start))
-                    continue
-                n = min(rows_left, n_total - start)
-                chunk.append((i, start, n))
-                rows_left -= n
-                if start + n < n_total:
-                    nxt.append((i, start + n))
-            pending = nxt
-            T = sum(n for _, _, n in chunk)
-            toks = np.concatenate([np.asarray(prompts[i][s:s + n], dtype=np.int32) for i, s, n in chunk])
-            slots = np.concatenate([np.full(n, adapter_slots[i], dtype=np.int32) for i, _, n in chunk])
-            row_slot, row_pos = kv.begin_forward([seq_ids[i] for i, _, _ in chunk], [n for _, _, n in chunk])
-            self._stage(self.tokens, toks, torch.int32)
-            self._stage(self.slots, slots, torch.int32)
-            self.n_distinct = len({int(s) for s in slots if s >= 0})
-            self.row_slot[:T].copy_(row_slot)
-            self.row_pos[:T].copy_(row_pos)
-            # tiles of the tensor-core prompt attention: <= 128 consecutive rows of one sequence each
-            tiles, a0 = [], 0
-            for i, s0, n in chunk:
-                for off in range(0, n, 128):
-                    tiles.append((kv.slot(seq_ids[i]), a0 + off, min(128, n - off), s0 + off))
-                a0 += n
-            self._n_pf_tiles = 0
-            if self.tc_prefill and len(tiles) <= self.pf_tiles.shape[0]:
-                self._stage(self.pf_tiles.view(-1), np.asarray(tiles, dtype=np.int32).reshape(-1), torch.int32)
-                self._n_pf_tiles = len(tiles)
-            ends, fin, a = [], [], 0
-            for i, s, n in chunk:
-                a += n
-                if s + n == len(prompts[i]):
-                    ends.append(a - 1)
-                    fin.append(i)
-            if ends:
-                self._stage(self.last_rows, ends, torch.int32)
-                lg, tk = self.forward(T, False, use_lora, self.last_rows, len(ends))
-                idx = torch.tensor(fin, device=self.m.device)
-                out_logits[idx] = lg
-                out_tok[idx] = tk
-            else:
-                self._stage(self.last_rows, [T - 1], torch.int32)
-                self.forward(T, False, use_lora, self.last_rows, 1)
-            kv.end_forward()
-            self._n_pf_tiles = 0
-        self.check_status()  # (synchronises; prefill is not the latency-critical call)
-        if int(self.pf_status.item()):
-            self.pf_status.zero_()
-            raise RuntimeError("mlora: the prompt attention kernel gave up a bounded wait; this pass's results are undefined")
-        return out_logits, out_tok
-
-    def decode(self, seq_ids, tokens, adapter_slots, use_lora=True):
-        """One eager decode step (host builds the row tables, as the reference's executor does)."""
-        B = len(seq_ids)
-        row_slot, row_pos = self.kv.begin_forward(seq_ids, [1] * B)
-        self._stage(self.tokens, tokens, torch.int32)
-        self._stage(self.slots, adapter_slots, torch.int32)
-        self.n_distinct = len({int(s) for s in adapter_slots if s >= 0})
-        self.row_slot[:B].copy_(row_slot)
-        self.row_pos[:B].copy_(row_pos)
-        out = self.forward(B, True, use_lora)
-        self.kv.end_forward()
-        return out
-
-    # -- CUDA-graph decode: the whole step, including position bookkeeping, is one graph ---------------
-    def capture_decode(self, seq_ids, adapter_slots, use_lora=True, reserve_tokens=0, feed_back=True):
-        """Capture a decode step for this batch.  Rows follow ``seq_ids``; each replay consumes
-        self.tokens[:B] (device) and leaves greedy tokens in self.next_tok[:B]."""
-        B, kv = len(seq_ids), self.kv
-        for sid in seq_ids:
-            kv.reserve(sid, kv.length(sid) + reserve_tokens + 1)
-        self._stage(self.row_slot, [kv.slot(s) for s in seq_ids], torch.int32)
-        self._stage(self.slots, adapter_slots, torch.int32)
-        self.n_distinct = len({int(s) for s in adapter_slots if s >= 0})
-        torch.cuda.synchronize()
-        saved = kv.seq_lens.clone()
-
-        def step():
-            ops.kv_begin_decode(self.row_slot[:B], kv.seq_lens, self.row_pos[:B])
-            self.forward(B, True, use_lora)
-            if feed_back:  # the greedy tokens become the next step's input without leaving the device
-                self.tokens[:B].copy_(self.next_tok[:B])
-
-        side = torch.cuda.Stream()
-        side.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(side):
-            step()  # warm-up outside capture (lazy module loading, attribute setting)
-        torch.cuda.current_stream().wait_stream(side)
-        torch.cuda.synchronize()
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
-            step()
-        kv.seq_lens.copy_(saved)  # warm-up advanced the device lengths; capture itself runs nothing
-        torch.cuda.synchronize()
-        return DecodeGraph(self, g, list(seq_ids), B)
-
-
-class DecodeGraph:
-    def __init__(self, engine, graph, seq_ids, B):
-        self.engine, self.graph, self.seq_ids, self.B = engine, graph, seq_ids, B
-        self._headroom = 0  # replays known to be covered by reserved pages (re-counted when it runs out)
-
-    def replay(self):
-        """One token for every row: consumes engine.tokens[:B], leaves greedy tokens in
-        engine.next_tok[:B] (and, when captured with feed_back, back in engine.tokens).
-        The step appends one token per sequence through block-table entries that must exist already:
-        pages are reserved here when the host allocator still has some, else the replay is refused."""
-        kv = self.engine.kv
-        if self._headroom <= 0:
-            for sid in self.seq_ids:
-                kv.reserve(sid, kv.length(sid) + 1)  # raises when the pool or the row's table is exhausted
-            self._headroom = min(kv.tokens_reserved(sid) - kv.length(sid) for sid in self.seq_ids)
-        self._headroom -= 1
-        self.graph.replay()
-        self.engine.kv.note_device_decode(self.seq_ids)
-
-
-class DecodeSession:
-    """The batched greedy loop of one fused decode node (``tvm/llama_auto_batcher/llama_exec_graph.py:102-141``)
-    with the batch state on the device: sequences finish on their end-of-sequence token or their own
-    ``max_gen_len`` and leave the batch without the host rebuilding anything.  Every step is a CUDA-graph replay
-    of ``decode_step_begin -> forward -> decode_step_end`` captured for a bucket of rows (powers of two up to the
-    node's size); the host only learns the live count (4 bytes, every ``sync_every`` steps) to pick the bucket and
-    to stop, and reads all generated tokens once at the end.
-
-    ``seq_ids`` must already be in bucketing order (``LlamaSeqInfo.order_seqs``): rows of one adapter adjacent."""
-
-    def __init__(self, engine: Engine, seq_ids, adapter_slots, first_tokens, max_gen, eos_id=None, use_lora=True):
-        self.eng, self.seq_ids, self.use_lora = engine, list(seq_ids), use_lora
-        kv, dev, n = engine.kv, engine.m.device, len(seq_ids)
-        self.n = n
-        self.max_len = int(max(max_gen)) + 1  # (a sequence always takes part in the node's first step)
-        i32 = lambda v: torch.as_tensor(np.asarray(v, dtype=np.int32)).pin_memory().to(dev, non_blocking=True)
-        self.live = torch.ones(n, dtype=torch.int32, device=dev)
-        self.seq_slot = i32([kv.slot(s) for s in seq_ids])
-        self.adapter_slot = i32(adapter_slots)
-        self.last_tok = i32(first_tokens)
-        self.max_gen = i32(max_gen)
-        self.gen_count = torch.ones(n, dtype=torch.int32, device=dev)  # the prefill's token is the first one
-        self.out_tokens = torch.zeros(n, self.max_len, dtype=torch.int32, device=dev)
-        self.out_tokens[:, 0] = self.last_tok
-        self.row_src = torch.full((max(n, 1),), -1, dtype=torch.int32, device=dev)
-        self.n_live = torch.zeros(1, dtype=torch.int32, device=dev)
-        self._n_live_host = torch.zeros(1, dtype=torch.int32).pin_memory()
-        self.eos_id = -1 if eos_id is None else int(eos_id)
-        self.n_distinct = len({int(a) for a in adapter_slots if a >= 0})
-        for sid, g in zip(seq_ids, max_gen):
-            kv.reserve(sid, kv.length(sid) + int(g) + 1)
-        self._graphs = {}
-        self.steps = 0
-        self.d2h_bytes = 0
-
-    def _step(self, rows):
-        e = self.eng
-        ops.decode_step_begin(self.live, self.seq_slot, self.adapter_slot, self.last_tok, rows, e.kv.seq_lens,
-                              self.row_src, e.row_slot, e.row_pos, e.slots, e.tokens, self.n_live)
-        e.n_distinct = self.n_distinct
-        e.forward(rows, True, self.use_lora)
-        ops.decode_step_end(self.row_src, e.next_tok, rows, self.live, self.last_tok, self.gen_count, self.max_gen,
-                            self.out_tokens, self.eos_id, self.n_live)
-
-    def _graph(self, rows):
-        g = self._graphs.get(rows)
-        if g is not None:
-            return g
-        e = self.eng
-        state = (self.live, self.last_tok, self.gen_count, self.out_tokens, e.kv.seq_lens, self.n_live)
-        saved = [t.clone() for t in state]
-        side = torch.cuda.Stream()
-        side.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(side):
-            self._step(rows)  # warm-up outside capture; its effects are undone below
-        torch.cuda.current_stream().wait_stream(side)
-        torch.cuda.synchronize()
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
-            self._step(rows)
-        for t, s in zip(state, saved):
-            t.copy_(s)
-        torch.cuda.synchronize()
-        self._graphs[rows] = g
-        return g
-
-    @staticmethod
-    def bucket(n_live, n):
-        """Rows of the step that serves ``n_live`` live sequences: the next power of two, capped at the node's size."""
-        b = 1
-        while b < n_live:
-            b *= 2
-        return min(b, n)
-
-    def run(self, sync_every=1):
-        """Runs until every sequence has finished.  Returns the token lists (first token included) in the order of
-        ``seq_ids``."""
-        bound = self.n  # upper bound of the live count (sequences only ever leave)
-        while bound > 0:
-            g = self._graph(self.bucket(bound, self.n))
-            for _ in range(max(1, sync_every)):
-                g.replay()
-                self.steps += 1
-            self._n_live_host.copy_(self.n_live, non_blocking=True)
-            torch.cuda.current_stream().synchronize()
-            self.d2h_bytes += 4
-            bound = int(self._n_live_host[0])
-        counts = self.gen_count.cpu().tolist()
-        toks = self.out_tokens.cpu().tolist()
-        self.d2h_bytes += 4 * (self.n + self.out_tokens.numel())
-        for sid, c in zip(self.seq_ids, counts):
-            self.eng.kv.note_device_decode([sid], c - 1)
-        return [t[:c] for t, c in zip(toks, counts)]

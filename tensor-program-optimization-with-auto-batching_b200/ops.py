@@ -488,3 +488,157 @@ def decode_step_end(row_src, next_tok, n_rows, live, last_tok, gen_count, max_ge
 
 def launch_count() -> int:
     return int(_lib.lib().mlora_launch_count())
+
+
+# ---------------------------------------------------------------- plain feed-forward activations, grouped projections, 32-bit
+ACT_RELU2, ACT_GELU = 256, 512
+F32_TILE_ROWS = 64  # rows per tile of the 32-bit kernel
+
+
+class GroupedWeight:
+    """``n`` weights of one shape [out, in] for :func:`grouped_linear` (bf16: pre-tiled one after the other; fp32: as is)."""
+
+    def __init__(self, W):
+        _need_cuda(W)
+        self.n, self.out, self.in_ = W.shape
+        self.dtype = W.dtype
+        if W.dtype == torch.float32:
+            self.data = W.contiguous()
+            return
+        per = _lib.lib().mlora_packed_weight_bytes(self.out, self.in_)
+        self.data = torch.empty(self.n * per, dtype=torch.uint8, device=W.device)
+        for g in range(self.n):
+            w = W[g].contiguous()
+            check(_lib.lib().mlora_pack_weight(_ptr(w), self.out, self.in_, _ptr(self.data[g * per:]), _stream()), "mlora_pack_weight")
+
+    def numel(self):
+        return self.n * self.out * self.in_
+
+
+def grouped_tile_rows(rows_per_group: float, dtype=torch.bfloat16) -> int:
+    """Rows per tile that suit an average group: wide enough that most groups are one tile when there are few rows (their
+    weights are then streamed once), and the largest tiles when there are many."""
+    if dtype == torch.float32:
+        return F32_TILE_ROWS
+    return 16 if rows_per_group <= 4 else 32 if rows_per_group <= 12 else 64 if rows_per_group <= 32 else \
+        128 if rows_per_group <= 192 else 256
+
+
+def grouped_linear(x, W: GroupedWeight, out, T=0, x_cols=0, y_cols=0, plan=None, gather=False, tile_rows=None, flags=0,
+                   gate=None, work=None):
+    """``mlora_grouped_linear`` (bf16) or ``mlora_linear_f32``.  Without ``plan`` every group works on the rows [0, T) and its
+    own column slices; with a :class:`MoePlan`, on its rows of the plan (``gather``: x rows are tokens, else plan rows)."""
+    _need_cuda(x, out)
+    tiles = plan.tiles if plan is not None else None
+    rows = plan.rows if gather else None
+    if W.dtype == torch.float32:
+        check(_lib.lib().mlora_linear_f32(
+            _ptr(x), x.stride(0), x_cols, _ptr(rows), _ptr(W.data), _ptr(out), out.stride(0), y_cols, _ptr(tiles),
+            plan.max_tiles if plan is not None else 0, W.n, T, W.in_, W.out, flags, _ptr(gate),
+            gate.stride(0) if gate is not None else 0, _stream()), "mlora_linear_f32")
+        return out
+    tr = plan.tile_rows if plan is not None else tile_rows
+    check(_lib.lib().mlora_grouped_linear(
+        _ptr(x), x.stride(0), x.shape[0], x_cols, _ptr(rows), _ptr(W.data), _ptr(out), out.stride(0), y_cols, _ptr(tiles),
+        W.n, T, tr, W.in_, W.out, flags, _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(work), work.numel(),
+        _stream()), "mlora_grouped_linear")
+    return out
+
+
+def linear_f32(x, W, flags=0, out=None):
+    """y = act(x W^T) in true 32-bit; W [out, in] fp32."""
+    _need_cuda(x, W)
+    T, K = x.shape
+    if out is None:
+        out = torch.empty(T, W.shape[0], dtype=torch.float32, device=x.device)
+    check(_lib.lib().mlora_linear_f32(_ptr(x), x.stride(0), 0, None, _ptr(W), _ptr(out), out.stride(0), 0, None, 0, 1, T, K,
+                                      W.shape[0], flags, None, 0, _stream()), "mlora_linear_f32")
+    return out
+
+
+# ---------------------------------------------------------------- mixture of experts
+class MoePlan:
+    """Buffers of the routing of up to ``max_tokens`` tokens (allocated once: a forward allocates nothing)."""
+
+    def __init__(self, max_tokens, n_experts, top, device):
+        self.E, self.top = n_experts, top
+        n = max_tokens * top
+        i32 = dict(dtype=torch.int32, device=device)
+        self.expert, self.pos, self.rows = torch.zeros(n, **i32), torch.zeros(n, **i32), torch.zeros(n, **i32)
+        self.weight = torch.zeros(n, dtype=torch.float32, device=device)
+        self.tiles = torch.zeros(4 * (2 + n // 16 + min(n_experts, n)), **i32)
+        self.work = new_workspace(_lib.lib().mlora_moe_plan_workspace(max_tokens, n_experts, top), device)
+        self.tile_rows = self.max_tiles = 0
+
+
+def moe_plan(logits, bias, plan: MoePlan, T, tile_rows):
+    _need_cuda(logits, bias)
+    plan.tile_rows = tile_rows
+    plan.max_tiles = T * plan.top // tile_rows + min(plan.E, T * plan.top)
+    check(_lib.lib().mlora_moe_plan(_ptr(logits), logits.stride(0), _ptr(bias), T, plan.E, plan.top, tile_rows,
+                                    _ptr(plan.expert), _ptr(plan.weight), _ptr(plan.pos), _ptr(plan.rows), _ptr(plan.tiles),
+                                    _ptr(plan.work), plan.work.numel(), _stream()), "mlora_moe_plan")
+    return plan
+
+
+# ---------------------------------------------------------------- dynamic tanh norm
+def residual_dyt(delta, res, w, b, alpha, out, expert_rows=None, plan: MoePlan = None, rows=None):
+    """res += delta (+ the plan's weighted expert rows); out = tanh(alpha res) w + b; see ``mlora_residual_dyt``."""
+    _need_cuda(res, w)
+    check(_lib.lib().mlora_residual_dyt(
+        _ptr(delta), _ptr(expert_rows), _ptr(plan.pos) if plan is not None else None,
+        _ptr(plan.weight) if plan is not None else None, plan.top if plan is not None else 0, _ptr(res), _ptr(rows), _ptr(w),
+        _ptr(b), _ptr(alpha), _ptr(out), out.shape[0], res.shape[1], int(out.dtype == torch.float32), _stream()),
+        "mlora_residual_dyt")
+    return out
+
+
+# ---------------------------------------------------------------- latent attention
+def latent_append(x, R, w, eps, pages, block_table, row_slot, row_pos):
+    """x [T, >= R] (a column slice is fine): normalised into the rows' places in ``pages``."""
+    _need_cuda(x, pages)
+    check(_lib.lib().mlora_latent_append(_ptr(x), x.stride(0), R, _ptr(w), eps, _ptr(pages), pages.shape[2], pages.shape[1],
+                                         _ptr(block_table), block_table.shape[1], _ptr(row_slot), _ptr(row_pos), x.shape[0],
+                                         int(x.dtype == torch.float32), _stream()), "mlora_latent_append")
+
+
+def latent_gather(pages, block_table, segs, n_segs, max_tokens, out):
+    check(_lib.lib().mlora_latent_gather(_ptr(pages), pages.shape[2], pages.shape[1], _ptr(block_table), block_table.shape[1],
+                                         _ptr(segs), n_segs, max_tokens, _ptr(out), _stream()), "mlora_latent_gather")
+    return out
+
+
+def prefill_attention_dense(q, kv, v_col, tiles, n_tiles, H, Dk, Dv, scale, out, gate=None, status=None):
+    check(_lib.lib().mlora_prefill_attention_dense(
+        _ptr(q), q.stride(0), _ptr(kv), kv.stride(0), kv.shape[0], v_col, _ptr(tiles), n_tiles, H, Dk, Dv, scale, _ptr(gate),
+        gate.stride(0) if gate is not None else 0, q.shape[0], _ptr(out), out.stride(0), _ptr(status), _stream()),
+        "mlora_prefill_attention_dense")
+    return out
+
+
+LATENT_TC_MAX_RANK = 512
+
+
+def latent_attention_splits(T, H, max_keys) -> int:
+    return int(_lib.lib().mlora_latent_attention_splits(T, H, max_keys))
+
+
+def latent_attention_workspace(T, H, q_pitch, n_splits) -> int:
+    return int(_lib.lib().mlora_latent_attention_workspace(T, H, q_pitch, n_splits))
+
+
+def latent_attention(qa, R, H, pages, block_table, row_slot, row_pos, scale, out, n_splits=1, work=None, status=None, simt=False):
+    """qa, out [T, H * q_pitch].  Tensor cores for bf16 and R <= 512, else (or with ``simt``) the CUDA-core kernel."""
+    _need_cuda(qa, pages)
+    T, pitch = qa.shape[0], qa.shape[1] // H
+    if simt or qa.dtype == torch.float32 or R > LATENT_TC_MAX_RANK:
+        check(_lib.lib().mlora_latent_attention_simt(
+            _ptr(qa), pitch, _ptr(pages), R, pages.shape[2], pages.shape[1], _ptr(block_table), block_table.shape[1],
+            _ptr(row_slot), _ptr(row_pos), T, H, scale, _ptr(out), int(qa.dtype == torch.float32), _stream()),
+            "mlora_latent_attention_simt")
+        return out
+    check(_lib.lib().mlora_latent_attention(
+        _ptr(qa), pitch, _ptr(pages), pages.shape[0], R, pages.shape[2], pages.shape[1], _ptr(block_table),
+        block_table.shape[1], _ptr(row_slot), _ptr(row_pos), T, H, scale, n_splits, _ptr(out), _ptr(work),
+        work.numel() if work is not None else 0, _ptr(status), _stream()), "mlora_latent_attention")
+    return out

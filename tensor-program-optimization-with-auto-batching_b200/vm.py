@@ -33,7 +33,6 @@ import torch
 
 from . import kv_cache as kvc
 from . import ops
-from .model import Engine, PackedLlama
 
 
 class ShapeTuple(tuple):
@@ -78,8 +77,8 @@ def _tensor(x, device, dtype=None):
 
 
 class B200VM:
-    def __init__(self, model: PackedLlama, type_slot_base=(0,)):
-        """``type_slot_base[t]`` = first slot of adapter type ``t`` in the model's packed stacks; the slot of
+    def __init__(self, model, type_slot_base=(0,)):
+        """``model``: any registered model.  ``type_slot_base[t]`` = first slot of adapter type ``t`` in the model's packed stacks; the slot of
         (type t, weight id w) is ``type_slot_base[t] + w`` (the reference uses the raw weight id as the index
         into that type's stack, ``compile_tvm.py:298-313``)."""
         self.model = model
@@ -142,9 +141,8 @@ class B200VM:
 
     def _create_paged_kv_cache(self, max_batch, max_total_seq_len, prefill_chunk, page_size):
         m = self.model
-        kv = kvc.PagedKVCache(m.L, m.Hkv, m.D, int(max_batch[0]), int(max_total_seq_len[0]), int(prefill_chunk[0]),
-                              int(page_size[0]), m.device)
-        self._engines[id(kv)] = Engine(m, kv, max(int(prefill_chunk[0]), int(max_batch[0])))
+        kv = m.new_cache(int(max_batch[0]), int(max_total_seq_len[0]), int(prefill_chunk[0]), int(page_size[0]))
+        self._engines[id(kv)] = m.new_engine(kv, max(int(prefill_chunk[0]), int(max_batch[0])))
         return kv
 
     def _run(self, hidden, kv, type_args, prefill):
