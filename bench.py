@@ -1063,6 +1063,200 @@ def run_kernel_case(which):
     emit({"kernel_case": which, "launches": ops.launch_count()})
 
 
+class KernelTimer:
+    """Times every operator call of an engine pass by itself: L2 flushed (a 256 MB write), CUDA events around the call on
+    the launching stream.  Calls of one operator and shape are averaged; the best of the passes counts."""
+
+    NAMES = ("linear", "grouped_linear", "moe_plan", "residual_dyt", "residual_rmsnorm", "latent_append", "latent_gather",
+             "latent_attention", "prefill_attention_dense", "embed", "argmax", "paged_attention", "prefill_attention",
+             "kv_append_rope")
+
+    def __init__(self, ops, torch, dev, hbm_gbs, tflops):
+        self.ops, self.torch, self.hbm, self.tflops = ops, torch, hbm_gbs, tflops
+        self.flush = torch.zeros(64 << 20, dtype=torch.float32, device=dev)
+        self.calls, self.saved = [], {}
+
+    def cost(self, name, a, k, lens, news):
+        """(label, algorithmic bytes, flops) of a call; ``lens`` / ``news``: context and new rows per sequence."""
+        pairs = sum((l - n) * n + n * (n + 1) / 2 for l, n in zip(lens, news))
+        if name == "linear":
+            x, W, fl = a[0], a[1], k.get("flags", 0)
+            T, (o, i) = x.shape[0], W.shape
+            cols = o // 2 if fl & self.ops.SILU_MUL else o
+            return f"{T} x {i} -> {o}", 2 * o * i + 2 * T * i + (4 if fl & self.ops.OUT_F32 else 2) * T * cols, 2.0 * T * o * i
+        if name == "grouped_linear":
+            x, W, y, plan = a[0], a[1], a[2], k.get("plan")
+            if plan is None:
+                n = k["T"] * W.n
+                return f"{W.n} heads, {k['T']} x {W.in_} -> {W.out}", 2 * (W.numel() + n * (W.in_ + W.out)), 2.0 * n * W.in_ * W.out
+            n, used = y.shape[0], len(set(plan.expert[:y.shape[0]].tolist()))
+            xb = x.shape[0] * W.in_
+            return (f"{used} experts, {n} x {W.in_} -> {W.out}", 2 * (used * W.in_ * W.out + xb + n * W.out),
+                    2.0 * n * W.in_ * W.out)
+        if name in ("residual_dyt", "residual_rmsnorm"):
+            T, H = (a[5].shape[0] if name == "residual_dyt" else a[1].shape[0]), a[1].shape[1]
+            delta, plan = a[0] is not None, k.get("plan")
+            return (f"{T} x {H}" + (f" + {plan.top} expert rows" if plan else ""),
+                    T * H * (4 + 2 + (2 if delta else 0) + (4 if delta or plan else 0) + (2 * plan.top if plan else 0)), 0.0)
+        if name == "latent_attention":
+            qa, R, H = a[0], a[1], a[2]
+            return f"{qa.shape[0]} rows, {H} heads, rank {R}", 2 * R * sum(lens) + 4 * qa.numel(), 4.0 * H * R * pairs
+        if name == "prefill_attention_dense":
+            H, dk, dv = a[5], a[6], a[7]
+            rows = sum(news)
+            return f"{rows} rows, {H} heads", 2 * (dk + dv) * H * (rows + sum(lens)), 2.0 * H * (dk + dv) * pairs
+        if name in ("paged_attention", "prefill_attention"):
+            Hq, Hkv, D = (a[6], a[7], a[8]) if name == "paged_attention" else (a[6], a[7], a[8])
+            return f"{sum(news)} rows, {Hq} heads", 4 * D * Hkv * sum(lens) + 4 * D * Hq * sum(news), 4.0 * Hq * D * pairs
+        if name == "latent_append":
+            return f"{a[0].shape[0]} rows", 4 * a[0].shape[0] * a[1], 0.0
+        if name == "latent_gather":
+            return f"{a[5].shape[0]} rows", 4 * a[5].numel(), 0.0
+        if name == "kv_append_rope":
+            return f"{a[0].shape[0]} rows", 4 * a[0].numel(), 0.0
+        if name == "moe_plan":
+            return f"{a[3]} tokens", 4 * a[3] * (a[2].E + 4 * a[2].top), 0.0
+        if name == "embed":
+            return f"{a[0].numel()} rows", a[0].numel() * a[1].shape[1] * 6, 0.0
+        return f"{a[0].shape[0]} rows", 4 * a[0].numel(), 0.0
+
+    def run(self, fn, lens, news, passes=3):
+        torch, best = self.torch, None
+        for name in self.NAMES:
+            self.saved[name] = getattr(self.ops, name)
+            setattr(self.ops, name, self._timed(name, lens, news))
+        try:
+            for _ in range(passes):
+                self.calls = []
+                fn()
+                torch.cuda.synchronize()
+                us = [1e3 * e0.elapsed_time(e1) for _, _, _, _, e0, e1 in self.calls]
+                best = us if best is None else [min(x, y) for x, y in zip(best, us)]
+        finally:
+            for name, f in self.saved.items():
+                setattr(self.ops, name, f)
+        rows = {}
+        for (name, label, nb, fl, _, _), us in zip(self.calls, best):
+            r = rows.setdefault((name, label), [0, 0.0, nb, fl])
+            r[0] += 1
+            r[1] += us
+        out = []
+        for (name, label), (n, us, nb, fl) in rows.items():
+            roof = max(nb / (self.hbm * 1e3), fl / (self.tflops * 1e6))
+            out.append({"op": name, "shape": label, "calls": n, "us": round(us / n, 1), "roofline_us": round(roof, 2),
+                        "frac": round(roof / (us / n), 3), "bound": "hbm" if nb / (self.hbm * 1e3) >= fl / (self.tflops * 1e6) else "tensor"})
+        return out
+
+    def _timed(self, name, lens, news):
+        f, torch = self.saved[name], self.torch
+
+        def call(*a, **k):
+            label, nb, fl = self.cost(name, a, k, lens, news)
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            self.flush.add_(1.0)
+            self.flush.add_(1.0)
+            e0.record()
+            r = f(*a, **k)
+            e1.record()
+            self.calls.append((name, label, nb, fl, e0, e1))
+            return r
+        return call
+
+
+def run_tevudra(args):
+    """Side measurement (its own JSON line): Tevudra at layer shapes of real models, random weights, beside the framework's
+    Llama path (no adapters) at equal width, heads and head size.  Prefill of 16 x 512 and 2 x 4096 tokens, decode steps (CUDA
+    graph) of 32 requests at contexts of 1024 and 8192; then every kernel of one pass by itself against its roofline."""
+    import numpy as np
+    import torch
+
+    ops, synth, reg = load("ops"), load("synth"), load("registry")
+    load("build").build()
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    hbm, src = measured_peak()
+    peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if src == "measured" else {}
+    tflops = float(peaks.get("bf16_tflops", 1590.0))
+    lines = []
+    for name in args.shapes.split(","):
+        tcfg = synth.tevudra_config(name)
+        W, heads = tcfg["width"], tcfg["layers"][0]["mixer"]["heads"]
+        lcfg = dict(synth.llama_config("llama2-7b"), hidden_size=W, num_attention_heads=heads, num_key_value_heads=heads,
+                    intermediate_size={2048: 5504, 4096: 11008}[W], num_hidden_layers=4, name=f"llama-{W}")
+        for design, cfg in (("tevudra", tcfg), ("llama", lcfg)):
+            w = (synth.tevudra_weights if design == "tevudra" else synth.base_weights)(cfg, dtype=torch.bfloat16, device=dev)
+            model = reg.build_model(cfg, w, device=dev)
+            del w
+            torch.cuda.empty_cache()
+            V = cfg.get("vocab", cfg.get("vocab_size"))
+            line = {"workload": "tevudra", "model": cfg["name"], "layers": 4, "peak_source": src, "dtype": "bf16", "data": "synthetic",
+                    "prefill": [], "decode": [], "kernels": {}}
+            timer = KernelTimer(ops, torch, dev, hbm, tflops)
+            for n_req, length in ((16, 512), (2, 4096)):
+                prompts = [p.tolist() for p in synth.prompts(n_req, length, V)]
+                kv = model.new_cache(n_req, n_req * (length + 32), 8192, PAGE)
+                eng = model.new_engine(kv, 8192)
+
+                def prefill():
+                    for s in range(n_req):
+                        kv.add_sequence(s)
+                    eng.prefill(list(range(n_req)), prompts, [-1] * n_req)
+                    for s in range(n_req):
+                        kv.remove_sequence(s)
+                ms = []
+                for it in range(6):
+                    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                    timer.flush.add_(1.0)
+                    e0.record()
+                    prefill()
+                    e1.record()
+                    torch.cuda.synchronize()
+                    ms.append(e0.elapsed_time(e1))
+                ms = statistics.median(ms[3:])
+                line["prefill"].append({"requests": n_req, "tokens_each": length, "ms": round(ms, 3), "tokens_per_s": round(n_req * length / ms * 1e3)})
+                line["kernels"][f"prefill {n_req}x{length}"] = timer.run(prefill, [length] * n_req, [length] * n_req)
+                del eng, kv
+            B = 32
+            for ctx in (1024, 8192):
+                kv = model.new_cache(B, B * (ctx + 64), B, PAGE, max_seq_len=ctx + 64)
+                eng = model.new_engine(kv, 128)
+                for t in (kv.pages.values() if isinstance(kv.pages, dict) else [kv.pages]):
+                    t.normal_()
+                for s in range(B):
+                    kv.add_sequence(s)
+                    kv.reserve(s, ctx + 48)
+                    kv._len_host[kv.slot(s)] = ctx
+                kv.seq_lens.fill_(ctx)
+                sids, slots = list(range(B)), [-1] * B
+                eng.tokens[:B].copy_(torch.arange(B, dtype=torch.int32, device=dev) * 7)
+                g = eng.capture_decode(sids, slots, reserve_tokens=40)
+                for _ in range(4):
+                    g.replay()
+                e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                e0.record()
+                for _ in range(32):
+                    g.replay()
+                e1.record()
+                torch.cuda.synchronize()
+                ms = e0.elapsed_time(e1) / 32
+                eng.check_status()
+                line["decode"].append({"requests": B, "context": ctx, "ms_per_step": round(ms, 4), "tokens_per_s": round(B / ms * 1e3)})
+                n_ctx = kv.length(0) + 1
+
+                def step():
+                    for s in sids:
+                        kv._len_host[kv.slot(s)] = n_ctx - 1
+                    eng.decode(sids, [1] * B, slots)
+                line["kernels"][f"decode {B} at {ctx}"] = timer.run(step, [n_ctx] * B, [1] * B)
+                del g, eng, kv
+                torch.cuda.empty_cache()
+            lines.append(line)
+            del model
+            torch.cuda.empty_cache()
+    for line in lines:
+        emit(line)
+
+
 _RESULT_FD = None
 
 
@@ -1096,11 +1290,13 @@ def main():
                          "(the number is then not a bench value)")
     ap.add_argument("--kernel-case", default="", choices=["", "linear", "attention", "operator", "prefill", "prefill-lora", "prefill-attn", "expand", "chain"],
                     help="profiling aid: launch one kernel a few times on a small case (> L2, < 1 GB) and exit")
-    ap.add_argument("--workload", default="", choices=["", "13b-shape", "13b-tp", "prefill-heavy"],
+    ap.add_argument("--workload", default="", choices=["", "13b-shape", "13b-tp", "prefill-heavy", "tevudra"],
                     help="side measurements (own JSON line, not the benchmark's): 13b-shape = the 13B shape and adapter "
                          "mix on one GPU; 13b-tp = the tensor-parallel configuration, tp size = number of ranks "
                          "(launch with torch.distributed.run); prefill-heavy = 64 x 512-token prompts, 64 rank-64 adapters on "
-                         "seven projections, Zipf ids, 16 decode tokens")
+                         "seven projections, Zipf ids, 16 decode tokens; tevudra = the Tevudra design beside the Llama path at "
+                         "equal layer sizes, prefill, decode and every kernel against its roofline")
+    ap.add_argument("--shapes", default="tevudra-2048,tevudra-4096", help="tevudra workload: shapes to run")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
@@ -1117,6 +1313,8 @@ def main():
         run_13b_tp(args, rank, world, local_rank)
     elif args.workload == "prefill-heavy":
         run_prefill_heavy(args)
+    elif args.workload == "tevudra":
+        run_tevudra(args)
     elif args.kernel_case:
         run_kernel_case(args.kernel_case)
     elif args.impl == "reference":

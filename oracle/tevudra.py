@@ -70,6 +70,9 @@ def latent_attention(h, c, w_q, w_uk, w_uv, w_g, w_o, heads, dim, vdim, scale):
 
 
 class OracleTevudra:
+    """``margin`` (after a forward): per token the smallest distance, over the layers, between the last chosen expert's
+    logit and the first one left out -- a 16-bit path may choose the other one where it is small."""
+
     def __init__(self, config, params, dtype=torch.float64):
         self.cfg = config
         self.p = {k: (v.to(dtype) if v.is_floating_point() else v) for k, v in params.items()}
@@ -80,6 +83,10 @@ class OracleTevudra:
 
     def _mlp(self, pre, m, h):
         p = self.p
+        if m["kind"] == "moe" and m["router"]["top"] < m["router"]["experts"]:
+            z = torch.sort(h @ p[pre + "router"].T + p[pre + "router.b"], dim=-1, descending=True).values
+            top = m["router"]["top"]
+            self.margin = torch.minimum(self.margin, z[:, top - 1] - z[:, top])
         if m["kind"] == "dense":
             return feed_forward(h, p[pre + "up"], p[pre + "down"], relu2)
         n_exp = m["router"]["experts"]
@@ -92,6 +99,7 @@ class OracleTevudra:
         p, eps = self.p, self.cfg["norm"]["eps"]
         x = p["embed"][torch.as_tensor(tokens, dtype=torch.long)]
         lat, stream = {}, []
+        self.margin = torch.full((len(tokens),), float("inf"), dtype=x.dtype)
         for i, layer in enumerate(self.cfg["layers"]):
             m, pre = layer["mixer"], f"l{i}."
             h = self._norm(pre + "norm1", x)

@@ -103,6 +103,60 @@ def lora_adapters(cfg: dict, n_adapters: int, ranks, targets=ATTN_PROJ, dtype=to
     return out
 
 
+def tevudra_config(name: str) -> dict:
+    """Tevudra shapes with layers like a real model's: four layers, two latents, dense and mixture-of-experts in turn."""
+    w, heads, ff, experts, eff, top, shared = {"tevudra-2048": (2048, 16, 8192, 64, 1408, 6, 2816),
+                                               "tevudra-4096": (4096, 32, 16384, 32, 2048, 4, 4096)}[name]
+    def layer(i):
+        mixer = {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": 512, "scale": 128 ** -0.5}
+        if i % 2:
+            mixer["kv_from"] = i - 1
+            mlp = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared}}
+        else:
+            mlp = {"kind": "dense", "ff": ff}
+        return {"type": "latent_attention", "mixer": mixer, "mlp": mlp}
+    return {"architecture": "Tevudra", "name": name, "vocab": 32000, "width": w, "norm": {"eps": 1e-6},
+            "layers": [layer(i) for i in range(4)]}
+
+
+def tevudra_weights(cfg: dict, dtype=torch.bfloat16, device="cpu") -> dict:
+    """Random weights of a Tevudra configuration: matrices ~ N(0, 1/in), norm weights 1 + N(0, 0.02), alpha 0.5."""
+    g = _gen(SEED_WEIGHTS, device)
+    rnd = lambda *s: torch.randn(*s, generator=g, device=device, dtype=torch.float32)
+    mat = lambda o, i: (rnd(o, i) / math.sqrt(i)).to(dtype)
+    W, V = cfg["width"], cfg["vocab"]
+    p = {"embed": rnd(V, W).to(dtype), "head": mat(V, W)}
+
+    def norm(name):
+        p[name], p[name + ".b"] = (1 + 0.02 * rnd(W)).to(dtype), (0.02 * rnd(W)).to(dtype)
+        p[name + ".alpha"] = torch.tensor(0.5, device=device).to(dtype)
+
+    def feed_forward(name, ff):
+        p[name + ".up"], p[name + ".down"] = mat(ff, W), mat(W, ff)
+
+    norm("final.norm")
+    for i, layer in enumerate(cfg["layers"]):
+        m, f, mix = layer["mixer"], layer["mlp"], f"l{i}.mix."
+        H, R = m["heads"], m["kv_rank"]
+        norm(f"l{i}.norm1")
+        p[mix + "q"], p[mix + "g"], p[mix + "o"] = mat(H * m["dim"], W), mat(H, W), mat(W, H * m["vdim"])
+        p[mix + "uk"], p[mix + "uv"] = mat(H * m["dim"], R), mat(H * m["vdim"], R)
+        if "kv_from" not in m:
+            p[mix + "dkv"], p[mix + "dkv.norm"] = mat(R, W), (1 + 0.02 * rnd(R)).to(dtype)
+        if f is None:
+            continue
+        norm(f"l{i}.norm2")
+        if f["kind"] == "dense":
+            feed_forward(f"l{i}.mlp", f["ff"])
+            continue
+        p[f"l{i}.mlp.router"], p[f"l{i}.mlp.router.b"] = mat(f["router"]["experts"], W), rnd(f["router"]["experts"]).to(dtype)
+        for e in range(f["router"]["experts"]):
+            feed_forward(f"l{i}.mlp.e{e}", f["expert"]["ff"])
+        if f.get("shared"):
+            feed_forward(f"l{i}.mlp.shared", f["shared"]["ff"])
+    return p
+
+
 def adapter_ids_uniform(n_requests: int, n_adapters: int) -> np.ndarray:
     return np.random.default_rng(SEED_IDS).integers(0, n_adapters, n_requests).astype(np.int32)
 

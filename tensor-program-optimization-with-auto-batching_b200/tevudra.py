@@ -198,6 +198,8 @@ class PackedTevudra:
 class TevudraEngine(EngineBase):
     # a prompt pass expands keys and values of at most this many context rows; beyond, its rows attend in latent space
     MAX_EXPANDED_ROWS = 1 << 18
+    # cost of an operation in latent space (row by row) against one of the tiled prompt attention
+    LATENT_COST = 3.0
 
     def __init__(self, model: PackedTevudra, kv: PagedLatentCache, max_rows: int):
         super().__init__(model, kv, max_rows)
@@ -230,7 +232,8 @@ class TevudraEngine(EngineBase):
                 shapes += [(m.H, lw.ffp), (lw.ffp, m.H)]
             elif lw.ff is not None:
                 shapes += [(m.H, lw.ff.experts)] + ([(m.H, lw.sffp), (lw.sffp, m.H)] if lw.ff.shared_ff else [])
-        need = max([lib.mlora_linear_workspace(T, k, n) for k, n in shapes] + [lib.mlora_grouped_linear_workspace(64)])
+        # (the expansion of a context may have more rows than the pass: scratch no longer grows beyond 128)
+        need = max([lib.mlora_linear_workspace(max(T, 128), k, n) for k, n in shapes] + [lib.mlora_grouped_linear_workspace(64)])
         self.ws_linear = ops.new_workspace(need, dev)
         self.status = torch.zeros(1, dtype=torch.int32, device=dev)
         # prompt passes: query tiles of <= 128 rows, context segments (whole pages) of the expanded keys and values
@@ -264,7 +267,7 @@ class TevudraEngine(EngineBase):
             R, d = lw.mix.rank, lw.dk + lw.dv
             latent += lw.mix.heads * 4 * R * pairs
             expanded += lw.mix.heads * (2 * d * pairs + 2 * R * d * sum(ctx))
-        if latent < expanded:
+        if latent * self.LATENT_COST < expanded:
             return
         tiles, segs, base = [], [], 0
         for (sid, r0, n, p0), c in zip(chunk, ctx):
