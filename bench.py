@@ -1067,7 +1067,7 @@ class KernelTimer:
     """Times every operator call of an engine pass by itself: L2 flushed (a 256 MB write), CUDA events around the call on
     the launching stream.  Calls of one operator and shape are averaged; the best of the passes counts."""
 
-    NAMES = ("linear", "grouped_linear", "moe_plan", "residual_dyt", "residual_rmsnorm", "latent_append", "latent_gather",
+    NAMES = ("linear", "grouped_linear", "moe_plan", "moe_route_plan", "residual_dyt", "residual_rmsnorm", "latent_append", "latent_gather",
              "latent_attention", "prefill_attention_dense", "embed", "argmax", "paged_attention", "prefill_attention",
              "kv_append_rope")
 
@@ -1116,6 +1116,8 @@ class KernelTimer:
             return f"{a[0].shape[0]} rows", 4 * a[0].numel(), 0.0
         if name == "moe_plan":
             return f"{a[3]} tokens", 4 * a[3] * (a[2].E + 4 * a[2].top), 0.0
+        if name == "moe_route_plan":
+            return f"{a[0].shape[0]} tokens", 2 * a[1].numel() + 2 * a[0].numel(), 2.0 * a[0].shape[0] * a[1].numel()
         if name == "embed":
             return f"{a[0].numel()} rows", a[0].numel() * a[1].shape[1] * 6, 0.0
         return f"{a[0].shape[0]} rows", 4 * a[0].numel(), 0.0
@@ -1246,7 +1248,7 @@ def run_tevudra(args):
                 def step():
                     for s in sids:
                         kv._len_host[kv.slot(s)] = n_ctx - 1
-                    eng.decode(sids, [1] * B, slots)
+                    eng.decode(sids, [7 * s + 1 for s in sids], slots)
                 line["kernels"][f"decode {B} at {ctx}"] = timer.run(step, [n_ctx] * B, [1] * B)
                 del g, eng, kv
                 torch.cuda.empty_cache()

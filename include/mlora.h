@@ -462,8 +462,15 @@ int mlora_linear_f32(const float* d_x, int64_t ldx, int32_t x_cols, const int32_
  * and the softmax over exactly those; then the T * top (token, expert) pairs grouped by expert, in token order inside one.
  *   d_expert, d_weight [T, top]; d_pos [T, top]: row of the pair in expert order; d_rows [T * top]: token of a row;
  *   d_tiles: the table of mlora_grouped_linear for tiles of tile_rows rows, room for 1 + T * top / tile_rows + min(E, T * top)
- *   entries of 16 bytes.  E <= 1024.  d_work: mlora_moe_plan_workspace(T, E, top) bytes (0 for decode sizes, one launch). */
+ *   entries of 16 bytes.  E <= 1024.  d_work: mlora_moe_plan_workspace(T, E, top) bytes, zero-filled once (a ticket that
+ *   resets itself).
+ * mlora_moe_route_plan: the router as well (logits = W h, W [E, in] row-major, fp32 sums; h and W bf16, or fp32 with f32 != 0)
+ *   and all of the plan in one launch, for the sizes of decode steps (mlora_moe_decode_fits). */
 size_t mlora_moe_plan_workspace(int32_t T, int32_t E, int32_t top);
+uint32_t mlora_moe_decode_fits(int32_t T, int32_t top);
+int mlora_moe_route_plan(const void* d_h, int64_t ldh, const void* d_W, int32_t in, const float* d_bias, int32_t T, int32_t E,
+                         int32_t top, int32_t tile_rows, int32_t* d_expert, float* d_weight, int32_t* d_pos, int32_t* d_rows,
+                         int32_t* d_tiles, void* d_work, size_t work_bytes, int32_t f32, void* stream);
 int mlora_moe_plan(const float* d_logits, int64_t ld, const float* d_bias, int32_t T, int32_t E, int32_t top, int32_t tile_rows,
                    int32_t* d_expert, float* d_weight, int32_t* d_pos, int32_t* d_rows, int32_t* d_tiles, void* d_work,
                    size_t work_bytes, void* stream);

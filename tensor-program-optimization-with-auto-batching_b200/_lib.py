@@ -78,6 +78,9 @@ PROTOTYPES = {
     "mlora_linear_f32": (C.c_int, [_vp, _i64, _i32, _vp, _vp, _vp, _i64, _i32, _vp, _i32, _i32, _i32, _i32, _i32,
                                    _i32, _vp, _i64, _vp]),
     "mlora_moe_plan_workspace": (_sz, [_i32, _i32, _i32]),
+    "mlora_moe_decode_fits": (C.c_uint32, [_i32, _i32]),
+    "mlora_moe_route_plan": (C.c_int, [_vp, _i64, _vp, _i32, _vp, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _sz,
+                                       _i32, _vp]),
     "mlora_moe_plan": (C.c_int, [_vp, _i64, _vp, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
     "mlora_residual_dyt": (C.c_int, [_vp, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _vp]),
     "mlora_latent_append": (C.c_int, [_vp, _i64, _i32, _vp, _f32, _vp, _i32, _i32, _vp, _i32, _vp, _vp, _i32, _i32,

@@ -28,6 +28,13 @@ int launch_grouped(const GroupedArgs& ga, void* work, cudaStream_t st) {
   p.g.ld_gate = ga.ld_gate;
   p.tok_tiles = ga.table ? 0 : ga.n_groups * p.g.tiles_per_group;
   p.n_tiles = p.row_tiles * p.tok_tiles;
+  // whole output chunks by TMA when y allows it (a ragged chunk never goes that way, so the map needs no row count)
+  CUtensorMap my = mx;
+  p.tma_store = !(a.flags & MLORA_OUT_F32) && aligned16(a.y) && a.ldy % 8 == 0 && ga.y_cols % 8 == 0 && a.out % 8 == 0;
+  if (p.tma_store) {
+    rc = make_out_map(&my, a.y, 1 << 30, (int)a.ldy, a.ldy, C::kChunk, BM, false);
+    if (rc) return rc;
+  }
   p.lora_sub = 16;
   p.n_sub = 1;
   p.status = (int32_t*)work;
@@ -41,7 +48,7 @@ int launch_grouped(const GroupedArgs& ga, void* work, cudaStream_t st) {
     if (e != cudaSuccess) return fail(MLORA_ECUDA, "grouped_linear: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
     attr_done.fetch_or(1ull << (dev & 63), std::memory_order_release);
   }
-  launch_pdl_if(pdl_enabled_gemm(), linear_tc_kernel<BN, 0, false, true>, sm_count(), kThreads, C::kSmemBytes, st, mx, mx, mx, mx, p);
+  launch_pdl_if(pdl_enabled_gemm(), linear_tc_kernel<BN, 0, false, true>, sm_count(), kThreads, C::kSmemBytes, st, mx, mx, mx, my, p);
   count_launch();
   MLORA_CHECK_LAUNCH("linear_tc_kernel (grouped)");
   return MLORA_OK;

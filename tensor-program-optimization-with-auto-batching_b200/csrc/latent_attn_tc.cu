@@ -2,16 +2,18 @@
 // prompt) against the paged latents, for up to 32 heads of the row in one CTA -- the latents of a key are read once for all
 // of them, as key and as value.
 //
-// CTA = (row, split of its keys, group of HG heads).  Keys are the M dimension, heads the N dimension:
-//   S^T [128 keys x HG]          = C [128 x R] . Qa^T [R x HG]      A = the latents as the pages hold them, K-major
-//   O^T [R x HG] (128 at a time) += C^T [R x 128] . P^T [128 x HG]  A = the same shared memory, now MN-major: the rank is
-//                                                                    the contiguous dimension, no transpose is made
-// so a head count of 32 wastes nothing, and both products read one copy of C.  Roles: warp 0 brings pages by TMA into a
-// ring of slots of 128 keys x 128 latent columns, warp 1 issues the MMAs, warps 2..5 (one thread per key = TMEM lane) do
-// the softmax in fp32.  The running maximum of a head is moved only when a block exceeds it by more than 2^8, and only then
-// are the sums in TMEM rescaled; the row sums stay per thread until the end.  A slot is refilled as soon as the O^T
-// product of its 128 columns has retired, so the ring keeps streaming across blocks.
+// CTA = (row, split of its keys, group of HG heads), 64 keys per block:
+//   S [heads x 64]          = Qa [heads x R] . C^T            A = the queries, in TMEM (lane = head), B = the latents as the
+//                                                             pages hold them, K-major
+//   O^T [R x HG] (by 128)  += C^T [R x 64] . P^T [64 x HG]    A = the same shared memory, now MN-major (the rank is the
+//                                                             contiguous dimension: no transpose is made), B = P
+// so both products read one copy of C, and a head is a TMEM lane for the softmax: one thread per head walks its 64 scores,
+// no value crosses lanes.  The scores and the probabilities are double buffered: the scores of block b + 1 are computed
+// while the softmax of block b runs, and the ring of 16 KB slots (64 keys x 128 latent columns) keeps streaming.  The
+// running maximum of a head is moved only when a block exceeds it by more than 2^8; only then do all four output warps
+// rescale the sums in TMEM, on request.
 //
+// Roles: warp 0 TMA, warp 1 MMA issue, warp 4 (TMEM lanes 0..31) softmax, warps 2..5 rescaling and output.
 // With several splits a CTA leaves unnormalised fp32 sums, its maxima and row sums, and a small kernel joins them.
 // Every wait is bounded; a CTA that gives up sets the status word and leaves its outputs undefined.
 #include <math.h>
@@ -24,11 +26,13 @@
 namespace mlora {
 namespace {
 
-constexpr int kKeys = 128;                     // keys per block
-constexpr int kSubTile = kKeys * 128;          // [128 keys][64 columns] bf16
+constexpr int kKeys = 64;                      // keys per block
+constexpr int kSubTile = kKeys * 128;          // [64 keys][64 columns] bf16
 constexpr int kSlot = 2 * kSubTile;            // 128 columns
+constexpr int kMaxSlots = 13;
 constexpr int kLtThreads = 192;
 constexpr int kMaxChunks = 4;                  // kv_rank up to 512
+constexpr int kTmemCols = 512;                 // S: 2 x 64, O^T: 4 x 32, queries: 256
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kRescale = 8.f;                // (log2) how far scores may exceed the reference maximum
 
@@ -36,7 +40,8 @@ struct LtArgs {
   const int32_t* block_table;
   int max_pages, page_size, n_page_rows;       // n_page_rows: rows of the page tensor (the first row that does not exist)
   const int32_t *row_slot, *row_pos;
-  int H, R, q_pitch, n_chunks, n_slots, n_splits;
+  const bf16* qa;                              // [T, H, q_pitch]
+  int H, q_pitch, n_chunks, n_slots, n_splits;
   float scale_log2;
   bf16* out;                                   // [T, H, q_pitch]
   float* part;                                 // [T, H, n_splits, q_pitch] unnormalised sums
@@ -58,6 +63,16 @@ __device__ __forceinline__ uint64_t desc_mn(uint32_t saddr, uint32_t lbo, uint32
   d |= (uint64_t)1 << 46;
   d |= (uint64_t)2 << 61;
   return d;
+}
+
+// D [128 x N] (+)= A [128 x 16] . B^T with A in TMEM: two bf16 of the K dimension per 32-bit column.
+__device__ __forceinline__ void umma_bf16_ta(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t acc) {
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+      ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(acc)
+      : "memory");
 }
 
 template <int N>
@@ -86,37 +101,15 @@ __device__ __forceinline__ void tmem_st(uint32_t addr, const float (&v)[32]) {
   asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
 }
 
-// Reduces N values per lane over the warp's lanes: afterwards lane l holds in v[0] the result of value l % N.
-template <int N, typename F>
-__device__ __forceinline__ void reduce_scatter(float (&v)[32], F f) {
-  const int lane = threadIdx.x & 31;
-  if constexpr (N == 16) {
-#pragma unroll
-    for (int i = 0; i < 16; ++i) v[i] = f(v[i], __shfl_xor_sync(0xffffffffu, v[i], 16));
-  }
-#pragma unroll
-  for (int off = N / 2; off >= 1; off >>= 1) {
-    const bool up = (lane & off) != 0;
-#pragma unroll
-    for (int j = 0; j < off; ++j) {
-      const float send = up ? v[j] : v[j + off], keep = up ? v[j + off] : v[j];
-      v[j] = f(keep, __shfl_xor_sync(0xffffffffu, send, off));
-    }
-  }
-}
-
 template <int HG>
-__global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q,
-                                                                       const __grid_constant__ CUtensorMap map_c, LtArgs a) {
+__global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __grid_constant__ CUtensorMap map_c, LtArgs a) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-  uint8_t* sq = ring + a.n_slots * kSlot;               // queries: sub-tiles [HG][64 columns]
-  uint8_t* sp = sq + 2 * a.n_chunks * HG * 128;         // probabilities: sub-tiles [HG][64 keys]
-  __shared__ uint64_t full_bar[8], empty_bar[8], q_bar, s_bar, p_bar, o_bar;
+  uint8_t* sp = ring + a.n_slots * kSlot;               // probabilities: two buffers [HG][64 keys]
+  __shared__ uint64_t full_bar[kMaxSlots], empty_bar[kMaxSlots], q_bar, s_bar[2], p_bar[2], o_bar[2], cmd_bar, ack_bar;
   __shared__ uint32_t tmem_slot;
-  __shared__ int s_abort, s_changed;
-  __shared__ float s_red[4][HG];
-  __shared__ __align__(16) float s_m[HG], s_f[HG];
+  __shared__ int s_abort, s_end;
+  __shared__ __align__(16) float s_f[32];
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int t = blockIdx.x, split = blockIdx.y, head0 = blockIdx.z * HG;
@@ -125,10 +118,10 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __g
   pdl_wait();
   const int n_keys = min(a.row_pos[t] + 1, a.max_pages * a.page_size);
   const int blocks = (n_keys + kKeys - 1) / kKeys, per = (blocks + a.n_splits - 1) / a.n_splits;
-  const int b0 = min(split * per, blocks), b1 = min(b0 + per, blocks);
+  const int b0 = min(split * per, blocks), nb = min(b0 + per, blocks) - b0;
   const size_t out_row = (size_t)t * a.H + head0;
 
-  if (b0 >= b1) {  // no keys for this CTA (a padding row, or more splits than blocks)
+  if (nb <= 0) {  // no keys for this CTA (a padding row, or more splits than blocks)
     if (a.n_splits == 1) {
       for (int i = tid; i < heads * a.q_pitch; i += kLtThreads) a.out[out_row * a.q_pitch + i] = __float2bfloat16_rn(0.f);
     } else if (tid < heads) {
@@ -138,196 +131,241 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __g
   }
 
   if (tid == 0) {
-    s_abort = 0;
+    s_abort = s_end = 0;
     for (int i = 0; i < a.n_slots; ++i) {
       mbar_init(&full_bar[i], 1);
       mbar_init(&empty_bar[i], 1);
     }
-    mbar_init(&q_bar, 1);
-    mbar_init(&s_bar, 1);
-    mbar_init(&p_bar, 128);
-    mbar_init(&o_bar, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&s_bar[i], 1);
+      mbar_init(&p_bar[i], 32);
+      mbar_init(&o_bar[i], 1);
+    }
+    mbar_init(&q_bar, 32);
+    mbar_init(&cmd_bar, 32);
+    mbar_init(&ack_bar, 128);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-    tma_prefetch_desc(&map_q);
     tma_prefetch_desc(&map_c);
   }
-  if (tid < HG) s_m[tid] = -INFINITY;
-  if (warp == 1) tmem_alloc(&tmem_slot, 256);
+  if (warp == 1) tmem_alloc(&tmem_slot, kTmemCols);
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem_s = tmem_slot, tmem_o = tmem_s + 32;  // S^T: HG columns; O^T: HG columns per 128 of the rank
+  const uint32_t tmem_s = tmem_slot, tmem_o = tmem_s + 128, tmem_q = tmem_s + 256;
 
   if (warp == 0) {
     // ---- producer ------------------------------------------------------------------------------------------------
-    if (lane == 0) mbar_expect_tx(&q_bar, 2 * a.n_chunks * HG * 128);
-    __syncwarp();
-    if (lane < 2 * a.n_chunks) tma_load_2d(sq + lane * HG * 128, &map_q, lane * 64, (int)out_row, &q_bar);
     const int32_t* bt = a.block_table + (size_t)a.row_slot[t] * a.max_pages;
     const int ppb = kKeys / a.page_size, half = lane & 1, p = lane >> 1;  // one (page, column half) per lane
     const int n_pages = (n_keys + a.page_size - 1) / a.page_size;
     auto row_of = [&](int b) {  // rows past the last page read as zeros
-      const int pg = b * ppb + p;
+      const int pg = (b0 + b) * ppb + p;
       return p < ppb && pg < n_pages ? bt[pg] * a.page_size : a.n_page_rows;
     };
-    int n = 0, next = row_of(b0);
+    int s = 0, next = row_of(0), next2 = nb > 1 ? row_of(1) : 0;
+    uint32_t par = 1;
     bool ok = true;
-    for (int b = b0; b < b1 && ok; ++b) {
+    for (int b = 0; b < nb && ok; ++b) {
       const int row = next;
-      if (b + 1 < b1) next = row_of(b + 1);
-      for (int j = 0; j < a.n_chunks; ++j, ++n) {
-        const int s = n % a.n_slots;
+      next = next2;
+      if (b + 2 < nb) next2 = row_of(b + 2);
+      for (int j = 0; j < a.n_chunks; ++j) {
         if (lane == 0) {
-          ok = mbar_wait(&empty_bar[s], ((n / a.n_slots) & 1) ^ 1, &s_abort);
+          ok = mbar_wait(&empty_bar[s], par, &s_abort);
           if (ok) mbar_expect_tx(&full_bar[s], kSlot);
         }
         ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
         if (!ok) break;
         if (p < ppb)
           tma_load_2d(ring + s * kSlot + half * kSubTile + p * a.page_size * 128, &map_c, j * 128 + half * 64, row, &full_bar[s]);
+        if (++s == a.n_slots) s = 0, par ^= 1;
       }
     }
     if (!ok) s_abort = 1;
   } else if (warp == 1) {
     // ---- MMA issue -----------------------------------------------------------------------------------------------
     if (lane == 0) {
-      constexpr uint32_t idesc_s = make_idesc(128, HG), idesc_o = make_idesc(128, HG) | (1u << 15);  // O^T: A is MN-major
+      constexpr uint32_t idesc_s = make_idesc(128, kKeys), idesc_o = make_idesc(128, HG) | (1u << 15);  // O^T: A is MN-major
       bool ok = mbar_wait(&q_bar, 0, &s_abort);
-      int n = 0;
-      for (int b = b0; b < b1 && ok; ++b) {
-        const uint32_t par = (b - b0) & 1;
-        for (int j = 0; j < a.n_chunks && ok; ++j) {
-          const int s = (n + j) % a.n_slots;
-          ok = mbar_wait(&full_bar[s], ((n + j) / a.n_slots) & 1, &s_abort);
-          if (!ok) break;
+      tc_fence_after();
+      int s_s = 0, s_o = 0;  // ring positions of the two products
+      uint32_t par = 0;
+      auto scores = [&](int b) {
+        for (int j = 0; j < a.n_chunks; ++j) {
+          if (!mbar_wait(&full_bar[s_s], par, &s_abort)) return false;
           tc_fence_after();
 #pragma unroll
           for (int h = 0; h < 2; ++h) {
-            const uint64_t ad = make_smem_desc(smem_u32(ring + s * kSlot + h * kSubTile));
-            const uint64_t bd = make_smem_desc(smem_u32(sq + (2 * j + h) * HG * 128));
+            const uint64_t bd = make_smem_desc(smem_u32(ring + s_s * kSlot + h * kSubTile));
 #pragma unroll
-            for (int k = 0; k < 4; ++k) umma_bf16(tmem_s, ad + 2 * k, bd + 2 * k, idesc_s, (j | h | k) ? 1u : 0u);
+            for (int k = 0; k < 4; ++k)
+              umma_bf16_ta(tmem_s + (b & 1) * kKeys, tmem_q + j * 64 + h * 32 + k * 8, bd + 2 * k, idesc_s, (j | h | k) ? 1u : 0u);
           }
+          if (++s_s == a.n_slots) s_s = 0, par ^= 1;
         }
-        if (!ok) break;
-        umma_commit(&s_bar);
-        ok = mbar_wait(&p_bar, par, &s_abort);
+        umma_commit(&s_bar[b & 1]);
+        return true;
+      };
+      ok = ok && scores(0);
+      for (int b = 0; b < nb && ok; ++b) {
+        if (b + 1 < nb) ok = scores(b + 1);  // (the softmax has read the scores of block b - 1: its probabilities came)
+        ok = ok && mbar_wait(&p_bar[b & 1], (b >> 1) & 1, &s_abort);
         if (!ok) break;
         tc_fence_after();
         for (int j = 0; j < a.n_chunks; ++j) {
-          const int s = (n + j) % a.n_slots;
-          const uint32_t c = smem_u32(ring + s * kSlot);
+          const uint32_t c = smem_u32(ring + s_o * kSlot);
 #pragma unroll
-          for (int k = 0; k < 8; ++k)  // 16 keys = 2048 bytes of a sub-tile
-            umma_bf16(tmem_o + j * HG, desc_mn(c + k * 2048, kSubTile, 1024),
-                      make_smem_desc(smem_u32(sp + (k >> 2) * HG * 128)) + 2 * (k & 3), idesc_o, (b > b0 || k > 0) ? 1u : 0u);
-          umma_commit(&empty_bar[s]);
+          for (int k = 0; k < 4; ++k)  // 16 keys = 2048 bytes of a sub-tile
+            umma_bf16(tmem_o + j * 32, desc_mn(c + k * 2048, kSubTile, 1024),
+                      make_smem_desc(smem_u32(sp + (b & 1) * HG * 128)) + 2 * k, idesc_o, (b | k) ? 1u : 0u);
+          umma_commit(&empty_bar[s_o]);
+          if (++s_o == a.n_slots) s_o = 0;
         }
-        n += a.n_chunks;
+        umma_commit(&o_bar[b & 1]);
       }
       if (!ok) s_abort = 1;
-      umma_commit(&o_bar);
     }
     __syncwarp();
   } else {
-    // ---- softmax: thread = key of the block ------------------------------------------------------------------------
-    const int q = warp & 3, kl = q * 32 + lane;
+    const int q = warp & 3;
     const uint32_t lane_base = (uint32_t)(q * 32) << 16;
-    float lp[HG];
-#pragma unroll
-    for (int i = 0; i < HG; ++i) lp[i] = 0.f;
     bool ok = true;
-    for (int b = b0; b < b1; ++b) {
-      ok = mbar_wait(&s_bar, (b - b0) & 1, &s_abort);  // every MMA issued before has retired as well: sp and O^T are free
-      if (!ok) s_abort = 1;
-      tc_fence_after();
-      const bool valid = b * kKeys + kl < n_keys;
-      float s[32], mx[32];
-      tmem_ld<HG>(tmem_s + lane_base, s);
+    auto rescale = [&]() {  // this warp's quarter of O^T, every head by its factor
+      for (int j = 0; j < a.n_chunks; ++j) {
+        float o[32];
+        tmem_ld<HG>(tmem_o + j * 32 + lane_base, o);
 #pragma unroll
-      for (int i = 0; i < HG; ++i) {
-        s[i] = valid ? s[i] * a.scale_log2 : -INFINITY;
-        mx[i] = s[i];
-      }
-      reduce_scatter<HG>(mx, [](float x, float y) { return fmaxf(x, y); });
-      if (lane < HG) s_red[q][lane] = mx[0];
-      if (kl == 0) s_changed = 0;
-      epi_bar_sync();
-      if (kl < HG) {
-        const float bm = fmaxf(fmaxf(s_red[0][kl], s_red[1][kl]), fmaxf(s_red[2][kl], s_red[3][kl]));
-        const float old = s_m[kl];
-        float f = 1.f;
-        if (bm > old + kRescale || old == -INFINITY) {
-          f = ex2(old - bm);  // (0 at the first block)
-          if (bm == -INFINITY) f = 1.f;  // (every score -inf: nothing to scale)
-          else s_m[kl] = bm;
-          s_changed = 1;
-        }
-        s_f[kl] = f;
-      }
-      epi_bar_sync();
-      if (s_changed && b > b0) {
-#pragma unroll
-        for (int i = 0; i < HG; ++i) lp[i] *= s_f[i];
-        for (int j = 0; j < a.n_chunks; ++j) {
-          float o[32];
-          tmem_ld<HG>(tmem_o + j * HG + lane_base, o);
-#pragma unroll
-          for (int i = 0; i < HG; ++i) o[i] *= s_f[i];
-          tmem_st<HG>(tmem_o + j * HG + lane_base, o);
-        }
-      }
-      uint8_t* pd = sp + (kl >> 6) * HG * 128 + (kl & 7) * 2;
-      const int cx = (kl & 63) >> 3;
-#pragma unroll
-      for (int i = 0; i < HG; ++i) {
-        const float m = s_m[i];
-        const float pr = valid ? ex2(s[i] - (m == -INFINITY ? 0.f : m)) : 0.f;
-        lp[i] += pr;
-        *reinterpret_cast<bf16*>(pd + i * 128 + ((cx ^ (i & 7)) << 4)) = __float2bfloat16_rn(pr);
-      }
-      if (!valid) {
-        // latents of keys that do not exist (whatever the last page holds there): their probability is 0, but 0 * NaN is not
-        for (int j = 0; j < a.n_chunks; ++j) {
-          uint8_t* c = ring + (((b - b0) * a.n_chunks + j) % a.n_slots) * kSlot + kl * 128;
-#pragma unroll
-          for (int i = 0; i < 8; ++i) {
-            reinterpret_cast<uint4*>(c)[i] = make_uint4(0u, 0u, 0u, 0u);
-            reinterpret_cast<uint4*>(c + kSubTile)[i] = make_uint4(0u, 0u, 0u, 0u);
-          }
-        }
+        for (int i = 0; i < HG; ++i) o[i] *= s_f[i];
+        tmem_st<HG>(tmem_o + j * 32 + lane_base, o);
       }
       tc_fence_before();
-      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-      mbar_arrive(&p_bar);
+    };
+    uint32_t n_cmd = 0;
+    if (q == 0) {
+      // ---- softmax: thread = head ------------------------------------------------------------------------------------
+      const bool live = lane < heads;
+      {
+        // queries -> TMEM, 32 columns (64 values) at a time
+        const uint4* src = reinterpret_cast<const uint4*>(a.qa + (out_row + (live ? lane : 0)) * a.q_pitch);
+        for (int c = 0; c < 2 * a.n_chunks; ++c) {
+          uint4 w[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) w[i] = live ? __ldg(src + c * 8 + i) : make_uint4(0u, 0u, 0u, 0u);
+          tmem_st<32>(tmem_q + c * 32, *reinterpret_cast<const float(*)[32]>(w));
+        }
+        tc_fence_before();
+        mbar_arrive(&q_bar);
+      }
+      float m = -INFINITY, l = 0.f;
+      for (int b = 0; b < nb; ++b) {
+        if (!mbar_wait(&s_bar[b & 1], (b >> 1) & 1, &s_abort)) s_abort = 1;
+        tc_fence_after();
+        float s0[32], s1[32];
+        tmem_ld32(tmem_s + (b & 1) * kKeys, s0);
+        tmem_ld32(tmem_s + (b & 1) * kKeys + 32, s1);
+        const int valid = n_keys - (b0 + b) * kKeys;  // keys of this block that exist (>= 64: all)
+        float mx0 = -INFINITY, mx1 = -INFINITY;
+        if (valid >= kKeys) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            s0[i] *= a.scale_log2, s1[i] *= a.scale_log2;
+            mx0 = fmaxf(mx0, s0[i]), mx1 = fmaxf(mx1, s1[i]);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            s0[i] = i < valid ? s0[i] * a.scale_log2 : -INFINITY, s1[i] = i + 32 < valid ? s1[i] * a.scale_log2 : -INFINITY;
+            mx0 = fmaxf(mx0, s0[i]), mx1 = fmaxf(mx1, s1[i]);
+          }
+        }
+        const float mx = fmaxf(mx0, mx1);
+        float f = 1.f;
+        if (live && mx > -INFINITY && (m == -INFINITY || mx > m + kRescale)) {
+          f = ex2(m - mx);  // (0 while nothing has been seen)
+          m = mx;
+          l *= f;
+        }
+        if (b > 0 && __any_sync(0xffffffffu, f != 1.f)) {
+          // every product issued so far must have retired before the sums are touched
+          if (!mbar_wait(&o_bar[(b - 1) & 1], ((b - 1) >> 1) & 1, &s_abort)) s_abort = 1;
+          tc_fence_after();
+          s_f[lane] = f;
+          __syncwarp();
+          mbar_arrive(&cmd_bar);
+          rescale();
+          mbar_arrive(&ack_bar);
+          if (!mbar_wait(&ack_bar, n_cmd & 1, &s_abort)) s_abort = 1;
+          ++n_cmd;
+        }
+        const float base = m == -INFINITY ? 0.f : m;
+        float l0 = 0.f, l1 = 0.f;
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          s0[i] = ex2(s0[i] - base), s1[i] = ex2(s1[i] - base);
+          l0 += s0[i], l1 += s1[i];
+        }
+        l += l0 + l1;
+        // the product of block b - 2 has read this buffer
+        if (b >= 2 && !mbar_wait(&o_bar[b & 1], ((b >> 1) & 1) ^ 1, &s_abort)) s_abort = 1;
+        if (lane < HG) {
+          uint8_t* pr = sp + (b & 1) * HG * 128 + lane * 128;
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const float f0[8] = {s0[8 * c], s0[8 * c + 1], s0[8 * c + 2], s0[8 * c + 3], s0[8 * c + 4], s0[8 * c + 5], s0[8 * c + 6], s0[8 * c + 7]};
+            const float f1[8] = {s1[8 * c], s1[8 * c + 1], s1[8 * c + 2], s1[8 * c + 3], s1[8 * c + 4], s1[8 * c + 5], s1[8 * c + 6], s1[8 * c + 7]};
+            *reinterpret_cast<uint4*>(pr + ((c ^ (lane & 7)) << 4)) = pack8(f0);
+            *reinterpret_cast<uint4*>(pr + (((c + 4) ^ (lane & 7)) << 4)) = pack8(f1);
+          }
+        }
+        if (valid < kKeys) {
+          // latents of keys that do not exist (whatever the last page holds there): their probability is 0, but 0 * NaN is
+          // not.  The scores of this block have been computed, so all its slots have landed.
+          for (int j = 0; j < a.n_chunks; ++j) {
+            uint8_t* c = ring + ((b * a.n_chunks + j) % a.n_slots) * kSlot;
+            for (int i = valid * 8 + lane; i < kKeys * 8; i += 32) {
+              reinterpret_cast<uint4*>(c)[i] = make_uint4(0u, 0u, 0u, 0u);
+              reinterpret_cast<uint4*>(c + kSubTile)[i] = make_uint4(0u, 0u, 0u, 0u);
+            }
+          }
+        }
+        tc_fence_before();
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+        mbar_arrive(&p_bar[b & 1]);
+      }
+      if (!mbar_wait(&o_bar[(nb - 1) & 1], ((nb - 1) >> 1) & 1, &s_abort)) s_abort = 1;
+      s_f[lane] = a.n_splits == 1 ? (l > 0.f ? 1.f / l : 0.f) : 1.f;
+      if (a.n_splits > 1 && live) a.ml[(out_row + lane) * a.n_splits + split] = make_float2(m, l);
+      if (lane == 0) s_end = 1;
+      __syncwarp();
+      mbar_arrive(&cmd_bar);
+    } else {
+      // ---- the other output warps: rescale on request, until the sums are complete -------------------------------------
+      while (true) {
+        ok = mbar_wait(&cmd_bar, n_cmd & 1, &s_abort);
+        if (!ok || *(volatile int*)&s_end) break;
+        tc_fence_after();
+        rescale();
+        mbar_arrive(&ack_bar);
+        if (!mbar_wait(&ack_bar, n_cmd & 1, &s_abort)) break;  // nobody is a request ahead of the others
+        ++n_cmd;
+      }
+      if (!ok) s_abort = 1;
     }
-    if (!mbar_wait(&o_bar, 0, &s_abort)) s_abort = 1;
     tc_fence_after();
-    // row sums over the 128 threads, head by head
-    float sum[32];
+    if (!*(volatile int*)&s_abort) {
+      for (int j = 0; j < a.n_chunks; ++j) {
+        float o[32];
+        tmem_ld<HG>(tmem_o + j * 32 + lane_base, o);
+        const int r = j * 128 + q * 32 + lane;
 #pragma unroll
-    for (int i = 0; i < HG; ++i) sum[i] = lp[i];
-    reduce_scatter<HG>(sum, [](float x, float y) { return x + y; });
-    if (lane < HG) s_red[q][lane] = sum[0];
-    epi_bar_sync();
-    if (kl < HG) {
-      const float l = (s_red[0][kl] + s_red[1][kl]) + (s_red[2][kl] + s_red[3][kl]);
-      s_f[kl] = a.n_splits == 1 ? (l > 0.f ? 1.f / l : 0.f) : 1.f;
-      if (a.n_splits > 1 && kl < heads) a.ml[(out_row + kl) * a.n_splits + split] = make_float2(s_m[kl], l);
-    }
-    epi_bar_sync();
-    for (int j = 0; j < a.n_chunks; ++j) {
-      float o[32];
-      tmem_ld<HG>(tmem_o + j * HG + lane_base, o);
-      const int r = j * 128 + kl;
-#pragma unroll
-      for (int i = 0; i < HG; ++i) {
-        if (i < heads) {
-          const size_t row = out_row + i;
-          if (a.n_splits == 1)
-            a.out[row * a.q_pitch + r] = __float2bfloat16_rn(o[i] * s_f[i]);
-          else
-            a.part[(row * a.n_splits + split) * a.q_pitch + r] = o[i];
+        for (int i = 0; i < HG; ++i) {
+          if (i < heads) {
+            const size_t row = out_row + i;
+            if (a.n_splits == 1)
+              a.out[row * a.q_pitch + r] = __float2bfloat16_rn(o[i] * s_f[i]);
+            else
+              a.part[(row * a.n_splits + split) * a.q_pitch + r] = o[i];
+          }
         }
       }
     }
@@ -338,7 +376,7 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __g
     if (tid == 0 && a.status) atomicOr(a.status, 1);
     for (int i = 0; i < 64; ++i) __nanosleep(1000);  // copies still in flight land before the CTA's shared memory goes
   }
-  if (warp == 1) tmem_dealloc(tmem_s, 256);
+  if (warp == 1) tmem_dealloc(tmem_s, kTmemCols);
 }
 
 // Joins the splits of one (row, head): weights 2^(m_s - max m), then one division.
@@ -372,8 +410,8 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
 
 int head_group(int H) { return H <= 16 ? 16 : 32; }
 
-// Splits of a row's keys: the count that finishes first when every CTA has an SM to itself, with about one block's time
-// of fixed cost per CTA.
+// Splits of a row's keys: the count that finishes first when every CTA has an SM to itself, with about three blocks'
+// time of fixed cost per CTA.
 int pick_splits(int T, int H, int max_keys) {
   int dev = 0, sms = 148;
   if (cudaGetDevice(&dev) == cudaSuccess) cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
@@ -383,15 +421,15 @@ int pick_splits(int T, int H, int max_keys) {
   double best_cost = 1e30;
   for (int s = 1; s <= 32 && s <= blocks; ++s) {
     const double waves = (double)((ctas * s + sms - 1) / sms);
-    const double cost = waves * ((blocks + s - 1) / s + 1.5) + (s > 1 ? 1.0 : 0.0);
+    const double cost = waves * ((blocks + s - 1) / s + 3.0) + (s > 1 ? 2.0 : 0.0);
     if (cost < best_cost - 1e-9) best_cost = cost, best = s;
   }
   return best;
 }
 
 template <int HG>
-int launch_lt(const CUtensorMap& mq, const CUtensorMap& mc, const LtArgs& a, int T, cudaStream_t st) {
-  const int smem = a.n_slots * kSlot + 2 * a.n_chunks * HG * 128 + 2 * HG * 128 + 1024;
+int launch_lt(const CUtensorMap& mc, const LtArgs& a, int T, cudaStream_t st) {
+  const int smem = a.n_slots * kSlot + 2 * HG * 128 + 1024;
   static std::atomic<unsigned long long> attr_done{0};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -400,7 +438,7 @@ int launch_lt(const CUtensorMap& mq, const CUtensorMap& mc, const LtArgs& a, int
     if (e != cudaSuccess) return fail(MLORA_ECUDA, "latent_attention: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
     attr_done.fetch_or(1ull << (dev & 63), std::memory_order_release);
   }
-  launch_pdl_if(pdl_enabled_attn(), latent_attn_tc_kernel<HG>, dim3(T, a.n_splits, (a.H + HG - 1) / HG), kLtThreads, smem, st, mq, mc, a);
+  launch_pdl_if(pdl_enabled_attn(), latent_attn_tc_kernel<HG>, dim3(T, a.n_splits, (a.H + HG - 1) / HG), kLtThreads, smem, st, mc, a);
   count_launch();
   MLORA_CHECK_LAUNCH("latent_attn_tc_kernel");
   return MLORA_OK;
@@ -438,10 +476,8 @@ extern "C" int mlora_latent_attention(const void* d_qa, int64_t q_pitch, const v
   MLORA_REQUIRE(!need || (d_work && aligned16(d_work) && work_bytes >= need), "latent_attention: workspace of %zu bytes needed, %zu given", need, work_bytes);
   if (T == 0) return MLORA_OK;
   const int HG = head_group(H);
-  CUtensorMap mq, mc;
-  int rc = make_map(&mq, d_qa, (long long)T * H, (int)q_pitch, q_pitch, HG, 64);
-  if (rc) return rc;
-  rc = make_map(&mc, d_pages, (long long)n_pages_total * page_size, pitch, pitch, page_size, 64);
+  CUtensorMap mc;
+  int rc = make_map(&mc, d_pages, (long long)n_pages_total * page_size, pitch, pitch, page_size, 64);
   if (rc) return rc;
   LtArgs a{};
   a.block_table = d_block_table;
@@ -450,21 +486,19 @@ extern "C" int mlora_latent_attention(const void* d_qa, int64_t q_pitch, const v
   a.n_page_rows = n_pages_total * page_size;
   a.row_slot = d_row_slot;
   a.row_pos = d_row_pos;
+  a.qa = (const bf16*)d_qa;
   a.H = H;
-  a.R = R;
   a.q_pitch = (int)q_pitch;
   a.n_chunks = n_chunks;
-  const int fixed = 2 * n_chunks * HG * 128 + 2 * HG * 128 + 1024;
-  a.n_slots = (224 * 1024 - fixed) / kSlot;
-  if (a.n_slots > 8) a.n_slots = 8;
-  if (a.n_slots > 2 * n_chunks) a.n_slots = 2 * n_chunks;
+  a.n_slots = (224 * 1024 - 2 * HG * 128 - 1024) / kSlot;
+  if (a.n_slots > kMaxSlots) a.n_slots = kMaxSlots;
   a.n_splits = n_splits;
   a.scale_log2 = scale * kLog2e;
   a.out = (bf16*)d_out;
   a.part = (float*)d_work;
   a.ml = (float2*)((float*)d_work + (size_t)T * H * n_splits * q_pitch);
   a.status = d_status;
-  rc = HG == 16 ? launch_lt<16>(mq, mc, a, T, (cudaStream_t)stream) : launch_lt<32>(mq, mc, a, T, (cudaStream_t)stream);
+  rc = HG == 16 ? launch_lt<16>(mc, a, T, (cudaStream_t)stream) : launch_lt<32>(mc, a, T, (cudaStream_t)stream);
   if (rc || n_splits == 1) return rc;
   launch_pdl(latent_merge_kernel, (unsigned)(T * H), 128, 0, (cudaStream_t)stream, a.part, a.ml, n_splits, (int)q_pitch, (bf16*)d_out);
   count_launch();

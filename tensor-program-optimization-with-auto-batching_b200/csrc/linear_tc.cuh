@@ -1160,18 +1160,41 @@ __global__ void __launch_bounds__(kThreads, 1) linear_tc_kernel(const __grid_con
           }
         }
         if constexpr (GRP) {
-          // per-thread stores: a warp writes 32 neighbouring features of one row, and a tile of one group must not touch
-          // the rows of the next
+          if (p.g.gate != nullptr) {  // one row's gate per lane, handed round
+            const int t = t0 + c0 + lane;
+            float gt = 0.f;
+            if (lane < C::kChunk && t < t_end)
+              gt = __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.g.gate[(size_t)t * p.g.ld_gate + group])));
+#pragma unroll
+            for (int i = 0; i < C::kChunk; ++i) v[i] *= __shfl_sync(0xffffffffu, gt, i);
+          }
+          if (p.tma_store) {
+            // as below, but a tile of one group must not touch the rows or columns of the next: only whole chunks leave by
+            // TMA, ragged ones row by row with 16-byte stores
+            if (etid == 0) bulk_wait_read0();
+            epi_bar_sync();
+            bf16* so = reinterpret_cast<bf16*>(s_out);
+#pragma unroll
+            for (int i = 0; i < C::kChunk; ++i) so[i * BM + etid] = __float2bfloat16_rn(v[i]);
+            if (t0 + c0 + C::kChunk <= t_end && row_tile * BM + BM <= a.out) {
+              asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+              epi_bar_sync();
+              if (etid == 0) tma_store_2d(&map_y, s_out, y_col + row_tile * BM, t0 + c0);
+              return;
+            }
+            epi_bar_sync();
+            bf16* y = reinterpret_cast<bf16*>(a.y);
+            for (int idx = etid; idx < C::kChunk * (BM / 8); idx += kEpiThreads) {
+              const int t = t0 + c0 + idx / (BM / 8), col = row_tile * BM + (idx % (BM / 8)) * 8;
+              if (t < t_end && col < a.out)
+                *reinterpret_cast<uint4*>(y + (size_t)t * a.ldy + y_col + col) = reinterpret_cast<const uint4*>(so)[idx];
+            }
+            return;
+          }
           if (row < a.out) {
 #pragma unroll
-            for (int i = 0; i < C::kChunk; ++i) {
-              const int t = t0 + c0 + i;
-              if (t < t_end) {
-                float o = v[i];
-                if (p.g.gate != nullptr) o = o / (1.f + __expf(-__bfloat162float(p.g.gate[(size_t)t * p.g.ld_gate + group])));
-                store_out(a, t, y_col + row, o);
-              }
-            }
+            for (int i = 0; i < C::kChunk; ++i)
+              if (t0 + c0 + i < t_end) store_out(a, t0 + c0 + i, y_col + row, v[i]);
           }
           return;
         }

@@ -1,19 +1,19 @@
 // Mixture-of-experts bookkeeping on the device: per token the `top` experts with the largest router logits and the softmax
 // over exactly those logits, and the grouping of all (token, expert) pairs by expert that the grouped projections read.
 //
-//   plan_small  one CTA does everything when there are few pairs (decode steps);
-//   route, then the framework's stable bucket sort with the expert as the key, then finish: prompt passes.
+//   decode sizes: one launch for everything, router included -- a CTA per token computes its logits and chooses, the last
+//   one to finish groups the pairs;
+//   prompt passes: route (choice, and the pairs' ranks inside their CTA), scan, scatter.
 // Either way pairs of one expert stay in token order, so the grouping is deterministic.
-#include <cfloat>
-
-#include "common.cuh"
+#include "act_io.cuh"
 
 namespace mlora {
 namespace {
 
-constexpr int kMoeThreads = 1024;
-constexpr int kMoeSmall = 2048;      // pairs one CTA handles by itself
 constexpr int kMoeMaxExperts = 1024;
+constexpr int kDecodeTokens = 64;    // one-launch form: tokens
+constexpr int kDecodePairs = 1024;   //                  and pairs
+constexpr int kLocalPairs = 4096;    // pairs of one CTA of the route kernel
 
 // One warp: experts and weights of one token.  Selected in order of decreasing logit, lower index first among equals.
 __device__ __forceinline__ void route_token(const float* __restrict__ z, const float* __restrict__ bias, int E, int top,
@@ -55,48 +55,87 @@ struct PlanOut {
   int32_t* tiles;  // [4 + 4 * max_tiles]: count, 0, 0, 0, then (expert, first row, rows, 0)
 };
 
-__global__ void __launch_bounds__(kMoeThreads) moe_plan_small_kernel(const float* __restrict__ logits, int64_t ld,
-                                                                     const float* __restrict__ bias, int T, int E, int top,
-                                                                     int tile_rows, PlanOut o) {
-  __shared__ int s_e[kMoeSmall];
+// Exclusive sums over the experts of their rows and of their tiles, by one warp; writes the tile count.
+__device__ __forceinline__ void scan_experts(const int* s_cnt, int* s_off, int* s_tile, int E, int tile_rows, int32_t* n_tiles) {
+  const int lane = threadIdx.x & 31;
+  int rows = 0, tiles = 0;
+  for (int e0 = 0; e0 < E; e0 += 32) {
+    const int e = e0 + lane, c = e < E ? s_cnt[e] : 0, nt = (c + tile_rows - 1) / tile_rows;
+    int a = c, b = nt;
+#pragma unroll
+    for (int d = 1; d < 32; d <<= 1) {
+      const int pa = __shfl_up_sync(0xffffffffu, a, d), pb = __shfl_up_sync(0xffffffffu, b, d);
+      if (lane >= d) a += pa, b += pb;
+    }
+    if (e < E) s_off[e] = rows + a - c, s_tile[e] = tiles + b - nt;
+    rows += __shfl_sync(0xffffffffu, a, 31);
+    tiles += __shfl_sync(0xffffffffu, b, 31);
+  }
+  if (lane == 0) *n_tiles = tiles;
+}
+__device__ __forceinline__ void write_tiles(const int* s_cnt, const int* s_off, const int* s_tile, int E, int tile_rows, int32_t* tiles) {
+  for (int e = threadIdx.x; e < E; e += blockDim.x)
+    for (int r = 0, i = s_tile[e]; r < s_cnt[e]; r += tile_rows, ++i)
+      reinterpret_cast<int4*>(tiles)[1 + i] = make_int4(e, s_off[e] + r, min(tile_rows, s_cnt[e] - r), 0);
+}
+
+// CTA = token.  z = W h + bias in fp32 (a warp takes every eighth expert), choice by warp 0; the last CTA groups.
+template <typename A>
+__global__ void __launch_bounds__(256) moe_decode_kernel(const A* __restrict__ h, int64_t ldh, const A* __restrict__ W, int in,
+                                                         const float* __restrict__ bias, int T, int E, int top, int tile_rows,
+                                                         PlanOut o, int32_t* __restrict__ ticket) {
+  __shared__ float s_z[kMoeMaxExperts];
   __shared__ int s_cnt[kMoeMaxExperts], s_off[kMoeMaxExperts], s_tile[kMoeMaxExperts];
+  __shared__ int s_e[kDecodePairs];
+  __shared__ int s_last;
   pdl_launch_dependents();
   pdl_wait();
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, n = T * top;
-  for (int t = warp; t < T; t += kMoeThreads / 32) {
-    route_token(logits + (size_t)t * ld, bias, E, top, o.idx + (size_t)t * top, o.wt + (size_t)t * top);
-    __syncwarp();
-    for (int k = lane; k < top; k += 32) s_e[t * top + k] = o.idx[(size_t)t * top + k];
-  }
-  for (int e = tid; e < E; e += kMoeThreads) s_cnt[e] = 0;
-  __syncthreads();
-  for (int i = tid; i < n; i += kMoeThreads) atomicAdd(&s_cnt[s_e[i]], 1);
-  __syncthreads();
-  // exclusive sums over the experts of their rows and of their tiles (one warp)
-  if (warp == 0) {
-    int rows = 0, tiles = 0;
-    for (int e0 = 0; e0 < E; e0 += 32) {
-      const int e = e0 + lane, c = e < E ? s_cnt[e] : 0, nt = (c + tile_rows - 1) / tile_rows;
-      int a = c, b = nt;
+  const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, n = T * top;
+  const A* x = h + (size_t)t * ldh;
+  for (int e0 = warp; e0 < E; e0 += 32) {  // four experts of the warp at a time
+    float acc[4] = {};
+    for (int k = lane * 8; k < in; k += 256) {
+      float xv[8], wv[8];
+      load8(x + k, xv);
 #pragma unroll
-      for (int d = 1; d < 32; d <<= 1) {
-        const int pa = __shfl_up_sync(0xffffffffu, a, d), pb = __shfl_up_sync(0xffffffffu, b, d);
-        if (lane >= d) a += pa, b += pb;
+      for (int j = 0; j < 4; ++j) {
+        if (e0 + 8 * j < E) {
+          load8(W + (size_t)(e0 + 8 * j) * in + k, wv);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) acc[j] = fmaf(xv[i], wv[i], acc[j]);
+        }
       }
-      if (e < E) s_off[e] = rows + a - c, s_tile[e] = tiles + b - nt;
-      rows += __shfl_sync(0xffffffffu, a, 31);
-      tiles += __shfl_sync(0xffffffffu, b, 31);
     }
-    if (lane == 0) o.tiles[0] = tiles;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float z = warp_sum(acc[j]);
+      if (lane == 0 && e0 + 8 * j < E) s_z[e0 + 8 * j] = z;
+    }
   }
   __syncthreads();
-  for (int e = tid; e < E; e += kMoeThreads)
-    for (int r = 0, i = s_tile[e]; r < s_cnt[e]; r += tile_rows, ++i)
-      reinterpret_cast<int4*>(o.tiles)[1 + i] = make_int4(e, s_off[e] + r, min(tile_rows, s_cnt[e] - r), 0);
+  if (warp == 0) {
+    route_token(s_z, bias, E, top, o.idx + (size_t)t * top, o.wt + (size_t)t * top);
+    __threadfence();
+    __syncwarp();
+    if (lane == 0) s_last = atomicAdd(ticket, 1) == T - 1;
+  }
+  __syncthreads();
+  if (!s_last) return;
+  if (tid == 0) *ticket = 0;  // ready for the next call
+  __threadfence();
+  for (int i = tid; i < n; i += 256) s_e[i] = __ldcg(o.idx + i);
+  for (int e = tid; e < E; e += 256) s_cnt[e] = 0;
+  __syncthreads();
+  for (int i = tid; i < n; i += 256) atomicAdd(&s_cnt[s_e[i]], 1);
+  __syncthreads();
+  if (warp == 0) scan_experts(s_cnt, s_off, s_tile, E, tile_rows, o.tiles);
+  __syncthreads();
+  write_tiles(s_cnt, s_off, s_tile, E, tile_rows, o.tiles);
   // row of pair i = first row of its expert + pairs of the same expert before it
-  for (int i = tid; i < n; i += kMoeThreads) {
+  for (int i = tid; i < n; i += 256) {
     const int e = s_e[i];
     int before = 0;
+#pragma unroll 8
     for (int j = 0; j < i; ++j) before += s_e[j] == e;
     const int p = s_off[e] + before;
     o.pos[i] = p;
@@ -104,56 +143,72 @@ __global__ void __launch_bounds__(kMoeThreads) moe_plan_small_kernel(const float
   }
 }
 
-__global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int64_t ld,
-                                                        const float* __restrict__ bias, int T, int E, int top,
-                                                        int32_t* __restrict__ idx, float* __restrict__ wt) {
+// Prompt passes.  CTA c: tokens [c * per, ...); hist[c * E + e] = its pairs of expert e; rank (in o.pos) = place of a pair
+// among the CTA's pairs of its expert.
+__global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int64_t ld, const float* __restrict__ bias,
+                                                        int T, int E, int top, int per, PlanOut o, int32_t* __restrict__ hist) {
+  __shared__ int s_e[kLocalPairs];
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (t < T) route_token(logits + (size_t)t * ld, bias, E, top, idx + (size_t)t * top, wt + (size_t)t * top);
+  const int t0 = blockIdx.x * per, n = (min(T, t0 + per) - t0) * top, warp = threadIdx.x >> 5;
+  for (int t = t0 + warp; t < min(T, t0 + per); t += 8) {
+    route_token(logits + (size_t)t * ld, bias, E, top, o.idx + (size_t)t * top, o.wt + (size_t)t * top);
+    __syncwarp();
+    for (int k = threadIdx.x & 31; k < top; k += 32) s_e[(t - t0) * top + k] = o.idx[(size_t)t * top + k];
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += 256) {
+    int c = 0;
+#pragma unroll 8
+    for (int i = 0; i < n; ++i)
+      if (s_e[i] == e) o.pos[(size_t)t0 * top + i] = c++;
+    hist[(size_t)blockIdx.x * E + e] = c;
+  }
 }
 
-// perm / segments: the bucket sort's outputs.  CTA 0 writes the tile table as well.
-__global__ void __launch_bounds__(256) moe_finish_kernel(const int32_t* __restrict__ perm, const int32_t* __restrict__ seg_off,
-                                                         const int32_t* __restrict__ seg_expert,
-                                                         const int32_t* __restrict__ counts, int n, int top, int tile_rows,
-                                                         PlanOut o) {
-  __shared__ int s_first[kMoeMaxExperts];
+// One CTA: hist[c][e] becomes the first row of CTA c's pairs of expert e; the tile table.
+__global__ void __launch_bounds__(1024) moe_scan_kernel(int32_t* __restrict__ hist, int n_cta, int E, int tile_rows, PlanOut o) {
+  __shared__ int s_cnt[kMoeMaxExperts], s_off[kMoeMaxExperts], s_tile[kMoeMaxExperts];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int e = warp; e < E; e += 32) {
+    int total = 0;
+    for (int c = lane; c < n_cta; c += 32) total += hist[(size_t)c * E + e];
+    total = __reduce_add_sync(0xffffffffu, total);
+    if (lane == 0) s_cnt[e] = total;
+  }
+  __syncthreads();
+  if (warp == 0) scan_experts(s_cnt, s_off, s_tile, E, tile_rows, o.tiles);
+  __syncthreads();
+  write_tiles(s_cnt, s_off, s_tile, E, tile_rows, o.tiles);
+  for (int e = warp; e < E; e += 32) {
+    int run = s_off[e];
+    for (int c0 = 0; c0 < n_cta; c0 += 32) {
+      const int c = c0 + lane, v = c < n_cta ? hist[(size_t)c * E + e] : 0;
+      int a = v;
+#pragma unroll
+      for (int d = 1; d < 32; d <<= 1) {
+        const int p = __shfl_up_sync(0xffffffffu, a, d);
+        if (lane >= d) a += p;
+      }
+      if (c < n_cta) hist[(size_t)c * E + e] = run + a - v;
+      run += __shfl_sync(0xffffffffu, a, 31);
+    }
+  }
+}
+
+__global__ void __launch_bounds__(256) moe_scatter_kernel(const int32_t* __restrict__ first, int n, int E, int top, int per, PlanOut o) {
   pdl_launch_dependents();
   pdl_wait();
   const int i = blockIdx.x * 256 + threadIdx.x;
-  if (i < n) {
-    const int p = perm[i];
-    o.pos[p] = i;
-    o.rows[i] = p / top;
-  }
-  if (blockIdx.x != 0) return;
-  const int n_seg = counts[0];
-  if (threadIdx.x < 32) {
-    int tiles = 0;
-    for (int s0 = 0; s0 < n_seg; s0 += 32) {
-      const int s = s0 + threadIdx.x;
-      const int nt = s < n_seg ? (seg_off[s + 1] - seg_off[s] + tile_rows - 1) / tile_rows : 0;
-      int b = nt;
-#pragma unroll
-      for (int d = 1; d < 32; d <<= 1) {
-        const int pb = __shfl_up_sync(0xffffffffu, b, d);
-        if ((int)threadIdx.x >= d) b += pb;
-      }
-      if (s < n_seg) s_first[s] = tiles + b - nt;
-      tiles += __shfl_sync(0xffffffffu, b, 31);
-    }
-    if (threadIdx.x == 0) o.tiles[0] = tiles;
-  }
-  __syncthreads();
-  for (int s = threadIdx.x; s < n_seg; s += 256) {
-    const int a = seg_off[s], c = seg_off[s + 1] - a;
-    for (int r = 0, j = s_first[s]; r < c; r += tile_rows, ++j)
-      reinterpret_cast<int4*>(o.tiles)[1 + j] = make_int4(seg_expert[s], a + r, min(tile_rows, c - r), 0);
-  }
+  if (i >= n) return;
+  const int t = i / top, p = first[(size_t)(t / per) * E + o.idx[i]] + o.pos[i];
+  o.pos[i] = p;
+  o.rows[p] = t;
 }
 
-size_t align256(size_t n) { return (n + 255) & ~(size_t)255; }
+int tokens_per_cta(int top) { return kLocalPairs / top < 64 ? kLocalPairs / top : 64; }
 
 }  // namespace
 }  // namespace mlora
@@ -161,53 +216,59 @@ size_t align256(size_t n) { return (n + 255) & ~(size_t)255; }
 using namespace mlora;
 
 extern "C" size_t mlora_moe_plan_workspace(int32_t T, int32_t E, int32_t top) {
-  const int64_t n = (int64_t)T * top;
-  if (T <= 0 || E <= 0 || top <= 0 || n <= kMoeSmall || n > 0x7fffffff) return 0;
-  return 3 * align256(4 * (size_t)n) + 3 * align256(4 * (size_t)(E + 2)) + 256 +
-         align256(mlora_bucket_sort_workspace((int32_t)n, 1, E));
+  if (T <= 0 || E <= 0 || top <= 0 || top > E || E > kMoeMaxExperts) return 256;
+  const int per = tokens_per_cta(top);
+  return 256 + (size_t)((T + per - 1) / per) * E * sizeof(int32_t);
 }
+
+#define MOE_CHECK(what)                                                                                                        \
+  MLORA_REQUIRE(T >= 0 && E > 0 && E <= kMoeMaxExperts && top > 0 && top <= E && tile_rows > 0,                                \
+                what ": bad sizes T=%d experts=%d (at most %d) top=%d", T, E, kMoeMaxExperts, top);                            \
+  MLORA_REQUIRE(d_bias && d_expert && d_weight && d_pos && d_rows && d_tiles && aligned16(d_tiles) && d_work,                  \
+                what ": null or unaligned pointer");                                                                           \
+  MLORA_REQUIRE((int64_t)T * top <= 0x7fffffff, what ": too many (token, expert) pairs");                                      \
+  MLORA_REQUIRE(work_bytes >= mlora_moe_plan_workspace(T, E, top), what ": workspace of %zu bytes needed, %zu given",           \
+                mlora_moe_plan_workspace(T, E, top), work_bytes)
 
 extern "C" int mlora_moe_plan(const float* d_logits, int64_t ld, const float* d_bias, int32_t T, int32_t E, int32_t top,
                               int32_t tile_rows, int32_t* d_expert, float* d_weight, int32_t* d_pos, int32_t* d_rows,
                               int32_t* d_tiles, void* d_work, size_t work_bytes, void* stream) {
-  MLORA_REQUIRE(T >= 0 && E > 0 && E <= kMoeMaxExperts && top > 0 && top <= E && tile_rows > 0 && ld >= E,
-                "moe_plan: bad sizes T=%d experts=%d (at most %d) top=%d", T, E, kMoeMaxExperts, top);
-  MLORA_REQUIRE(d_logits && d_bias && d_expert && d_weight && d_pos && d_rows && d_tiles && aligned16(d_tiles),
-                "moe_plan: null or unaligned pointer");
-  MLORA_REQUIRE((int64_t)T * top <= 0x7fffffff, "moe_plan: too many (token, expert) pairs");
+  MOE_CHECK("moe_plan");
+  MLORA_REQUIRE(d_logits && ld >= E, "moe_plan: null logits or pitch below the number of experts");
   if (T == 0) return MLORA_OK;
   cudaStream_t st = (cudaStream_t)stream;
   const PlanOut o{d_expert, d_weight, d_pos, d_rows, d_tiles};
-  const int n = T * top;
-  if (n <= kMoeSmall) {
-    launch_pdl(moe_plan_small_kernel, 1, kMoeThreads, 0, st, d_logits, ld, d_bias, T, E, top, tile_rows, o);
-    count_launch();
-    MLORA_CHECK_LAUNCH("moe_plan_small_kernel");
-    return MLORA_OK;
-  }
-  const size_t need = mlora_moe_plan_workspace(T, E, top);
-  MLORA_REQUIRE(d_work && work_bytes >= need, "moe_plan: workspace of %zu bytes needed, %zu given", need, work_bytes);
-  uint8_t* w = (uint8_t*)d_work;
-  auto take = [&](size_t bytes) {
-    uint8_t* p = w;
-    w += align256(bytes);
-    return (int32_t*)p;
-  };
-  int32_t* perm = take(4 * (size_t)n);
-  int32_t* s_tid = take(4 * (size_t)n);
-  int32_t* s_wid = take(4 * (size_t)n);
-  int32_t* seg_off = take(4 * (size_t)(E + 2));
-  int32_t* seg_tid = take(4 * (size_t)(E + 2));
-  int32_t* seg_wid = take(4 * (size_t)(E + 2));
-  int32_t* counts = take(256);
-  launch_pdl(moe_route_kernel, (T + 7) / 8, 256, 0, st, d_logits, ld, d_bias, T, E, top, d_expert, d_weight);
+  const int n = T * top, per = tokens_per_cta(top), n_cta = (T + per - 1) / per;
+  int32_t* hist = (int32_t*)((uint8_t*)d_work + 256);
+  launch_pdl(moe_route_kernel, n_cta, 256, 0, st, d_logits, ld, d_bias, T, E, top, per, o, hist);
+  launch_pdl(moe_scan_kernel, 1, 1024, 0, st, hist, n_cta, E, tile_rows, o);
+  launch_pdl(moe_scatter_kernel, (n + 255) / 256, 256, 0, st, hist, n, E, top, per, o);
+  count_launch(3);
+  MLORA_CHECK_LAUNCH("moe_plan");
+  return MLORA_OK;
+}
+
+extern "C" uint32_t mlora_moe_decode_fits(int32_t T, int32_t top) {
+  return T > 0 && T <= kDecodeTokens && top > 0 && (int64_t)T * top <= kDecodePairs ? 1u : 0u;
+}
+
+extern "C" int mlora_moe_route_plan(const void* d_h, int64_t ldh, const void* d_W, int32_t in, const float* d_bias, int32_t T,
+                                    int32_t E, int32_t top, int32_t tile_rows, int32_t* d_expert, float* d_weight,
+                                    int32_t* d_pos, int32_t* d_rows, int32_t* d_tiles, void* d_work, size_t work_bytes,
+                                    int32_t f32, void* stream) {
+  MOE_CHECK("moe_route_plan");
+  MLORA_REQUIRE(T == 0 || mlora_moe_decode_fits(T, top), "moe_route_plan: at most %d tokens and %d pairs", kDecodeTokens, kDecodePairs);
+  MLORA_REQUIRE(d_h && d_W && in > 0 && in % 8 == 0 && ldh % 8 == 0 && aligned16(d_h) && aligned16(d_W),
+                "moe_route_plan: h and W 16-byte aligned, in and ldh multiples of 8");
+  if (T == 0) return MLORA_OK;
+  const PlanOut o{d_expert, d_weight, d_pos, d_rows, d_tiles};
+  if (f32)
+    launch_pdl_if(pdl_enabled_norm(), moe_decode_kernel<float>, T, 256, 0, (cudaStream_t)stream, (const float*)d_h, ldh,
+                  (const float*)d_W, in, d_bias, T, E, top, tile_rows, o, (int32_t*)d_work);
+  else
+    launch_pdl_if(pdl_enabled_norm(), moe_decode_kernel<bf16>, T, 256, 0, (cudaStream_t)stream, (const bf16*)d_h, ldh,
+                  (const bf16*)d_W, in, d_bias, T, E, top, tile_rows, o, (int32_t*)d_work);
   count_launch();
-  MLORA_CHECK_LAUNCH("moe_route_kernel");
-  const int rc = mlora_bucket_sort(nullptr, d_expert, n, 1, E, 0, perm, s_tid, s_wid, seg_off, seg_tid, seg_wid, counts, w,
-                                   mlora_bucket_sort_workspace(n, 1, E), stream);
-  if (rc != MLORA_OK) return rc;
-  launch_pdl(moe_finish_kernel, (n + 255) / 256, 256, 0, st, perm, seg_off, seg_wid, counts, n, top, tile_rows, o);
-  count_launch();
-  MLORA_CHECK_LAUNCH("moe_finish_kernel");
+  MLORA_CHECK_LAUNCH("moe_decode_kernel");
   return MLORA_OK;
 }

@@ -581,6 +581,23 @@ def moe_plan(logits, bias, plan: MoePlan, T, tile_rows):
     return plan
 
 
+def moe_decode_fits(T, top) -> bool:
+    return bool(_lib.lib().mlora_moe_decode_fits(T, top))
+
+
+def moe_route_plan(h, W, bias, plan: MoePlan, tile_rows):
+    """Router and plan of a decode step's tokens in one launch; W [E, in] row-major in h's dtype."""
+    _need_cuda(h, W)
+    T = h.shape[0]
+    plan.tile_rows = tile_rows
+    plan.max_tiles = T * plan.top // tile_rows + min(plan.E, T * plan.top)
+    check(_lib.lib().mlora_moe_route_plan(_ptr(h), h.stride(0), _ptr(W), W.shape[1], _ptr(bias), T, plan.E, plan.top, tile_rows,
+                                          _ptr(plan.expert), _ptr(plan.weight), _ptr(plan.pos), _ptr(plan.rows),
+                                          _ptr(plan.tiles), _ptr(plan.work), plan.work.numel(), int(h.dtype == torch.float32),
+                                          _stream()), "mlora_moe_route_plan")
+    return plan
+
+
 # ---------------------------------------------------------------- dynamic tanh norm
 def residual_dyt(delta, res, w, b, alpha, out, expert_rows=None, plan: MoePlan = None, rows=None):
     """res += delta (+ the plan's weighted expert rows); out = tanh(alpha res) w + b; see ``mlora_residual_dyt``."""

@@ -149,7 +149,7 @@ def tevudra_weights(cfg: dict, dtype=torch.bfloat16, device="cpu") -> dict:
         if f["kind"] == "dense":
             feed_forward(f"l{i}.mlp", f["ff"])
             continue
-        p[f"l{i}.mlp.router"], p[f"l{i}.mlp.router.b"] = mat(f["router"]["experts"], W), rnd(f["router"]["experts"]).to(dtype)
+        p[f"l{i}.mlp.router"], p[f"l{i}.mlp.router.b"] = (4 * mat(f["router"]["experts"], W)).to(dtype), (0.1 * rnd(f["router"]["experts"])).to(dtype)
         for e in range(f["router"]["experts"]):
             feed_forward(f"l{i}.mlp.e{e}", f["expert"]["ff"])
         if f.get("shared"):

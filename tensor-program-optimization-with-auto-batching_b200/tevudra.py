@@ -173,7 +173,8 @@ class PackedTevudra:
             lw.up, lw.down = self._weight(get(p + "up"), (lw.ffp, H)), self._weight(get(p + "down"), (H, lw.ffp))
             return lw
         lw.ffp = _up(ff.ff, 8)
-        lw.router = self._weight(get(p + "router"), (_up(ff.experts, 4), H))
+        lw.router_rows = self._mat(get(p + "router"), (ff.experts, H))  # decode steps: routed in one launch
+        lw.router = ops.GroupedWeight(lw.router_rows[None])
         lw.router_b = get(p + "router.b").to(dev, torch.float32).contiguous()
         stack = lambda n, shape: ops.GroupedWeight(torch.stack([self._mat(get(f"{p}e{e}.{n}"), shape) for e in range(ff.experts)]))
         lw.e_up, lw.e_down = stack("up", (lw.ffp, H)), stack("down", (H, lw.ffp))
@@ -221,7 +222,7 @@ class TevudraEngine(EngineBase):
                 key = (lw.ff.experts, lw.ff.top)
                 if key not in self.plans:
                     self.plans[key] = ops.MoePlan(T, *key, dev)
-            self.router_out = torch.zeros(T * widest(lambda lw: _up(lw.ff.experts, 4), moes), dtype=torch.float32, device=dev)
+            self.router_out = torch.zeros(T * widest(lambda lw: lw.ff.experts, moes), dtype=torch.float32, device=dev)
             self.e_act = torch.zeros(widest(lambda lw: pairs(lw) * lw.ffp, moes), **act)
             self.e_out = torch.zeros(widest(lambda lw: pairs(lw) * m.H, moes), **act)
         lib = ops._lib.lib()
@@ -231,7 +232,7 @@ class TevudraEngine(EngineBase):
             if isinstance(lw.ff, Dense):
                 shapes += [(m.H, lw.ffp), (lw.ffp, m.H)]
             elif lw.ff is not None:
-                shapes += [(m.H, lw.ff.experts)] + ([(m.H, lw.sffp), (lw.sffp, m.H)] if lw.ff.shared_ff else [])
+                shapes += [(m.H, lw.sffp), (lw.sffp, m.H)] if lw.ff.shared_ff else []
         # (the expansion of a context may have more rows than the pass: scratch no longer grows beyond 128)
         need = max([lib.mlora_linear_workspace(max(T, 128), k, n) for k, n in shapes] + [lib.mlora_grouped_linear_workspace(64)])
         self.ws_linear = ops.new_workspace(need, dev)
@@ -291,11 +292,14 @@ class TevudraEngine(EngineBase):
 
     # -- pieces of a layer ----------------------------------------------------------------------------------------
     def _linear(self, x, W, out, flags=0):
-        if self.m.dtype == torch.float32:
+        if self.m.dtype == torch.float32:  # (OUT_F32: what it writes anyway)
             return ops.linear_f32(x, W, flags & ~OUT_F32, out=out)
         return ops.linear(x, W, flags=flags, out=out, work=self.ws_linear)
 
-    def _grouped(self, x, W, out, **kw):
+    def _grouped(self, x, W, out, flags=0, **kw):
+        if self.m.dtype == torch.float32:
+            flags &= ~OUT_F32
+        kw["flags"] = flags
         return ops.grouped_linear(x, W, out, work=self.ws_linear, **kw)
 
     def _attention(self, T, lw, fused_append):
@@ -334,12 +338,19 @@ class TevudraEngine(EngineBase):
         if isinstance(ff, Dense):
             a = self._linear(xn, lw.up, self.act[:T * lw.ffp].view(T, lw.ffp), ACT_RELU2)
             return self._linear(a, lw.down, y), None, None
-        E = _up(ff.experts, 4)
-        logits = self._linear(xn, lw.router, self.router_out[:T * E].view(T, E), OUT_F32)
-        plan = ops.moe_plan(logits, lw.router_b, self.plans[ff.experts, ff.top], T,
-                            ops.grouped_tile_rows(T * ff.top / ff.experts, m.dtype))
-        n = T * ff.top
-        a = self._grouped(xn, lw.e_up, self.e_act[:n * lw.ffp].view(n, lw.ffp), plan=plan, gather=True, flags=ACT_GELU)
+        plan, n = self.plans[ff.experts, ff.top], T * ff.top
+        tr = ops.grouped_tile_rows(n / ff.experts, m.dtype)
+        if ops.moe_decode_fits(T, ff.top):
+            ops.moe_route_plan(xn, lw.router_rows, lw.router_b, plan, tr)
+        else:
+            # few outputs, many rows: 64-row tiles fill the grid where the plain projection's larger ones do not
+            logits = self._grouped(xn, lw.router, self.router_out[:T * ff.experts].view(T, ff.experts), T=T, tile_rows=64, flags=OUT_F32)
+            ops.moe_plan(logits, lw.router_b, plan, T, tr)
+        x, gather = xn, True
+        if m.dtype == torch.bfloat16 and tr >= 128:
+            # large tiles: rows copied into expert order first (four-row gathers cannot keep up with the tensor cores)
+            x, gather = ops.embed(plan.rows[:n], xn, out_bf16=self._grow("e_in", n * m.H).view(n, m.H)), False
+        a = self._grouped(x, lw.e_up, self.e_act[:n * lw.ffp].view(n, lw.ffp), plan=plan, gather=gather, flags=ACT_GELU)
         e = self._grouped(a, lw.e_down, self.e_out[:n * m.H].view(n, m.H), plan=plan)
         if not ff.shared_ff:
             return None, e, plan

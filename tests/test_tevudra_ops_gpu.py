@@ -70,7 +70,23 @@ def test_moe_plan(ops, cuda, T, E, top, tile):
     b[: E // 2] = 0.5  # equal logits in token 0: the lower index first
     plan = ops.MoePlan(T, E, top, cuda)
     ops.moe_plan(z.to(cuda), b.to(cuda), plan, T, tile)
-    total = z[:, :E] + b
+    _check_plan(plan, z[:, :E] + b, T, E, top, tile)
+
+
+@pytest.mark.parametrize("dtype", [BF, F32])
+@pytest.mark.parametrize("T,E,top,width", [(1, 1, 1, 8), (1, 12, 2, 40), (5, 7, 7, 320), (32, 70, 6, 264), (64, 300, 8, 1000), (64, 5, 3, 72)])
+def test_moe_route_plan_in_one_launch(ops, cuda, dtype, T, E, top, width):
+    g = gen(E + T)
+    # small integers: the logits are exact in fp32 whatever the order of the sum
+    h, W = (torch.randint(-3, 4, s, generator=g).to(dtype) for s in ((T, width), (E, width)))
+    b = torch.randn(E, generator=g)
+    plan = ops.MoePlan(T, E, top, cuda)
+    for _ in range(2):  # (the ticket resets itself)
+        ops.moe_route_plan(h.to(cuda), W.to(cuda), b.to(cuda), plan, 16)
+        _check_plan(plan, h.float() @ W.float().T + b, T, E, top, 16)
+
+
+def _check_plan(plan, total, T, E, top, tile):
     order = torch.sort(total, dim=-1, descending=True, stable=True)
     idx, wt = plan.expert[:T * top].cpu().view(T, top), plan.weight[:T * top].cpu().view(T, top)
     assert torch.equal(idx.long(), order.indices[:, :top])
