@@ -485,8 +485,10 @@ int mlora_residual_dyt(const void* d_delta, const void* d_expert_rows, const int
                        int32_t T, int32_t H, int32_t f32, void* stream);
 
 /* ---- latent attention ----------------------------------------------------------------------------------------
- * The cache holds one vector of R = kv_rank values per token (pages [n_pages, page_size, pitch], bf16 or fp32); keys and
- * values of all heads are linear maps of it.
+ * The cache holds one vector of R = kv_rank values per token (pages of page_size * pitch elements, bf16 or fp32, pitch = R
+ * rounded up to 64); keys and values of all heads are linear maps of it.  A page is stored as
+ * [page_size / 8][pitch / 64][8 rows][64 columns], the 8-column chunk c of a row at place c ^ (row & 7): the image the tensor
+ * cores read, so that a page is one contiguous copy (csrc/latent.cuh).
  * mlora_latent_append: c = x / sqrt(mean(x^2) + eps) * w into the row's place (rows with row_pos < 0 are skipped).
  * mlora_latent_gather: segments int32 [n][4] = (cache slot, first output row (a multiple of page_size), tokens, 0): the
  *   pages of the sequence as consecutive rows (bf16), for callers that expand keys and values of a whole context.

@@ -7,6 +7,7 @@
 #include <cfloat>
 
 #include "act_io.cuh"
+#include "latent.cuh"
 
 namespace mlora {
 namespace {
@@ -34,8 +35,9 @@ __global__ void __launch_bounds__(256) latent_append_kernel(const A* __restrict_
   ss = warp_sum(ss);
   const float inv = 1.f / sqrtf(ss / (float)R + eps);
   const int page = bt[(size_t)row_slot[t] * max_pages + pos / page_size];
-  A* c = pages + ((size_t)page * page_size + pos % page_size) * pitch;
-  for (int k = lane; k < pitch; k += 32) c[k] = from_f32<A>(k < R ? to_f32(xr[k]) * inv * to_f32(w[k]) : 0.f);
+  A* c = pages + (size_t)page * page_size * pitch;
+  for (int k = lane; k < pitch; k += 32)
+    c[latent_offset(pos % page_size, k, pitch)] = from_f32<A>(k < R ? to_f32(xr[k]) * inv * to_f32(w[k]) : 0.f);
 }
 
 // CTA (page p, segment s): rows [base, base + page_size) of the dense copy = page p of the segment's sequence.
@@ -47,7 +49,11 @@ __global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* __restr
   if (p * page_size >= sg.z || p >= max_pages) return;
   const uint4* src = pages + (size_t)bt[(size_t)sg.x * max_pages + p] * vec_per_page;
   uint4* dst = out + ((size_t)sg.y / page_size + p) * vec_per_page;
-  for (int i = threadIdx.x; i < vec_per_page; i += 128) dst[i] = src[i];
+  const int per_row = vec_per_page / page_size;  // 16-byte chunks of a row
+  for (int i = threadIdx.x; i < vec_per_page; i += 128) {
+    const int row = i / per_row, c = i - row * per_row;
+    dst[i] = src[latent_offset(row, c * 8, per_row * 8) >> 3];
+  }
 }
 
 constexpr int kLaKeys = 64;   // keys per step
@@ -79,9 +85,10 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const A* __restrict__ 
   for (int k0 = 0; k0 < n; k0 += kLaKeys) {
     const int m = min(kLaKeys, n - k0);
     for (int j = warp; j < m; j += 4) {
-      const A* c = pages + ((size_t)table[(k0 + j) / page_size] * page_size + (k0 + j) % page_size) * pitch;
+      const A* c = pages + (size_t)table[(k0 + j) / page_size] * page_size * pitch;
+      const int r = (k0 + j) % page_size;
       float s = 0.f;
-      for (int k = lane; k < R; k += 32) s = fmaf(s_q[k], to_f32(c[k]), s);
+      for (int k = lane; k < R; k += 32) s = fmaf(s_q[k], to_f32(c[latent_offset(r, k, pitch)]), s);
       s = warp_sum(s);
       if (lane == 0) s_p[j] = s * scale;
     }
@@ -105,11 +112,12 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const A* __restrict__ 
 #pragma unroll
     for (int i = 0; i < kLaMaxAcc; ++i) acc[i] *= corr;
     for (int j = 0; j < m; ++j) {
-      const A* c = pages + ((size_t)table[(k0 + j) / page_size] * page_size + (k0 + j) % page_size) * pitch;
+      const A* c = pages + (size_t)table[(k0 + j) / page_size] * page_size * pitch;
+      const int r = (k0 + j) % page_size;
       const float p = s_p[j];
 #pragma unroll
       for (int i = 0; i < kLaMaxAcc; ++i)
-        if (tid + i * 128 < R) acc[i] = fmaf(p, to_f32(c[tid + i * 128]), acc[i]);
+        if (tid + i * 128 < R) acc[i] = fmaf(p, to_f32(c[latent_offset(r, tid + i * 128, pitch)]), acc[i]);
     }
     __syncthreads();
   }
@@ -127,15 +135,19 @@ using namespace mlora;
 extern "C" int mlora_latent_append(const void* d_x, int64_t ld, int32_t R, const void* d_w, float eps, void* d_pages,
                                    int32_t pitch, int32_t page_size, const int32_t* d_block_table, int32_t max_pages,
                                    const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, int32_t f32, void* stream) {
-  MLORA_REQUIRE(T >= 0 && R > 0 && pitch >= R && page_size > 0 && max_pages > 0 && ld >= R, "latent_append: bad sizes");
+  MLORA_REQUIRE(T >= 0 && R > 0 && pitch >= R && pitch % 64 == 0 && page_size > 0 && page_size % 8 == 0 && max_pages > 0 && ld >= R,
+                "latent_append: bad sizes (pitch a multiple of 64, page size of 8)");
   MLORA_REQUIRE(d_x && d_w && d_pages && d_block_table && d_row_slot && d_row_pos, "latent_append: null pointer");
   if (T == 0) return MLORA_OK;
+  const auto launch = [&](auto zero) {
+    using A = decltype(zero);
+    launch_pdl_if(pdl_enabled_norm(), latent_append_kernel<A>, (T + 7) / 8, 256, 0, (cudaStream_t)stream, (const A*)d_x, ld, R, (const bf16*)d_w, eps,
+                  (A*)d_pages, pitch, page_size, d_block_table, max_pages, d_row_slot, d_row_pos, T);
+  };
   if (f32)
-    launch_pdl(latent_append_kernel<float>, (T + 7) / 8, 256, 0, (cudaStream_t)stream, (const float*)d_x, ld, R, (const bf16*)d_w,
-               eps, (float*)d_pages, pitch, page_size, d_block_table, max_pages, d_row_slot, d_row_pos, T);
+    launch(0.f);
   else
-    launch_pdl(latent_append_kernel<bf16>, (T + 7) / 8, 256, 0, (cudaStream_t)stream, (const bf16*)d_x, ld, R, (const bf16*)d_w, eps,
-               (bf16*)d_pages, pitch, page_size, d_block_table, max_pages, d_row_slot, d_row_pos, T);
+    launch(bf16());
   count_launch();
   MLORA_CHECK_LAUNCH("latent_append_kernel");
   return MLORA_OK;
@@ -144,7 +156,7 @@ extern "C" int mlora_latent_append(const void* d_x, int64_t ld, int32_t R, const
 extern "C" int mlora_latent_gather(const void* d_pages, int32_t pitch, int32_t page_size, const int32_t* d_block_table,
                                    int32_t max_pages, const int32_t* d_segs, int32_t n_segs, int32_t max_tokens, void* d_out,
                                    void* stream) {
-  MLORA_REQUIRE(n_segs >= 0 && n_segs <= 65535 && pitch > 0 && pitch % 8 == 0 && page_size > 0 && max_tokens >= 0, "latent_gather: bad sizes");
+  MLORA_REQUIRE(n_segs >= 0 && n_segs <= 65535 && pitch > 0 && pitch % 64 == 0 && page_size > 0 && page_size % 8 == 0 && max_tokens >= 0, "latent_gather: bad sizes");
   MLORA_REQUIRE(d_pages && d_block_table && d_segs && d_out && aligned16(d_pages) && aligned16(d_segs) && aligned16(d_out),
                 "latent_gather: null or unaligned pointer");
   if (n_segs == 0 || max_tokens == 0) return MLORA_OK;
@@ -159,7 +171,7 @@ extern "C" int mlora_latent_attention_simt(const void* d_qa, int64_t q_pitch, co
                                            int32_t page_size, const int32_t* d_block_table, int32_t max_pages,
                                            const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, int32_t H, float scale,
                                            void* d_out, int32_t f32, void* stream) {
-  MLORA_REQUIRE(T >= 0 && H > 0 && H <= 65535 && R > 0 && pitch >= R && q_pitch >= R && page_size > 0 && max_pages > 0,
+  MLORA_REQUIRE(T >= 0 && H > 0 && H <= 65535 && R > 0 && pitch >= R && pitch % 64 == 0 && q_pitch >= R && page_size > 0 && page_size % 8 == 0 && max_pages > 0,
                 "latent_attention_simt: bad sizes");
   MLORA_REQUIRE(q_pitch <= 128 * kLaMaxAcc, "latent_attention_simt: kv_rank up to %d (row pitch %lld)", 128 * kLaMaxAcc, (long long)q_pitch);
   MLORA_REQUIRE(d_qa && d_pages && d_block_table && d_row_slot && d_row_pos && d_out, "latent_attention_simt: null pointer");

@@ -9,27 +9,26 @@
 //                                                             contiguous dimension: no transpose is made), B = P
 // so both products read one copy of C, and a head is a TMEM lane for the softmax: one thread per head walks its 64 scores,
 // no value crosses lanes.  The scores and the probabilities are double buffered: the scores of block b + 1 are computed
-// while the softmax of block b runs, and the ring of 16 KB slots (64 keys x 128 latent columns) keeps streaming.  The
+// while the softmax of block b runs, and the ring of blocks keeps streaming.  A page lies in memory as the operand image
+// (latent.cuh) and arrives as one bulk copy: with a TMA box per 64 columns (2 KB) the copies' issue rate was the bound.  The
 // running maximum of a head is moved only when a block exceeds it by more than 2^8; only then do all four output warps
 // rescale the sums in TMEM, on request.
 //
-// Roles: warp 0 TMA, warp 1 MMA issue, warp 4 (TMEM lanes 0..31) softmax, warps 2..5 rescaling and output.
+// Roles: warp 0 copies, warp 1 MMA issue, warp 4 (TMEM lanes 0..31) softmax, warps 2..5 rescaling and output.
 // With several splits a CTA leaves unnormalised fp32 sums, its maxima and row sums, and a small kernel joins them.
 // Every wait is bounded; a CTA that gives up sets the status word and leaves its outputs undefined.
 #include <math.h>
 
 #include <atomic>
 
-#include "common.cuh"
+#include "latent.cuh"
 #include "tc_ptx.cuh"
 
 namespace mlora {
 namespace {
 
 constexpr int kKeys = 64;                      // keys per block
-constexpr int kSubTile = kKeys * 128;          // [64 keys][64 columns] bf16
-constexpr int kSlot = 2 * kSubTile;            // 128 columns
-constexpr int kMaxSlots = 13;
+constexpr int kMaxSlots = 8;                   // blocks in the ring
 constexpr int kLtThreads = 192;
 constexpr int kMaxChunks = 4;                  // kv_rank up to 512
 constexpr int kTmemCols = 512;                 // S: 2 x 64, O^T: 4 x 32, queries: 256
@@ -38,10 +37,11 @@ constexpr float kRescale = 8.f;                // (log2) how far scores may exce
 
 struct LtArgs {
   const int32_t* block_table;
-  int max_pages, page_size, n_page_rows;       // n_page_rows: rows of the page tensor (the first row that does not exist)
+  int max_pages, page_size;
+  const uint8_t* pages;
   const int32_t *row_slot, *row_pos;
   const bf16* qa;                              // [T, H, q_pitch]
-  int H, q_pitch, n_chunks, n_slots, n_splits;
+  int H, R, pitch, q_pitch, n_chunks, n_slots, n_splits;
   float scale_log2;
   bf16* out;                                   // [T, H, q_pitch]
   float* part;                                 // [T, H, n_splits, q_pitch] unnormalised sums
@@ -102,10 +102,11 @@ __device__ __forceinline__ void tmem_st(uint32_t addr, const float (&v)[32]) {
 }
 
 template <int HG>
-__global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __grid_constant__ CUtensorMap map_c, LtArgs a) {
+__global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(LtArgs a) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-  uint8_t* sp = ring + a.n_slots * kSlot;               // probabilities: two buffers [HG][64 keys]
+  const int slot_bytes = kKeys * a.pitch * 2;           // a block: row groups of 8 keys, slices of 64 columns
+  uint8_t* sp = ring + a.n_slots * slot_bytes;               // probabilities: two buffers [HG][64 keys]
   __shared__ uint64_t full_bar[kMaxSlots], empty_bar[kMaxSlots], q_bar, s_bar[2], p_bar[2], o_bar[2], cmd_bar, ack_bar;
   __shared__ uint32_t tmem_slot;
   __shared__ int s_abort, s_end;
@@ -145,7 +146,6 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __g
     mbar_init(&cmd_bar, 32);
     mbar_init(&ack_bar, 128);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-    tma_prefetch_desc(&map_c);
   }
   if (warp == 1) tmem_alloc(&tmem_slot, kTmemCols);
   tc_fence_before();
@@ -154,55 +154,52 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __g
   const uint32_t tmem_s = tmem_slot, tmem_o = tmem_s + 128, tmem_q = tmem_s + 256;
 
   if (warp == 0) {
-    // ---- producer ------------------------------------------------------------------------------------------------
+    // ---- producer: one page per lane -------------------------------------------------------------------------------
     const int32_t* bt = a.block_table + (size_t)a.row_slot[t] * a.max_pages;
-    const int ppb = kKeys / a.page_size, half = lane & 1, p = lane >> 1;  // one (page, column half) per lane
+    const int ppb = kKeys / a.page_size, page_bytes = a.page_size * a.pitch * 2;
     const int n_pages = (n_keys + a.page_size - 1) / a.page_size;
-    auto row_of = [&](int b) {  // rows past the last page read as zeros
-      const int pg = (b0 + b) * ppb + p;
-      return p < ppb && pg < n_pages ? bt[pg] * a.page_size : a.n_page_rows;
+    auto page_of = [&](int b) {
+      const int pg = (b0 + b) * ppb + lane;
+      return b < nb && lane < ppb && pg < n_pages ? bt[pg] : -1;
     };
-    int s = 0, next = row_of(0), next2 = nb > 1 ? row_of(1) : 0;
+    int s = 0, next = page_of(0), next2 = page_of(1);
     uint32_t par = 1;
     bool ok = true;
     for (int b = 0; b < nb && ok; ++b) {
-      const int row = next;
+      const int page = next;
       next = next2;
-      if (b + 2 < nb) next2 = row_of(b + 2);
-      for (int j = 0; j < a.n_chunks; ++j) {
-        if (lane == 0) {
-          ok = mbar_wait(&empty_bar[s], par, &s_abort);
-          if (ok) mbar_expect_tx(&full_bar[s], kSlot);
-        }
-        ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
-        if (!ok) break;
-        if (p < ppb)
-          tma_load_2d(ring + s * kSlot + half * kSubTile + p * a.page_size * 128, &map_c, j * 128 + half * 64, row, &full_bar[s]);
-        if (++s == a.n_slots) s = 0, par ^= 1;
+      next2 = page_of(b + 2);
+      const int valid = __popc(__ballot_sync(0xffffffffu, page >= 0));
+      if (lane == 0) {
+        ok = mbar_wait(&empty_bar[s], par, &s_abort);
+        if (ok) mbar_expect_tx(&full_bar[s], valid * page_bytes);
       }
+      ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
+      if (ok && page >= 0) bulk_load(ring + s * slot_bytes + lane * page_bytes, a.pages + (size_t)page * page_bytes, page_bytes, &full_bar[s]);
+      if (++s == a.n_slots) s = 0, par ^= 1;
     }
     if (!ok) s_abort = 1;
   } else if (warp == 1) {
     // ---- MMA issue -----------------------------------------------------------------------------------------------
-    if (lane == 0) {
+    if (elect_one()) {
       constexpr uint32_t idesc_s = make_idesc(128, kKeys), idesc_o = make_idesc(128, HG) | (1u << 15);  // O^T: A is MN-major
       bool ok = mbar_wait(&q_bar, 0, &s_abort);
       tc_fence_after();
+      const int group = 16 * a.pitch, slices = a.pitch / 64;  // bytes of 8 keys
+      // K-major operand (keys x 64 columns of a slice): row groups `group` bytes apart instead of adjacent
+      auto desc_k = [&](uint32_t addr) { return (make_smem_desc(addr) & ~((uint64_t)0x3FFF << 32)) | ((uint64_t)(group >> 4) << 32); };
       int s_s = 0, s_o = 0;  // ring positions of the two products
       uint32_t par = 0;
       auto scores = [&](int b) {
-        for (int j = 0; j < a.n_chunks; ++j) {
-          if (!mbar_wait(&full_bar[s_s], par, &s_abort)) return false;
-          tc_fence_after();
+        if (!mbar_wait(&full_bar[s_s], par, &s_abort)) return false;
+        tc_fence_after();
+        for (int j = 0; j < slices; ++j) {
+          const uint64_t bd = desc_k(smem_u32(ring + s_s * slot_bytes + j * 1024));
 #pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            const uint64_t bd = make_smem_desc(smem_u32(ring + s_s * kSlot + h * kSubTile));
-#pragma unroll
-            for (int k = 0; k < 4; ++k)
-              umma_bf16_ta(tmem_s + (b & 1) * kKeys, tmem_q + j * 64 + h * 32 + k * 8, bd + 2 * k, idesc_s, (j | h | k) ? 1u : 0u);
-          }
-          if (++s_s == a.n_slots) s_s = 0, par ^= 1;
+          for (int k = 0; k < 4; ++k)
+            umma_bf16_ta(tmem_s + (b & 1) * kKeys, tmem_q + j * 32 + k * 8, bd + 2 * k, idesc_s, (j | k) ? 1u : 0u);
         }
+        if (++s_s == a.n_slots) s_s = 0, par ^= 1;
         umma_commit(&s_bar[b & 1]);
         return true;
       };
@@ -212,16 +209,18 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __g
         ok = ok && mbar_wait(&p_bar[b & 1], (b >> 1) & 1, &s_abort);
         if (!ok) break;
         tc_fence_after();
+        const uint64_t pd = make_smem_desc(smem_u32(sp + (b & 1) * HG * 128));
         for (int j = 0; j < a.n_chunks; ++j) {
-          const uint32_t c = smem_u32(ring + s_o * kSlot);
+          // 128 of the rank = two slices, 1 KB apart.  (Where the rank ends in the first of them, the second reads the next
+          // row group's first slice: those sums are not stored.)
+          const uint32_t c = smem_u32(ring + s_o * slot_bytes + j * 2048);
 #pragma unroll
-          for (int k = 0; k < 4; ++k)  // 16 keys = 2048 bytes of a sub-tile
-            umma_bf16(tmem_o + j * 32, desc_mn(c + k * 2048, kSubTile, 1024),
-                      make_smem_desc(smem_u32(sp + (b & 1) * HG * 128)) + 2 * k, idesc_o, (b | k) ? 1u : 0u);
-          umma_commit(&empty_bar[s_o]);
-          if (++s_o == a.n_slots) s_o = 0;
+          for (int k = 0; k < 4; ++k)  // 16 keys = two row groups
+            umma_bf16(tmem_o + j * 32, desc_mn(c + k * 2 * group, 1024, group), pd + 2 * k, idesc_o, (b | k) ? 1u : 0u);
         }
+        umma_commit(&empty_bar[s_o]);
         umma_commit(&o_bar[b & 1]);
+        if (++s_o == a.n_slots) s_o = 0;
       }
       if (!ok) s_abort = 1;
     }
@@ -318,15 +317,12 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __g
           }
         }
         if (valid < kKeys) {
-          // latents of keys that do not exist (whatever the last page holds there): their probability is 0, but 0 * NaN is
-          // not.  The scores of this block have been computed, so all its slots have landed.
-          for (int j = 0; j < a.n_chunks; ++j) {
-            uint8_t* c = ring + ((b * a.n_chunks + j) % a.n_slots) * kSlot;
-            for (int i = valid * 8 + lane; i < kKeys * 8; i += 32) {
-              reinterpret_cast<uint4*>(c)[i] = make_uint4(0u, 0u, 0u, 0u);
-              reinterpret_cast<uint4*>(c + kSubTile)[i] = make_uint4(0u, 0u, 0u, 0u);
-            }
-          }
+          // latents of keys that do not exist (whatever the last page holds there, and pages that were not copied): their probability is 0, but 0 * NaN is
+          // not.  The scores of this block have been computed, so its pages have landed.
+          uint4* c = reinterpret_cast<uint4*>(ring + (b % a.n_slots) * slot_bytes);
+          const int per_group = a.pitch;  // 16-byte chunks of 8 keys: [slice][key][8]
+          for (int i = (valid >> 3) * per_group + lane; i < 8 * per_group; i += 32)
+            if (i >= ((valid + 7) >> 3) * per_group || ((i >> 3) & 7) >= (valid & 7)) c[i] = make_uint4(0u, 0u, 0u, 0u);
         }
         tc_fence_before();
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -362,9 +358,9 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(const __g
           if (i < heads) {
             const size_t row = out_row + i;
             if (a.n_splits == 1)
-              a.out[row * a.q_pitch + r] = __float2bfloat16_rn(o[i] * s_f[i]);
+              a.out[row * a.q_pitch + r] = __float2bfloat16_rn(r < a.R ? o[i] * s_f[i] : 0.f);
             else
-              a.part[(row * a.n_splits + split) * a.q_pitch + r] = o[i];
+              a.part[(row * a.n_splits + split) * a.q_pitch + r] = r < a.R ? o[i] : 0.f;
           }
         }
       }
@@ -428,8 +424,8 @@ int pick_splits(int T, int H, int max_keys) {
 }
 
 template <int HG>
-int launch_lt(const CUtensorMap& mc, const LtArgs& a, int T, cudaStream_t st) {
-  const int smem = a.n_slots * kSlot + 2 * HG * 128 + 1024;
+int launch_lt(const LtArgs& a, int T, cudaStream_t st) {
+  const int smem = a.n_slots * kKeys * a.pitch * 2 + 2 * HG * 128 + 1024;
   static std::atomic<unsigned long long> attr_done{0};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -438,7 +434,7 @@ int launch_lt(const CUtensorMap& mc, const LtArgs& a, int T, cudaStream_t st) {
     if (e != cudaSuccess) return fail(MLORA_ECUDA, "latent_attention: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
     attr_done.fetch_or(1ull << (dev & 63), std::memory_order_release);
   }
-  launch_pdl_if(pdl_enabled_attn(), latent_attn_tc_kernel<HG>, dim3(T, a.n_splits, (a.H + HG - 1) / HG), kLtThreads, smem, st, mc, a);
+  launch_pdl_if(pdl_enabled_attn(), latent_attn_tc_kernel<HG>, dim3(T, a.n_splits, (a.H + HG - 1) / HG), kLtThreads, smem, st, a);
   count_launch();
   MLORA_CHECK_LAUNCH("latent_attn_tc_kernel");
   return MLORA_OK;
@@ -463,10 +459,10 @@ extern "C" int mlora_latent_attention(const void* d_qa, int64_t q_pitch, const v
                                       const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, int32_t H, float scale,
                                       int32_t n_splits, void* d_out, void* d_work, size_t work_bytes, int32_t* d_status,
                                       void* stream) {
-  MLORA_REQUIRE(T >= 0 && H > 0 && R > 0 && R <= kMaxChunks * 128 && pitch >= R && pitch % 8 == 0 && max_pages > 0 && n_pages_total > 0,
-                "latent_attention: bad sizes (kv_rank up to %d, cache pitch a multiple of 8)", kMaxChunks * 128);
-  MLORA_REQUIRE(page_size == 16 || page_size == 32, "latent_attention: page size 16 or 32 (got %d)", page_size);
   const int n_chunks = (R + 127) / 128;
+  MLORA_REQUIRE(T >= 0 && H > 0 && R > 0 && R <= kMaxChunks * 128 && pitch >= R && pitch % 64 == 0 && pitch <= n_chunks * 128 && max_pages > 0 && n_pages_total > 0,
+                "latent_attention: bad sizes (kv_rank up to %d, cache pitch a multiple of 64)", kMaxChunks * 128);
+  MLORA_REQUIRE(page_size == 16 || page_size == 32, "latent_attention: page size 16 or 32 (got %d)", page_size);
   MLORA_REQUIRE(q_pitch == n_chunks * 128, "latent_attention: rows of qa and out have kv_rank rounded up to 128 columns (got %lld)", (long long)q_pitch);
   MLORA_REQUIRE(d_qa && d_pages && d_block_table && d_row_slot && d_row_pos && d_out && aligned16(d_qa) && aligned16(d_pages) &&
                     aligned16(d_out) && (int64_t)n_pages_total * page_size < 0x7fffffff && (int64_t)T * H < 0x7fffffff,
@@ -476,21 +472,20 @@ extern "C" int mlora_latent_attention(const void* d_qa, int64_t q_pitch, const v
   MLORA_REQUIRE(!need || (d_work && aligned16(d_work) && work_bytes >= need), "latent_attention: workspace of %zu bytes needed, %zu given", need, work_bytes);
   if (T == 0) return MLORA_OK;
   const int HG = head_group(H);
-  CUtensorMap mc;
-  int rc = make_map(&mc, d_pages, (long long)n_pages_total * page_size, pitch, pitch, page_size, 64);
-  if (rc) return rc;
   LtArgs a{};
   a.block_table = d_block_table;
   a.max_pages = max_pages;
   a.page_size = page_size;
-  a.n_page_rows = n_pages_total * page_size;
+  a.pages = (const uint8_t*)d_pages;
+  a.R = R;
+  a.pitch = pitch;
   a.row_slot = d_row_slot;
   a.row_pos = d_row_pos;
   a.qa = (const bf16*)d_qa;
   a.H = H;
   a.q_pitch = (int)q_pitch;
   a.n_chunks = n_chunks;
-  a.n_slots = (224 * 1024 - 2 * HG * 128 - 1024) / kSlot;
+  a.n_slots = (224 * 1024 - 2 * HG * 128 - 1024) / (kKeys * pitch * 2);
   if (a.n_slots > kMaxSlots) a.n_slots = kMaxSlots;
   a.n_splits = n_splits;
   a.scale_log2 = scale * kLog2e;
@@ -498,9 +493,9 @@ extern "C" int mlora_latent_attention(const void* d_qa, int64_t q_pitch, const v
   a.part = (float*)d_work;
   a.ml = (float2*)((float*)d_work + (size_t)T * H * n_splits * q_pitch);
   a.status = d_status;
-  rc = HG == 16 ? launch_lt<16>(mc, a, T, (cudaStream_t)stream) : launch_lt<32>(mc, a, T, (cudaStream_t)stream);
+  const int rc = HG == 16 ? launch_lt<16>(a, T, (cudaStream_t)stream) : launch_lt<32>(a, T, (cudaStream_t)stream);
   if (rc || n_splits == 1) return rc;
-  launch_pdl(latent_merge_kernel, (unsigned)(T * H), 128, 0, (cudaStream_t)stream, a.part, a.ml, n_splits, (int)q_pitch, (bf16*)d_out);
+  launch_pdl_if(pdl_enabled_norm(), latent_merge_kernel, (unsigned)(T * H), 128, 0, (cudaStream_t)stream, a.part, a.ml, n_splits, (int)q_pitch, (bf16*)d_out);
   count_launch();
   MLORA_CHECK_LAUNCH("latent_merge_kernel");
   return MLORA_OK;

@@ -302,8 +302,10 @@ __device__ __forceinline__ GroupTile group_tile(const TcParams& p, int tok_tile,
 template <bool WAVE>
 __device__ __forceinline__ int grouped_per_cta(const TcParams& p, int n_tiles) {
   const long long total = (long long)n_tiles * p.k_blocks;
-  const long long even = (total + gridDim.x - 1) / gridDim.x;
-  return (int)(even < 4 ? 4 : even);
+  // no split tiles where one tile per CTA fills most of the grid, and no CTA with less than four k-blocks (or a tile)
+  if (n_tiles <= (int)gridDim.x && 2 * n_tiles > (int)gridDim.x) return p.k_blocks;
+  const int even = (int)((total + gridDim.x - 1) / gridDim.x);
+  return max(even, min(4, p.k_blocks));
 }
 template <bool WAVE, bool GRP>
 __device__ __forceinline__ Range cta_range(const TcParams& p, int cta, int n_tiles, int per_cta) {

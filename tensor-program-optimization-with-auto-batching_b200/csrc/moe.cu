@@ -15,36 +15,50 @@ constexpr int kDecodeTokens = 64;    // one-launch form: tokens
 constexpr int kDecodePairs = 1024;   //                  and pairs
 constexpr int kLocalPairs = 4096;    // pairs of one CTA of the route kernel
 
-// One warp: experts and weights of one token.  Selected in order of decreasing logit, lower index first among equals.
-__device__ __forceinline__ void route_token(const float* __restrict__ z, const float* __restrict__ bias, int E, int top,
-                                            int32_t* __restrict__ idx, float* __restrict__ wt) {
+// One warp: experts and weights of one token, in order of decreasing logit, lower index first among equals.  `z(e)` is the
+// logit of expert e; lane l keeps those of experts l, l + 32, ... in R registers.
+template <int R, typename F>
+__device__ __forceinline__ void route_token(F z, int E, int top, int32_t* __restrict__ idx, float* __restrict__ wt) {
   const int lane = threadIdx.x & 31;
-  float last = INFINITY, z0 = 0.f, sum = 0.f;
-  int last_i = -1;
+  float v[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) v[r] = lane + 32 * r < E ? z(lane + 32 * r) : -INFINITY;
+  unsigned taken = 0;  // bit r: register r has been chosen (or does not exist)
+#pragma unroll
+  for (int r = 0; r < R; ++r)
+    if (lane + 32 * r >= E) taken |= 1u << r;
+  float z0 = 0.f, sum = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int bi = 0x7fffffff;
-    for (int e = lane; e < E; e += 32) {
-      const float v = z[e] + bias[e];
-      const bool after = v < last || (v == last && e > last_i);  // not chosen yet
-      if (after && (bi == 0x7fffffff || v > best)) best = v, bi = e;
-    }
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (!(taken >> r & 1) && (bi == 0x7fffffff || v[r] > best)) best = v[r], bi = lane + 32 * r;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ov = __shfl_xor_sync(0xffffffffu, best, o);
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (oi != 0x7fffffff && (bi == 0x7fffffff || ov > best || (ov == best && oi < bi))) best = ov, bi = oi;
     }
-    if (bi == 0x7fffffff) bi = k < E ? k : 0, best = -INFINITY;  // (only with NaN logits: stay in range)
+    bi = __shfl_sync(0xffffffffu, bi, 0);  // (one view of the choice, NaN logits included)
+    best = __shfl_sync(0xffffffffu, best, 0);
+    if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
     if (k == 0) z0 = best;
     const float w = expf(best - z0);
     sum += w;
     if (lane == 0) idx[k] = bi, wt[k] = w;
-    last = best;
-    last_i = bi;
   }
   __syncwarp();
   for (int k = lane; k < top; k += 32) wt[k] /= sum;
+}
+template <typename F>
+__device__ __forceinline__ void route_any(F z, int E, int top, int32_t* __restrict__ idx, float* __restrict__ wt) {
+  if (E <= 64)
+    route_token<2>(z, E, top, idx, wt);
+  else if (E <= 256)
+    route_token<8>(z, E, top, idx, wt);
+  else
+    route_token<32>(z, E, top, idx, wt);
 }
 
 struct PlanOut {
@@ -79,11 +93,13 @@ __device__ __forceinline__ void write_tiles(const int* s_cnt, const int* s_off, 
       reinterpret_cast<int4*>(tiles)[1 + i] = make_int4(e, s_off[e] + r, min(tile_rows, s_cnt[e] - r), 0);
 }
 
-// CTA = token.  z = W h + bias in fp32 (a warp takes every eighth expert), choice by warp 0; the last CTA groups.
+// CTA = token.  z = W h + bias in fp32 (two experts per warp at a time), choice by warp 0; the last CTA groups.
+constexpr int kDecodeThreads = 1024;
+
 template <typename A>
-__global__ void __launch_bounds__(256) moe_decode_kernel(const A* __restrict__ h, int64_t ldh, const A* __restrict__ W, int in,
-                                                         const float* __restrict__ bias, int T, int E, int top, int tile_rows,
-                                                         PlanOut o, int32_t* __restrict__ ticket) {
+__global__ void __launch_bounds__(kDecodeThreads, 1) moe_decode_kernel(const A* __restrict__ h, int64_t ldh, const A* __restrict__ W,
+                                                                       int in, const float* __restrict__ bias, int T, int E, int top,
+                                                                       int tile_rows, PlanOut o, int32_t* __restrict__ ticket) {
   __shared__ float s_z[kMoeMaxExperts];
   __shared__ int s_cnt[kMoeMaxExperts], s_off[kMoeMaxExperts], s_tile[kMoeMaxExperts];
   __shared__ int s_e[kDecodePairs];
@@ -92,29 +108,30 @@ __global__ void __launch_bounds__(256) moe_decode_kernel(const A* __restrict__ h
   pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, n = T * top;
   const A* x = h + (size_t)t * ldh;
-  for (int e0 = warp; e0 < E; e0 += 32) {  // four experts of the warp at a time
-    float acc[4] = {};
+  for (int e0 = warp * 2; e0 < E; e0 += kDecodeThreads / 16) {
+    const bool two = e0 + 1 < E;
+    const A* w0 = W + (size_t)e0 * in;
+    const A* w1 = two ? w0 + in : w0;
+    float a0 = 0.f, a1 = 0.f;
+#pragma unroll 4
     for (int k = lane * 8; k < in; k += 256) {
-      float xv[8], wv[8];
+      float xv[8], u[8], v[8];
       load8(x + k, xv);
+      load8(w0 + k, u);
+      load8(w1 + k, v);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        if (e0 + 8 * j < E) {
-          load8(W + (size_t)(e0 + 8 * j) * in + k, wv);
-#pragma unroll
-          for (int i = 0; i < 8; ++i) acc[j] = fmaf(xv[i], wv[i], acc[j]);
-        }
-      }
+      for (int i = 0; i < 8; ++i) a0 = fmaf(xv[i], u[i], a0), a1 = fmaf(xv[i], v[i], a1);
     }
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const float z = warp_sum(acc[j]);
-      if (lane == 0 && e0 + 8 * j < E) s_z[e0 + 8 * j] = z;
+    a0 = warp_sum(a0);
+    a1 = warp_sum(a1);
+    if (lane == 0) {
+      s_z[e0] = a0 + bias[e0];
+      if (two) s_z[e0 + 1] = a1 + bias[e0 + 1];
     }
   }
   __syncthreads();
   if (warp == 0) {
-    route_token(s_z, bias, E, top, o.idx + (size_t)t * top, o.wt + (size_t)t * top);
+    route_any([&](int e) { return s_z[e]; }, E, top, o.idx + (size_t)t * top, o.wt + (size_t)t * top);
     __threadfence();
     __syncwarp();
     if (lane == 0) s_last = atomicAdd(ticket, 1) == T - 1;
@@ -123,16 +140,16 @@ __global__ void __launch_bounds__(256) moe_decode_kernel(const A* __restrict__ h
   if (!s_last) return;
   if (tid == 0) *ticket = 0;  // ready for the next call
   __threadfence();
-  for (int i = tid; i < n; i += 256) s_e[i] = __ldcg(o.idx + i);
-  for (int e = tid; e < E; e += 256) s_cnt[e] = 0;
+  for (int i = tid; i < n; i += kDecodeThreads) s_e[i] = __ldcg(o.idx + i);
+  for (int e = tid; e < E; e += kDecodeThreads) s_cnt[e] = 0;
   __syncthreads();
-  for (int i = tid; i < n; i += 256) atomicAdd(&s_cnt[s_e[i]], 1);
+  for (int i = tid; i < n; i += kDecodeThreads) atomicAdd(&s_cnt[s_e[i]], 1);
   __syncthreads();
   if (warp == 0) scan_experts(s_cnt, s_off, s_tile, E, tile_rows, o.tiles);
   __syncthreads();
   write_tiles(s_cnt, s_off, s_tile, E, tile_rows, o.tiles);
   // row of pair i = first row of its expert + pairs of the same expert before it
-  for (int i = tid; i < n; i += 256) {
+  for (int i = tid; i < n; i += kDecodeThreads) {
     const int e = s_e[i];
     int before = 0;
 #pragma unroll 8
@@ -143,7 +160,7 @@ __global__ void __launch_bounds__(256) moe_decode_kernel(const A* __restrict__ h
   }
 }
 
-// Prompt passes.  CTA c: tokens [c * per, ...); hist[c * E + e] = its pairs of expert e; rank (in o.pos) = place of a pair
+// Prompt passes.  CTA c: tokens [c * per, ...); hist[e * CTAs + c] = its pairs of expert e; rank (in o.pos) = place of a pair
 // among the CTA's pairs of its expert.
 __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int64_t ld, const float* __restrict__ bias,
                                                         int T, int E, int top, int per, PlanOut o, int32_t* __restrict__ hist) {
@@ -152,7 +169,8 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict_
   pdl_wait();
   const int t0 = blockIdx.x * per, n = (min(T, t0 + per) - t0) * top, warp = threadIdx.x >> 5;
   for (int t = t0 + warp; t < min(T, t0 + per); t += 8) {
-    route_token(logits + (size_t)t * ld, bias, E, top, o.idx + (size_t)t * top, o.wt + (size_t)t * top);
+    const float* z = logits + (size_t)t * ld;
+    route_any([&](int e) { return z[e] + bias[e]; }, E, top, o.idx + (size_t)t * top, o.wt + (size_t)t * top);
     __syncwarp();
     for (int k = threadIdx.x & 31; k < top; k += 32) s_e[(t - t0) * top + k] = o.idx[(size_t)t * top + k];
   }
@@ -162,11 +180,11 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict_
 #pragma unroll 8
     for (int i = 0; i < n; ++i)
       if (s_e[i] == e) o.pos[(size_t)t0 * top + i] = c++;
-    hist[(size_t)blockIdx.x * E + e] = c;
+    hist[(size_t)e * gridDim.x + blockIdx.x] = c;
   }
 }
 
-// One CTA: hist[c][e] becomes the first row of CTA c's pairs of expert e; the tile table.
+// One CTA: hist[e][c] becomes the first row of CTA c's pairs of expert e; the tile table.
 __global__ void __launch_bounds__(1024) moe_scan_kernel(int32_t* __restrict__ hist, int n_cta, int E, int tile_rows, PlanOut o) {
   __shared__ int s_cnt[kMoeMaxExperts], s_off[kMoeMaxExperts], s_tile[kMoeMaxExperts];
   pdl_launch_dependents();
@@ -174,7 +192,7 @@ __global__ void __launch_bounds__(1024) moe_scan_kernel(int32_t* __restrict__ hi
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int e = warp; e < E; e += 32) {
     int total = 0;
-    for (int c = lane; c < n_cta; c += 32) total += hist[(size_t)c * E + e];
+    for (int c = lane; c < n_cta; c += 32) total += hist[(size_t)e * n_cta + c];
     total = __reduce_add_sync(0xffffffffu, total);
     if (lane == 0) s_cnt[e] = total;
   }
@@ -185,30 +203,31 @@ __global__ void __launch_bounds__(1024) moe_scan_kernel(int32_t* __restrict__ hi
   for (int e = warp; e < E; e += 32) {
     int run = s_off[e];
     for (int c0 = 0; c0 < n_cta; c0 += 32) {
-      const int c = c0 + lane, v = c < n_cta ? hist[(size_t)c * E + e] : 0;
+      const int c = c0 + lane, v = c < n_cta ? hist[(size_t)e * n_cta + c] : 0;
       int a = v;
 #pragma unroll
       for (int d = 1; d < 32; d <<= 1) {
         const int p = __shfl_up_sync(0xffffffffu, a, d);
         if (lane >= d) a += p;
       }
-      if (c < n_cta) hist[(size_t)c * E + e] = run + a - v;
+      if (c < n_cta) hist[(size_t)e * n_cta + c] = run + a - v;
       run += __shfl_sync(0xffffffffu, a, 31);
     }
   }
 }
 
-__global__ void __launch_bounds__(256) moe_scatter_kernel(const int32_t* __restrict__ first, int n, int E, int top, int per, PlanOut o) {
+__global__ void __launch_bounds__(256) moe_scatter_kernel(const int32_t* __restrict__ first, int n, int n_cta, int top, int per, PlanOut o) {
   pdl_launch_dependents();
   pdl_wait();
   const int i = blockIdx.x * 256 + threadIdx.x;
   if (i >= n) return;
-  const int t = i / top, p = first[(size_t)(t / per) * E + o.idx[i]] + o.pos[i];
+  const int t = i / top, p = first[(size_t)o.idx[i] * n_cta + t / per] + o.pos[i];
   o.pos[i] = p;
   o.rows[p] = t;
 }
 
-int tokens_per_cta(int top) { return kLocalPairs / top < 64 ? kLocalPairs / top : 64; }
+// (8 warps: a token or a few each)
+int tokens_per_cta(int top) { return kLocalPairs / top < 32 ? kLocalPairs / top : 32; }
 
 }  // namespace
 }  // namespace mlora
@@ -240,9 +259,9 @@ extern "C" int mlora_moe_plan(const float* d_logits, int64_t ld, const float* d_
   const PlanOut o{d_expert, d_weight, d_pos, d_rows, d_tiles};
   const int n = T * top, per = tokens_per_cta(top), n_cta = (T + per - 1) / per;
   int32_t* hist = (int32_t*)((uint8_t*)d_work + 256);
-  launch_pdl(moe_route_kernel, n_cta, 256, 0, st, d_logits, ld, d_bias, T, E, top, per, o, hist);
-  launch_pdl(moe_scan_kernel, 1, 1024, 0, st, hist, n_cta, E, tile_rows, o);
-  launch_pdl(moe_scatter_kernel, (n + 255) / 256, 256, 0, st, hist, n, E, top, per, o);
+  launch_pdl_if(pdl_enabled_norm(), moe_route_kernel, n_cta, 256, 0, st, d_logits, ld, d_bias, T, E, top, per, o, hist);
+  launch_pdl_if(pdl_enabled_norm(), moe_scan_kernel, 1, 1024, 0, st, hist, n_cta, E, tile_rows, o);
+  launch_pdl_if(pdl_enabled_norm(), moe_scatter_kernel, (n + 255) / 256, 256, 0, st, hist, n, n_cta, top, per, o);
   count_launch(3);
   MLORA_CHECK_LAUNCH("moe_plan");
   return MLORA_OK;
@@ -263,10 +282,10 @@ extern "C" int mlora_moe_route_plan(const void* d_h, int64_t ldh, const void* d_
   if (T == 0) return MLORA_OK;
   const PlanOut o{d_expert, d_weight, d_pos, d_rows, d_tiles};
   if (f32)
-    launch_pdl_if(pdl_enabled_norm(), moe_decode_kernel<float>, T, 256, 0, (cudaStream_t)stream, (const float*)d_h, ldh,
+    launch_pdl_if(pdl_enabled_norm(), moe_decode_kernel<float>, T, kDecodeThreads, 0, (cudaStream_t)stream, (const float*)d_h, ldh,
                   (const float*)d_W, in, d_bias, T, E, top, tile_rows, o, (int32_t*)d_work);
   else
-    launch_pdl_if(pdl_enabled_norm(), moe_decode_kernel<bf16>, T, 256, 0, (cudaStream_t)stream, (const bf16*)d_h, ldh,
+    launch_pdl_if(pdl_enabled_norm(), moe_decode_kernel<bf16>, T, kDecodeThreads, 0, (cudaStream_t)stream, (const bf16*)d_h, ldh,
                   (const bf16*)d_W, in, d_bias, T, E, top, tile_rows, o, (int32_t*)d_work);
   count_launch();
   MLORA_CHECK_LAUNCH("moe_decode_kernel");

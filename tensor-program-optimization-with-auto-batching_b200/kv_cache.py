@@ -161,15 +161,15 @@ class PagedKVCache(PagedCache):
 
 class PagedLatentCache(PagedCache):
     """One latent vector per token for every layer that computes latents: ``[n_pages, page_size, pitch]`` per such
-    layer.  Layers that attend to another layer's latents hold nothing and read that layer's pages.
+    layer, a page in the tiled order of ``csrc/latent.cuh`` (:meth:`untile`).  Layers that attend to another layer's latents hold nothing and read that layer's pages.
 
-    ``ranks``: layer -> kv_rank of the layers that own latents (the pitch is the rank rounded up to 8)."""
+    ``ranks``: layer -> kv_rank of the layers that own latents (the pitch is the rank rounded up to 64)."""
 
     def __init__(self, ranks, max_batch, max_total_seq_len, prefill_chunk_size, page_size, device, max_seq_len=None,
                  dtype=torch.bfloat16):
         super().__init__(max_batch, max_total_seq_len, prefill_chunk_size, page_size, device, max_seq_len)
         self.ranks = dict(ranks)
-        self.pages = {l: torch.zeros(self.n_pages, self.page_size, -(-r // 8) * 8, dtype=dtype, device=self.device)
+        self.pages = {l: torch.zeros(self.n_pages, self.page_size, -(-r // 64) * 64, dtype=dtype, device=self.device)
                       for l, r in self.ranks.items()}
 
     def latent_pages(self, layer):
@@ -177,7 +177,16 @@ class PagedLatentCache(PagedCache):
 
     def gather(self, sid, layer):
         """Latents of a sequence, dense [n, kv_rank]."""
-        return self._gather_pages(self.pages[layer], sid)[:, :self.ranks[layer]]
+        return self._gather_pages(self.untile(self.pages[layer]), sid)[:, :self.ranks[layer]]
+
+    @staticmethod
+    def untile(pages):
+        """Row-major copy of ``pages`` [n_pages, page_size, pitch] stored as [page_size / 8][pitch / 64][8][8 chunks][8]
+        with chunk c of row r at place c ^ r."""
+        n, ps, pitch = pages.shape
+        r = torch.arange(8, device=pages.device)
+        t = pages.reshape(n, ps // 8, pitch // 64, 8, 8, 8)[:, :, :, r[:, None], r[:, None] ^ r[None, :]]
+        return t.transpose(2, 3).reshape(n, ps, pitch)
 
 
 # The three global functions of the reference's runtime, same names and argument order.

@@ -161,7 +161,7 @@ class PackedTevudra:
         lw.expand = None
         if self.dtype == torch.bfloat16 and lw.dk <= 128 and lw.dv <= 128 and mix.scale > 0:
             ukv = torch.cat([uk.flatten(0, 1), uv.flatten(0, 1)])
-            lw.expand = self._weight(ukv, (ukv.shape[0], _up(mix.rank, 8)))
+            lw.expand = self._weight(ukv, (ukv.shape[0], _up(mix.rank, 64)))
         o = get(p + "o").reshape(self.width, mix.heads, mix.vdim)
         lw.w_o = self._weight(self._mat(o, (H, mix.heads, lw.dv)).flatten(1), (H, mix.heads * lw.dv))
         if ff is None:

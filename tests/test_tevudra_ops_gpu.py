@@ -154,12 +154,23 @@ def test_grouped_heads_with_gates(ops, cuda, dtype, T, H, k, n, tile):
 
 
 # ---------------------------------------------------------------- latents in pages
+def tile(pages):
+    """Row-major pages to the stored order, element by element from its definition."""
+    n, ps, pitch = pages.shape
+    row, k = torch.meshgrid(torch.arange(ps), torch.arange(pitch), indexing="ij")
+    chunk = ((k % 64) // 8) ^ (row % 8)
+    off = (row // 8) * 8 * pitch + (k // 64) * 512 + (row % 8) * 64 + chunk * 8 + k % 8
+    out = torch.empty(n, ps * pitch, dtype=pages.dtype)
+    out[:, off.flatten()] = pages.flatten(1)
+    return out.view(n, ps, pitch)
+
+
 class Pages:
     """Scrambled page table over sequences of the given lengths; every place no sequence uses holds NaN."""
 
     def __init__(self, lens, R, ps, dtype, dev, seed=0):
         g = gen(seed)
-        self.lens, self.R, self.ps, self.pitch = lens, R, ps, -(-R // 8) * 8
+        self.lens, self.R, self.ps, self.pitch = lens, R, ps, -(-R // 64) * 64
         need = [-(-n // ps) for n in lens]
         self.max_pages = max(need) + 2
         ids = torch.randperm(sum(need) + 3, generator=g).tolist()
@@ -177,23 +188,24 @@ class Pages:
             for j in range(len(c)):
                 row = self.pages[self.bt[s, j // self.ps], j % self.ps]
                 row[: self.R], row[self.R:] = c[j], 0
-        return self.pages.to(self.dev), self.bt.to(self.dev)
+        return tile(self.pages).to(self.dev), self.bt.to(self.dev)
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("R", [3, 30, 128, 264])
-def test_latent_append_and_gather(ops, cuda, dtype, R):
+@pytest.mark.parametrize("R,col", [(3, 5), (30, 5), (128, 8), (264, 16), (512, 0), (96, 8), (264, 3), (520, 8)])
+def test_latent_append_and_gather(ops, cuda, dtype, R, col):
     lens = [1, 16, 17, 40]
     pg = Pages(lens, R, 16, dtype, cuda)
     pages, bt = pg.pages.clone().to(cuda), pg.bt.to(cuda)
     slot = torch.tensor([s for s, n in enumerate(lens) for _ in range(n)] + [0], dtype=torch.int32)
     pos = torch.tensor([j for n in lens for j in range(n)] + [-1], dtype=torch.int32)  # the last row is padding
     perm = torch.randperm(len(slot), generator=gen(1))
-    x = torch.randn(len(slot), R + 5, generator=gen(2)).to(dtype)
+    x = torch.randn(len(slot), -(-(R + col) // 8) * 8, generator=gen(2)).to(dtype)
     w = torch.randn(R, generator=gen(3)).bfloat16()
-    ops.latent_append(x[perm].to(cuda)[:, 5:], R, w.to(cuda), 0.1, pages, bt, slot[perm].to(cuda), pos[perm].to(cuda))
-    want = ot.rms(x[:, 5:].double(), w.double(), 0.1)
-    got = pages.cpu()
+    ops.latent_append(x[perm].to(cuda)[:, col:], R, w.to(cuda), 0.1, pages, bt, slot[perm].to(cuda), pos[perm].to(cuda))
+    want = ot.rms(x[:, col:col + R].double(), w.double(), 0.1)
+    got = load("kv_cache").PagedLatentCache.untile(pages.cpu())
+    assert torch.equal(torch.nan_to_num(tile(got), nan=7.0), torch.nan_to_num(pages.cpu(), nan=7.0))
     used = torch.zeros(got.shape[:2], dtype=torch.bool)
     for i in range(len(slot) - 1):
         p, o = int(pg.bt[slot[i], pos[i] // 16]), int(pos[i]) % 16
