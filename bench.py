@@ -801,6 +801,8 @@ def run_kernel_case(which):
     T = N_REQ
     if which == "operator":
         return run_operator_case(ops, synth, dev, torch)
+    if which in ("latent", "experts"):
+        return run_tevudra_kernel_case(which, ops, dev, torch)
     if which == "linear":
         # the q/k/v projection of one layer with its LoRA stack: 4 weight copies = 403 MB
         c = synth.operator_case(T, 4096, 12288, N_ADAPTERS, RANK, device=dev)
@@ -1259,6 +1261,47 @@ def run_tevudra(args):
         emit(line)
 
 
+def run_tevudra_kernel_case(which, ops, dev, torch):
+    """latent: decode attention of 32 rows, 32 heads, rank 512 at 8192 keys each (268 MB of latents); experts: the up
+    projections of 64 experts, 192 (token, expert) pairs, 2048 -> 1408 (369 MB of weights).  A few launches, then CUDA-event
+    time."""
+    T, g = 32, torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *s: torch.randn(*s, generator=g, device=dev).to(torch.bfloat16)
+    i32 = dict(dtype=torch.int32, device=dev)
+    if which == "latent":
+        H, R, ctx = 32, 512, 8192
+        pages = rnd(T * ctx // PAGE, PAGE, R)
+        bt = torch.randperm(T * ctx // PAGE, device=dev, generator=g).to(torch.int32).view(T, -1)
+        qa, out, status = rnd(T, H * R) / 22, torch.empty(T, H * R, dtype=torch.bfloat16, device=dev), torch.zeros(1, **i32)
+        slot, pos = torch.arange(T, **i32), torch.full((T,), ctx - 1, **i32)
+        s = ops.latent_attention_splits(T, H, ctx)
+        work = ops.new_workspace(ops.latent_attention_workspace(T, H, R, s), dev)
+        fn = lambda: ops.latent_attention(qa, R, H, pages, bt, slot, pos, 128 ** -0.5, out, n_splits=s, work=work, status=status)
+        by = 2 * R * T * ctx + 4 * qa.numel()
+    else:
+        E, top, W, ff = 64, 6, 2048, 1408
+        x, y, plan = rnd(T, W), torch.empty(T * top, ff, dtype=torch.bfloat16, device=dev), ops.MoePlan(T, E, top, dev)
+        weight = ops.GroupedWeight(rnd(E, ff, W))
+        tr = ops.grouped_tile_rows(T * top / E)
+        ops.moe_route_plan(x, rnd(E, W), torch.zeros(E, device=dev), plan, tr)
+        work = ops.new_workspace(ops._lib.lib().mlora_grouped_linear_workspace(tr), dev)
+        fn = lambda: ops.grouped_linear(x, weight, y, plan=plan, gather=True, flags=ops.ACT_GELU, work=work)
+        used = len(set(plan.expert[:T * top].tolist()))
+        by = 2 * (used * W * ff + x.numel() + y.numel())
+    for _ in range(5):
+        fn()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for _ in range(10):
+        fn()
+    e1.record()
+    torch.cuda.synchronize()
+    us = 1e3 * e0.elapsed_time(e1) / 10
+    peak, src = measured_peak()
+    emit({"kernel_case": which, "us_per_launch": us, "algorithmic_bytes": by, "achieved_gbs": by / us / 1e3,
+          "frac_of_peak": by / us / 1e3 / peak, "peak_source": src, "launches": ops.launch_count()})
+
+
 _RESULT_FD = None
 
 
@@ -1290,7 +1333,8 @@ def main():
     ap.add_argument("--skip-prefill", action="store_true",
                     help="profiling aid: fill the KV cache with seeded random values instead of running prefill "
                          "(the number is then not a bench value)")
-    ap.add_argument("--kernel-case", default="", choices=["", "linear", "attention", "operator", "prefill", "prefill-lora", "prefill-attn", "expand", "chain"],
+    ap.add_argument("--kernel-case", default="", choices=["", "linear", "attention", "operator", "prefill", "prefill-lora", "prefill-attn", "expand", "chain",
+                                                               "latent", "experts"],
                     help="profiling aid: launch one kernel a few times on a small case (> L2, < 1 GB) and exit")
     ap.add_argument("--workload", default="", choices=["", "13b-shape", "13b-tp", "prefill-heavy", "tevudra"],
                     help="side measurements (own JSON line, not the benchmark's): 13b-shape = the 13B shape and adapter "

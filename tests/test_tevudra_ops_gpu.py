@@ -61,7 +61,7 @@ def test_residual_dyt(ops, cuda, dtype, T, H):
 
 
 # ---------------------------------------------------------------- routing
-@pytest.mark.parametrize("T,E,top,tile", [(1, 1, 1, 16), (1, 12, 2, 16), (5, 7, 7, 32), (32, 70, 6, 16), (2, 300, 8, 64),
+@pytest.mark.parametrize("T,E,top,tile", [(1, 1, 1, 16), (1, 11, 2, 16), (5, 7, 7, 32), (32, 70, 6, 16), (2, 300, 8, 64),
                                           (900, 5, 2, 256), (700, 64, 6, 128), (3000, 9, 1, 64), (1024, 2, 2, 16)])
 def test_moe_plan(ops, cuda, T, E, top, tile):
     g = gen(E * T)
@@ -74,7 +74,7 @@ def test_moe_plan(ops, cuda, T, E, top, tile):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("T,E,top,width", [(1, 1, 1, 8), (1, 12, 2, 40), (5, 7, 7, 320), (32, 70, 6, 264), (64, 300, 8, 1000), (64, 5, 3, 72)])
+@pytest.mark.parametrize("T,E,top,width", [(1, 1, 1, 8), (1, 11, 2, 40), (5, 7, 7, 320), (32, 70, 6, 264), (64, 300, 8, 1000), (64, 5, 3, 72)])
 def test_moe_route_plan_in_one_launch(ops, cuda, dtype, T, E, top, width):
     g = gen(E + T)
     # small integers: the logits are exact in fp32 whatever the order of the sum
