@@ -520,6 +520,76 @@ int mlora_latent_attention_simt(const void* d_qa, int64_t q_pitch, const void* d
                                 const int32_t* d_row_pos, int32_t T, int32_t H, float scale, void* d_out, int32_t f32,
                                 void* stream);
 
+/* ---- hyper-connections + layer norm ---------------------------------------------------------------------------
+ * The residual as n streams of H columns per row.  With delta (the result of the sublayer before): stream t becomes
+ * sum_s mix[s, t] stream_s + back[t] * delta, all of them from the old ones (d_back = back[n], then mix[n, n], [from, to]).
+ * Then u = sum_s read[s] stream_s and out = (u - mean) / sqrt(variance + eps) * w over the first `width` columns (the others
+ * are zero; w [H] bf16).  d_src: streams before, row r at d_src + r * ld_src, stream s src_stream further (0: all streams are
+ * the same row).  d_dst [T][n][H] (may be d_src with ld_src = n * H, src_stream = H; NULL: the new streams are not kept).
+ * d_rows: output row i is row d_rows[i] (then only those rows are updated).  delta and out are bf16, or fp32 with f32 != 0;
+ * streams and coefficients fp32.  n <= 16. */
+int mlora_residual_streams_layernorm(const void* d_delta, const float* d_src, int64_t ld_src, int64_t src_stream, float* d_dst,
+                                     const float* d_back, const float* d_read, const int32_t* d_rows, const void* d_w, float eps,
+                                     void* d_out, int32_t T, int32_t n, int32_t H, int32_t width, int32_t f32, void* stream);
+
+/* ---- attention with rotated, normalised keys that are their own values; chunks; sinks -----------------------------
+ * mlora_rotate_rms_append: x rows [q heads | k heads] of `dim` columns; x += bias; the first `rot` columns of a head rotated
+ *   by position * inv_freq[i] (column i paired with i + rot / 2), then the head divided by sqrt(mean(x^2) + eps).  Queries,
+ *   times q_scale, to d_q [T, Hq, pad]; keys to their place in d_k_pages, and x + bias as it was before to d_v_pages
+ *   (pages [page][Hkv][page_size][pad]; columns from dim to pad are zero; rows with row_pos < 0 store nothing).  dim <= 512.
+ * mlora_paged_attention_masked, mlora_prefill_attention_masked: mlora_paged_attention (fused_append = 0) and
+ *   mlora_prefill_attention with the scale of the scores as an argument (positive for the latter), `chunk` > 0: position i
+ *   sees the positions j <= i with j / chunk == i / chunk only, and d_sink [Hq] (NULL: none): exp(sink[h]) is added to the
+ *   sum of a head's softmax.  Prompt form: heads of 64 or 128, pages of a multiple of 16.
+ * mlora_paged_attention_any: the same for heads of up to 512, bf16 or fp32, on the CUDA cores, one query row per CTA. */
+int mlora_rotate_rms_append(const void* d_x, int64_t ld, const float* d_bias, const float* d_inv_freq, int32_t rot, int32_t dim,
+                            int32_t pad, float eps, float q_scale, void* d_q, void* d_k_pages, void* d_v_pages,
+                            const int32_t* d_block_table, int32_t max_pages, const int32_t* d_row_slot, const int32_t* d_row_pos,
+                            int32_t T, int32_t Hq, int32_t Hkv, int32_t page_size, int32_t f32, void* stream);
+int mlora_paged_attention_masked(const void* d_q, int64_t ld, const void* d_k_pages, const void* d_v_pages,
+                                 const int32_t* d_block_table, int32_t max_pages, const int32_t* d_row_slot,
+                                 const int32_t* d_row_pos, int32_t T, int32_t Hq, int32_t Hkv, int32_t D, int32_t page_size,
+                                 float scale, int32_t chunk, const float* d_sink, void* d_out, int64_t ld_out, int32_t n_splits,
+                                 void* d_work, size_t work_bytes, void* stream);
+int mlora_prefill_attention_masked(const void* d_q, int64_t ld, const void* d_k_pages, const void* d_v_pages,
+                                   int32_t n_pages_total, const int32_t* d_block_table, int32_t max_pages, const int32_t* d_tiles,
+                                   int32_t n_tiles, int32_t Hq, int32_t Hkv, int32_t D, int32_t page_size, float scale,
+                                   int32_t chunk, const float* d_sink, int32_t T, void* d_out, int64_t ld_out, int32_t* d_status,
+                                   void* stream);
+int mlora_paged_attention_any(const void* d_q, const void* d_k_pages, const void* d_v_pages, const int32_t* d_block_table,
+                              int32_t max_pages, const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, int32_t Hq,
+                              int32_t Hkv, int32_t D, int32_t page_size, float scale, int32_t chunk, const float* d_sink,
+                              void* d_out, int64_t ld_out, int32_t f32, void* stream);
+
+/* ---- gated delta rule -----------------------------------------------------------------------------------------------
+ * A state M [dim, vdim] (fp32) per head and sequence:  M' = c M + k w^T with w = step (v - c M^T k),  o = M'^T q.  k and q are
+ * divided by their length (1e-6 under the root), q then times q_scale; step = sigmoid(b); log c = -exp(A_log) softplus(a +
+ * dt_bias).  Before that q, k and v are silu(causal convolution of `taps` <= 8 tokens) of the projected rows' columns
+ * q [kv_heads, dim] | k [kv_heads, dim] | v [heads, vdim] (C columns, a multiple of 8); value head h uses q and k head
+ * h / (heads / kv_heads).  dim <= 256 and vdim multiples of 8 (pad with zero weights).
+ * State [slot][heads][dim][vdim]; ring [slot][taps][C]: the convolution's inputs, token p at place p % taps.  Neither is read
+ * for a sequence's position 0, so neither needs clearing.  Activations are bf16, or fp32 with f32 != 0.
+ * mlora_short_conv: convolution and silu of all rows of a pass (rows of one sequence are consecutive; w [taps][C] fp32, the
+ *   last row is the current token's).
+ * mlora_delta_scan: the recurrence over the rows of each segment int32 [n][4] = (slot, first row, rows, position of the first
+ *   row), one segment per sequence; xc from mlora_short_conv, x the projected rows with b and a from columns b_col and a_col.
+ *   Leaves state and ring after the segment's last row, and o [T, heads * vdim] fp32.
+ * mlora_gated_rms: out = o / sqrt(mean(o^2) + eps) * w * silu(gate) per head (mean over the first vdim_true columns).
+ * mlora_delta_step: everything for one new token per row (gate from column g_col); rows with row_pos < 0 give zeros. */
+int mlora_short_conv(const void* d_x, int64_t ld, int32_t C, int32_t taps, const float* d_w, const void* d_ring,
+                     const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, void* d_out, int32_t f32, void* stream);
+int mlora_delta_scan(const void* d_xc, const void* d_x, int64_t ld, int32_t C, int32_t taps, int32_t b_col, int32_t a_col,
+                     const float* d_A_log, const float* d_dt_bias, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim,
+                     float q_scale, const int32_t* d_segs, int32_t n_segs, float* d_state, void* d_ring, float* d_out, int32_t f32,
+                     void* stream);
+int mlora_gated_rms(const float* d_o, const void* d_gate, int64_t ld_gate, const float* d_w, int32_t T, int32_t heads, int32_t vdim,
+                    int32_t vdim_true, float eps, void* d_out, int32_t f32, void* stream);
+int mlora_delta_step(const void* d_x, int64_t ld, int32_t C, int32_t taps, int32_t g_col, int32_t b_col, int32_t a_col,
+                     const float* d_conv, const float* d_A_log, const float* d_dt_bias, const float* d_norm_w, float eps,
+                     int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t vdim_true, float q_scale,
+                     const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, float* d_state, void* d_ring, void* d_out,
+                     int32_t f32, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

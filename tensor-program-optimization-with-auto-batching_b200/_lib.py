@@ -94,6 +94,22 @@ PROTOTYPES = {
                                          _f32, _i32, _vp, _vp, _sz, _vp, _vp]),
     "mlora_latent_attention_simt": (C.c_int, [_vp, _i64, _vp, _i32, _i32, _i32, _vp, _i32, _vp, _vp, _i32, _i32,
                                               _f32, _vp, _i32, _vp]),
+    "mlora_residual_streams_layernorm": (C.c_int, [_vp, _vp, _i64, _i64, _vp, _vp, _vp, _vp, _vp, _f32, _vp, _i32, _i32, _i32,
+                                                   _i32, _i32, _vp]),
+    "mlora_rotate_rms_append": (C.c_int, [_vp, _i64, _vp, _vp, _i32, _i32, _i32, _f32, _f32, _vp, _vp, _vp, _vp, _i32, _vp,
+                                          _vp, _i32, _i32, _i32, _i32, _i32, _vp]),
+    "mlora_paged_attention_masked": (C.c_int, [_vp, _i64, _vp, _vp, _vp, _i32, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _f32,
+                                               _i32, _vp, _vp, _i64, _i32, _vp, _sz, _vp]),
+    "mlora_prefill_attention_masked": (C.c_int, [_vp, _i64, _vp, _vp, _i32, _vp, _i32, _vp, _i32, _i32, _i32, _i32, _i32,
+                                                 _f32, _i32, _vp, _i32, _vp, _i64, _vp, _vp]),
+    "mlora_paged_attention_any": (C.c_int, [_vp, _vp, _vp, _vp, _i32, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _f32, _i32, _vp,
+                                            _vp, _i64, _i32, _vp]),
+    "mlora_short_conv": (C.c_int, [_vp, _i64, _i32, _i32, _vp, _vp, _vp, _vp, _i32, _vp, _i32, _vp]),
+    "mlora_delta_scan": (C.c_int, [_vp, _vp, _i64, _i32, _i32, _i32, _i32, _vp, _vp, _i32, _i32, _i32, _i32, _f32, _vp, _i32,
+                                   _vp, _vp, _vp, _i32, _vp]),
+    "mlora_gated_rms": (C.c_int, [_vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _f32, _vp, _i32, _vp]),
+    "mlora_delta_step": (C.c_int, [_vp, _i64, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _f32, _i32, _i32, _i32, _i32,
+                                   _i32, _f32, _vp, _vp, _i32, _vp, _vp, _vp, _i32, _vp]),
     "mlora_decode_step_begin": (C.c_int, [_vp, _vp, _vp, _vp, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),
     "mlora_decode_step_end": (C.c_int, [_vp, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _vp, _vp]),
 }

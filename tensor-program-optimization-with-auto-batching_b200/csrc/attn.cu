@@ -33,6 +33,9 @@ struct AttnArgs {
   int64_t ld_out;
   int n_splits;
   float* work;
+  float qscale;        // of the scores, times log2(e)
+  int chunk;           // > 0: a row sees only positions of its own chunk of this many (counted from position 0)
+  const float* sink;   // [Hq] or NULL: a logit per head that only enters the softmax's sum
   // optional: the LoRA shrink of the projection that reads `out` (o_proj), computed in this kernel's tail
   const bf16* sh_A;            // [N, sh_r, Hq*D] or nullptr
   const int32_t* sh_slots;     // [T]
@@ -94,7 +97,7 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(AttnArgs a) {
   const int slot = a.row_slot[t], pos = a.row_pos[t];
   const int32_t* bt = a.block_table + (size_t)slot * a.max_pages;
   const bf16* row = a.qkv + (size_t)t * a.ld;
-  const float qscale = rsqrtf((float)D) * kLog2e;
+  const float qscale = a.qscale;
   const bool last_split = split == a.n_splits - 1;
   const bool has_new = a.fused && last_split;
   // A position beyond the row's block-table entries (a step issued without reserved pages) is never
@@ -144,11 +147,13 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(AttnArgs a) {
 #pragma unroll
   for (int e = 0; e < 8; ++e) qf[e] = sq[dl * 8 + e];
 
-  // tokens read from the pages: [0, n_tok)
+  // tokens read from the pages: [lo, n_tok)
   const int n_tok = min(max(a.fused ? pos : pos + 1, 0), a.max_pages * PS);
   const int n_pg = (n_tok + PS - 1) / PS;
-  const int per = (n_pg + a.n_splits - 1) / a.n_splits;
-  const int pg_begin = min(split * per, n_pg), pg_end = min(pg_begin + per, n_pg);
+  const int lo = (a.chunk > 0 && pos > 0) ? pos - pos % a.chunk : 0;
+  const int pg_lo = min(lo / PS, n_pg);
+  const int per = (n_pg - pg_lo + a.n_splits - 1) / a.n_splits;
+  const int pg_begin = min(pg_lo + split * per, n_pg), pg_end = min(pg_begin + per, n_pg);
 
   float m = -INFINITY, l = 0.f, acc[8];
 #pragma unroll
@@ -176,7 +181,8 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(AttnArgs a) {
       for (int e = 0; e < 8; ++e) d = fmaf(qf[e], kf[e], d);
 #pragma unroll
       for (int o = LPT / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-      const bool valid = pg * PS + it * TPW + g < n_tok;
+      const int key = pg * PS + it * TPW + g;
+      const bool valid = key < n_tok && key >= lo;
       s[it] = valid ? d : -INFINITY;
       mx = fmaxf(mx, s[it]);
     }
@@ -231,10 +237,13 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(AttnArgs a) {
   float o_val = 0.f;
   if (tid < D) {
     float M = has_new ? s_new : -INFINITY;
+    const float sink = (a.sink && last_split) ? a.sink[h] * kLog2e : -INFINITY;  // (of several splits, the last one counts it)
+    M = fmaxf(M, sink);
 #pragma unroll
     for (int w = 0; w < 4; ++w) M = fmaxf(M, wm[w]);
     float L = 0.f, O = 0.f;
     if (M != -INFINITY) {
+      if (sink != -INFINITY) L = exp2f(sink - M);
 #pragma unroll
       for (int w = 0; w < 4; ++w) {
         const float c = (wm[w] == -INFINITY) ? 0.f : exp2f(wm[w] - M);
@@ -430,12 +439,19 @@ struct ShrinkTail {
   int32_t* tickets = nullptr;
 };
 
+// What the scores are multiplied by, which keys a row sees, and the sinks (see mlora_paged_attention_masked).
+struct Softmax {
+  float scale;
+  int chunk = 0;
+  const float* sink = nullptr;
+};
+
 static int attention_impl(const void* d_qkv, int64_t ld, void* d_k_pages, void* d_v_pages,
                           const int32_t* d_block_table, int32_t max_pages, const int32_t* d_row_slot,
                           const int32_t* d_row_pos, int32_t T, int32_t Hq, int32_t Hkv, int32_t D,
                           int32_t page_size, float rope_theta, int32_t fused_append, void* d_out,
                           int64_t ld_out, int32_t n_splits, void* d_work, size_t work_bytes,
-                          void* stream, const ShrinkTail& sh) {
+                          void* stream, const ShrinkTail& sh, const Softmax& sm) {
   int rc = check_kv_common("paged_attention", T, Hq, Hkv, D, page_size);
   if (rc) return rc;
   MLORA_REQUIRE(d_qkv && d_k_pages && d_v_pages && d_block_table && d_row_slot && d_row_pos && d_out && max_pages > 0,
@@ -444,7 +460,7 @@ static int attention_impl(const void* d_qkv, int64_t ld, void* d_k_pages, void* 
   if (T == 0) return MLORA_OK;
   MLORA_REQUIRE(T <= 65535, "paged_attention: T=%d exceeds 65535 rows per call", T);
   if (n_splits <= 0) {
-    n_splits = pick_splits(T, Hq, max_pages);
+    n_splits = pick_splits(T, Hq, sm.chunk > 0 ? min(max_pages, sm.chunk / page_size + 1) : max_pages);
     while (n_splits > 1 && mlora_paged_attention_workspace(T, Hq, D, n_splits) > work_bytes) --n_splits;
   }
   MLORA_REQUIRE(n_splits <= 64, "paged_attention: n_splits=%d exceeds 64", n_splits);
@@ -455,7 +471,7 @@ static int attention_impl(const void* d_qkv, int64_t ld, void* d_k_pages, void* 
   }
   AttnArgs a{(const bf16*)d_qkv, ld, (bf16*)d_k_pages, (bf16*)d_v_pages, d_block_table, max_pages, d_row_slot,
              d_row_pos, T, Hq, Hkv, page_size, rope_theta, fused_append ? 1 : 0, (bf16*)d_out, ld_out, n_splits,
-             (float*)d_work, (const bf16*)sh.A, sh.slots, sh.n_adapters, sh.r, sh.u, sh.part, sh.tickets};
+             (float*)d_work, sm.scale * kLog2e, sm.chunk, sm.sink, (const bf16*)sh.A, sh.slots, sh.n_adapters, sh.r, sh.u, sh.part, sh.tickets};
   dim3 grid(Hq, T, n_splits);
   cudaStream_t st = (cudaStream_t)stream;
   if (D == 128 && page_size == 16)
@@ -483,7 +499,18 @@ extern "C" int mlora_paged_attention(const void* d_qkv, int64_t ld, void* d_k_pa
                                      void* stream) {
   return attention_impl(d_qkv, ld, d_k_pages, d_v_pages, d_block_table, max_pages, d_row_slot, d_row_pos, T, Hq, Hkv, D,
                         page_size, rope_theta, fused_append, d_out, ld_out, n_splits, d_work, work_bytes, stream,
-                        ShrinkTail{});
+                        ShrinkTail{}, Softmax{1.f / sqrtf((float)(D > 0 ? D : 1))});
+}
+
+extern "C" int mlora_paged_attention_masked(const void* d_q, int64_t ld, const void* d_k_pages, const void* d_v_pages,
+                                            const int32_t* d_block_table, int32_t max_pages, const int32_t* d_row_slot,
+                                            const int32_t* d_row_pos, int32_t T, int32_t Hq, int32_t Hkv, int32_t D,
+                                            int32_t page_size, float scale, int32_t chunk, const float* d_sink, void* d_out,
+                                            int64_t ld_out, int32_t n_splits, void* d_work, size_t work_bytes, void* stream) {
+  MLORA_REQUIRE(chunk >= 0, "paged_attention_masked: bad chunk (%d)", chunk);
+  return attention_impl(d_q, ld, (void*)d_k_pages, (void*)d_v_pages, d_block_table, max_pages, d_row_slot, d_row_pos, T, Hq,
+                        Hkv, D, page_size, 1.f, 0, d_out, ld_out, n_splits, d_work, work_bytes, stream, ShrinkTail{},
+                        Softmax{scale, chunk, d_sink});
 }
 
 extern "C" uint32_t mlora_paged_attention_splits(int32_t T, int32_t Hq, int32_t max_pages) {
@@ -524,7 +551,7 @@ extern "C" int mlora_paged_attention_shrink(const void* d_qkv, int64_t ld, void*
   sh.tickets = (int32_t*)d_shrink_work;
   sh.part = (float*)((uint8_t*)d_shrink_work + (((size_t)T * sizeof(int32_t) + 255) & ~(size_t)255));
   return attention_impl(d_qkv, ld, d_k_pages, d_v_pages, d_block_table, max_pages, d_row_slot, d_row_pos, T, Hq, Hkv, D,
-                        page_size, rope_theta, fused_append, d_out, ld_out, 1, nullptr, 0, stream, sh);
+                        page_size, rope_theta, fused_append, d_out, ld_out, 1, nullptr, 0, stream, sh, Softmax{1.f / sqrtf((float)(D > 0 ? D : 1))});
 }
 
 // ---- allocation-free variant -------------------------------------------------------------------------

@@ -25,8 +25,7 @@
 namespace mlora {
 namespace {
 
-constexpr int kD = 128;            // head dimension of the paged form
-constexpr int kPS = 16;            // page size
+constexpr int kPS = 16;            // keys per copy of the paged form: a page, or a part of one
 constexpr int kTile = 128;         // query rows per CTA = keys per block
 constexpr int kPfThreads = 160;    // warps 0..3: one thread per query row; warp 4: TMA + MMA issue
 constexpr int kSub = kTile * 64 * 2;  // one [128 x 64] bf16 sub-tile: 16 KB
@@ -63,10 +62,13 @@ struct PfArgs {
   const bf16* gate; // dense form: a head's result of row t is multiplied by sigmoid(gate[t * ld_gate + head]); NULL: no gate
   int64_t ld_gate;
   int v_col;        // dense form: column of head 0's values in a row of keys and values
+  int page_parts;   // paged form: page size in 16s
+  int chunk;        // > 0: a row sees only positions of its own chunk of this many (counted from position 0)
+  const float* sink;  // [Hq] or NULL: a logit per head that only enters the softmax's sum
 };
 
-// NK, NV: query/key and value size of a head in 64s.  PAGED: keys and values of 128-wide heads come page by page through
-// the block table; else they are consecutive rows [key][head 0's key, head 1's key, ..., head 0's value, ...], one TMA
+// NK, NV: query/key and value size of a head in 64s.  PAGED: keys and values come 16 at a time through the block table,
+// from the first page of the chunk that the tile's first row lies in; else they are consecutive rows [key][head 0's key, head 1's key, ..., head 0's value, ...], one TMA
 // box per 128 keys.
 template <int NK, int NV, bool PAGED>
 __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_q,
@@ -88,8 +90,11 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
   const int slot = a.tiles[tile * 4 + 0], row0 = a.tiles[tile * 4 + 1], rows = a.tiles[tile * 4 + 2], pos0 = a.tiles[tile * 4 + 3];
   const int32_t* bt = PAGED ? a.block_table + (size_t)slot * a.max_pages : nullptr;
   constexpr int kDv = NV * 64;
+  const int chunk = a.chunk > 0 ? a.chunk : 0x7fffffff;
+  const int key0 = PAGED ? (pos0 - pos0 % chunk) / kPS * kPS : 0;  // first key that is read
+  const int lo_last = pos0 + rows - 1 - (pos0 + rows - 1) % chunk;  // first key the last row sees
   const int n_keys = pos0 + rows;                       // keys any row of the tile may see
-  const int n_blocks = (n_keys + kTile - 1) / kTile;
+  const int n_blocks = (n_keys - key0 + kTile - 1) / kTile;
   const int n_pages = (n_keys + kPS - 1) / kPS;
 
   if (tid == 0) {
@@ -114,26 +119,31 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
   float o_reg[kDv];
 #pragma unroll
   for (int i = 0; i < kDv; ++i) o_reg[i] = 0.f;
-  float m_run = -INFINITY, l_run = 0.f;
   const int q_pos = pos0 + tid;  // position of this thread's query row
+  const int q_lo = q_pos - q_pos % chunk;  // first key it sees
   const float scale = a.scale * kLog2e;
+  float m_run = a.sink ? a.sink[h] * kLog2e : -INFINITY, l_run = a.sink ? 1.f : 0.f;
   bool ok = true;
 
   // Block-table entries are read one block ahead (lane p of warp 4 keeps page p of the block's eight), so that no block
   // starts with a dependent chain of two global round trips.
-  auto page_of = [&](int pg) { return pg < n_pages ? bt[pg] : -1; };
-  int page_next = (PAGED && warp == 4 && lane < kTile / kPS) ? page_of(lane) : -1;
+  // (row of the first of 16 keys in the pages seen as rows; a missing entry reads as rows before 0: zeros)
+  auto page_of = [&](int pg) {
+    return pg < n_pages ? ((bt[pg / a.page_parts] * a.Hkv + kvh) * a.page_parts + pg % a.page_parts) * kPS : -kPS;
+  };
+  int page_next = (PAGED && warp == 4 && lane < kTile / kPS) ? page_of(key0 / kPS + lane) : -kPS;
 
   for (int kb = 0; kb < n_blocks; ++kb) {
     const uint32_t par = kb & 1;
-    const int page0 = kb * (kTile / kPS);
+    const int kstart = key0 + kb * kTile;  // first key of the block
+    const int page0 = kstart / kPS;
     const int page_cur = page_next;
     const int valid = min(kTile / kPS, n_pages - page0);
     if (PAGED && kb + 1 < n_blocks && warp == 4 && lane < kTile / kPS) page_next = page_of(page0 + kTile / kPS + lane);
     // ---- loads: K and V pages (and Q once) by TMA -----------------------------------------------------------------------------
     if (warp == 4) {
       if (lane == 0) {
-        mbar_expect_tx(&kbar, (PAGED ? (uint32_t)valid * 4 * (kPS * 128) : (uint32_t)(NK + NV) * kSub) + (kb == 0 ? NK * kSub : 0));
+        mbar_expect_tx(&kbar, (PAGED ? (uint32_t)valid * (NK + NV) * (kPS * 128) : (uint32_t)(NK + NV) * kSub) + (kb == 0 ? NK * kSub : 0));
         if (kb == 0) {
 #pragma unroll
           for (int j = 0; j < NK; ++j) tma_load_2d(sq + j * kSub, &map_q, h * NK * 64 + j * 64, row0, &kbar);
@@ -147,19 +157,18 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
         }
       }
       __syncwarp();
-      if (PAGED && lane < valid) {  // one page per lane, both 64-column halves of K and of V (a missing table entry reads as rows before 0: zeros)
-        const int r = (page_cur * a.Hkv + kvh) * kPS;
-        tma_load_2d(sk + lane * (kPS * 128), &map_k, 0, r, &kbar);
-        tma_load_2d(sk + kSub + lane * (kPS * 128), &map_k, 64, r, &kbar);
-        tma_load_2d(sv + lane * (kPS * 128), &map_v, 0, r, &kbar);
-        tma_load_2d(sv + kSub + lane * (kPS * 128), &map_v, 64, r, &kbar);
+      if (PAGED && lane < valid) {  // 16 keys per lane, every 64-column part of K and of V
+#pragma unroll
+        for (int j = 0; j < NK; ++j) tma_load_2d(sk + j * kSub + lane * (kPS * 128), &map_k, j * 64, page_cur, &kbar);
+#pragma unroll
+        for (int j = 0; j < NV; ++j) tma_load_2d(sv + j * kSub + lane * (kPS * 128), &map_v, j * 64, page_cur, &kbar);
       }
-    } else if (n_keys - kb * kTile < kTile) {
+    } else if (n_keys - kstart < kTile) {
       // Last block, not full: the V rows of keys that do not exist (the tail of the last page, whatever the cache holds
       // there, and the pages that were not loaded) are zeroed once the copies have landed -- their probabilities are 0,
       // but 0 * NaN is not.  K needs nothing: those scores are masked.  (A swizzled row stays inside its own 128 bytes.)
       if (!mbar_wait(&kbar, par, &s_abort)) s_abort = 1;
-      if (tid >= n_keys - kb * kTile) {
+      if (tid >= n_keys - kstart) {
 #pragma unroll
         for (int half = 0; half < NV; ++half)
 #pragma unroll
@@ -188,9 +197,9 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
       if (!mbar_wait(&sbar, par, &s_abort)) s_abort = 1;
       tc_fence_after();
       const uint32_t t_addr = tmem_base + ((uint32_t)(warp * 32) << 16);
-      // Only the blocks on or past the diagonal need the causal / length mask (uniform per CTA): every row of the
-      // tile sees every key of the blocks before.
-      const bool need_mask = kb * kTile + kTile - 1 > pos0;
+      // Only the blocks on or past the diagonal need the causal / length mask, and those before the last row's chunk the
+      // chunk's (uniform per CTA): every row of the tile sees every key of the blocks between.
+      const bool need_mask = kstart + kTile - 1 > pos0 || kstart < lo_last;
       // pass 1: row maximum over the valid keys (of the raw scores: the scale is positive)
       float mx = -INFINITY;
 #pragma unroll 1
@@ -203,8 +212,8 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
-            const int key = kb * kTile + c0 + i;
-            if (key <= q_pos && key < n_keys) mx = fmaxf(mx, s[i]);
+            const int key = kstart + c0 + i;
+            if (key <= q_pos && key >= q_lo && key < n_keys) mx = fmaxf(mx, s[i]);
           }
         }
       }
@@ -229,8 +238,8 @@ __global__ void __launch_bounds__(kPfThreads, 2) prefill_attn_tc_kernel(const __
           } else {
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
-              const int key = kb * kTile + c0 + g * 8 + i;
-              const bool valid = key <= q_pos && key < n_keys;
+              const int key = kstart + c0 + g * 8 + i;
+              const bool valid = key <= q_pos && key >= q_lo && key < n_keys;
               p[i] = valid ? fast_exp2(fmaf(s[g * 8 + i], scale, neg_m)) : 0.f;
               lsum += p[i];
             }
@@ -334,29 +343,44 @@ int launch_prefill(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorM
 
 using namespace mlora;
 
-extern "C" int mlora_prefill_attention(const void* d_qkv, int64_t ld, const void* d_k_pages, const void* d_v_pages,
-                                       int32_t n_pages_total, const int32_t* d_block_table, int32_t max_pages,
-                                       const int32_t* d_tiles, int32_t n_tiles, int32_t Hq, int32_t Hkv, int32_t D,
-                                       int32_t page_size, int32_t T, void* d_out, int64_t ld_out, int32_t* d_status,
-                                       void* stream) {
-  MLORA_REQUIRE(D == kD && page_size == kPS, "prefill_attention: head_dim 128 and page size 16 only (got %d, %d)", D, page_size);
+extern "C" int mlora_prefill_attention_masked(const void* d_q, int64_t ld, const void* d_k_pages, const void* d_v_pages,
+                                              int32_t n_pages_total, const int32_t* d_block_table, int32_t max_pages,
+                                              const int32_t* d_tiles, int32_t n_tiles, int32_t Hq, int32_t Hkv, int32_t D,
+                                              int32_t page_size, float scale, int32_t chunk, const float* d_sink, int32_t T,
+                                              void* d_out, int64_t ld_out, int32_t* d_status, void* stream) {
+  MLORA_REQUIRE((D == 64 || D == 128) && page_size > 0 && page_size % kPS == 0,
+                "prefill_attention: head_dim 64 or 128 and pages of a multiple of 16 only (got %d, %d)", D, page_size);
+  MLORA_REQUIRE(scale > 0.f && chunk >= 0, "prefill_attention: the scale must be positive, the chunk not negative");
   MLORA_REQUIRE(n_tiles >= 0 && T >= 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0 && n_pages_total > 0 && max_pages > 0,
                 "prefill_attention: bad sizes");
-  MLORA_REQUIRE(d_qkv && d_k_pages && d_v_pages && d_block_table && d_tiles && d_out, "prefill_attention: null pointer");
-  MLORA_REQUIRE(aligned16(d_qkv) && aligned16(d_k_pages) && aligned16(d_v_pages) && aligned16(d_out) && (ld * 2) % 16 == 0 &&
+  MLORA_REQUIRE(d_q && d_k_pages && d_v_pages && d_block_table && d_tiles && d_out, "prefill_attention: null pointer");
+  MLORA_REQUIRE(aligned16(d_q) && aligned16(d_k_pages) && aligned16(d_v_pages) && aligned16(d_out) && (ld * 2) % 16 == 0 &&
                     (ld_out * 2) % 16 == 0,
                 "prefill_attention: 16-byte alignment of tensors and row pitches");
   MLORA_REQUIRE(n_tiles <= 2147483647 / 4 && Hq <= 65535, "prefill_attention: too many tiles / heads");
   if (n_tiles == 0 || T == 0) return MLORA_OK;
   CUtensorMap mq, mk, mv;
-  int rc = make_map(&mq, d_qkv, T, Hq * kD, ld, kTile, 64);  // only the q part of every row is mapped
+  int rc = make_map(&mq, d_q, T, Hq * D, ld, kTile, 64);  // only the q part of every row is mapped
   if (rc) return rc;
-  rc = make_map(&mk, d_k_pages, (long long)n_pages_total * Hkv * kPS, kD, kD, kPS, 64);
+  rc = make_map(&mk, d_k_pages, (long long)n_pages_total * Hkv * page_size, D, D, kPS, 64);
   if (rc) return rc;
-  rc = make_map(&mv, d_v_pages, (long long)n_pages_total * Hkv * kPS, kD, kD, kPS, 64);
+  rc = make_map(&mv, d_v_pages, (long long)n_pages_total * Hkv * page_size, D, D, kPS, 64);
   if (rc) return rc;
-  PfArgs a{d_block_table, max_pages, d_tiles, Hq, Hkv, (bf16*)d_out, ld_out, d_status, 1.f / sqrtf((float)kD), nullptr, 0, 0};
-  return launch_prefill<2, 2, true>(mq, mk, mv, a, n_tiles, (cudaStream_t)stream);
+  PfArgs a{d_block_table, max_pages, d_tiles, Hq, Hkv, (bf16*)d_out, ld_out, d_status, scale, nullptr, 0, 0,
+           page_size / kPS, chunk, d_sink};
+  return D == 64 ? launch_prefill<1, 1, true>(mq, mk, mv, a, n_tiles, (cudaStream_t)stream)
+                 : launch_prefill<2, 2, true>(mq, mk, mv, a, n_tiles, (cudaStream_t)stream);
+}
+
+extern "C" int mlora_prefill_attention(const void* d_qkv, int64_t ld, const void* d_k_pages, const void* d_v_pages,
+                                       int32_t n_pages_total, const int32_t* d_block_table, int32_t max_pages,
+                                       const int32_t* d_tiles, int32_t n_tiles, int32_t Hq, int32_t Hkv, int32_t D,
+                                       int32_t page_size, int32_t T, void* d_out, int64_t ld_out, int32_t* d_status,
+                                       void* stream) {
+  MLORA_REQUIRE(D == 128 && page_size == kPS, "prefill_attention: head_dim 128 and page size 16 only (got %d, %d)", D, page_size);
+  return mlora_prefill_attention_masked(d_qkv, ld, d_k_pages, d_v_pages, n_pages_total, d_block_table, max_pages, d_tiles, n_tiles,
+                                        Hq, Hkv, D, page_size, 1.f / sqrtf((float)D), 0, nullptr, T, d_out, ld_out, d_status,
+                                        stream);
 }
 
 extern "C" int mlora_prefill_attention_dense(const void* d_q, int64_t ld, const void* d_kv, int64_t ld_kv, int32_t kv_rows,
@@ -377,7 +401,7 @@ extern "C" int mlora_prefill_attention_dense(const void* d_q, int64_t ld, const 
   if (rc) return rc;
   rc = make_map(&mkv, d_kv, kv_rows, v_col + H * Dv, ld_kv, kTile, 64);
   if (rc) return rc;
-  PfArgs a{nullptr, 0, d_tiles, H, H, (bf16*)d_out, ld_out, d_status, scale, (const bf16*)d_gate, ld_gate, v_col};
+  PfArgs a{nullptr, 0, d_tiles, H, H, (bf16*)d_out, ld_out, d_status, scale, (const bf16*)d_gate, ld_gate, v_col, 1, 0, nullptr};
   cudaStream_t st = (cudaStream_t)stream;
   if (Dk == 64 && Dv == 64) return launch_prefill<1, 1, false>(mq, mkv, mkv, a, n_tiles, st);
   if (Dk == 64) return launch_prefill<1, 2, false>(mq, mkv, mkv, a, n_tiles, st);

@@ -166,7 +166,7 @@ class EngineBase:
         self.n_distinct = len({int(s) for s in adapter_slots if s >= 0})
         self.max_keys = max(kv.tokens_reserved(s) for s in seq_ids)
         torch.cuda.synchronize()
-        saved = kv.seq_lens.clone()
+        saved, undo = kv.seq_lens.clone(), kv.snapshot(seq_ids)
 
         def step():
             ops.kv_begin_decode(self.row_slot[:B], kv.seq_lens, self.row_pos[:B])
@@ -183,9 +183,45 @@ class EngineBase:
         g = torch.cuda.CUDAGraph()
         with torch.cuda.graph(g):
             step()
-        kv.seq_lens.copy_(saved)  # warm-up advanced the device lengths; capture itself runs nothing
+        kv.seq_lens.copy_(saved)  # warm-up advanced the device lengths (and states); capture itself runs nothing
+        undo()
         torch.cuda.synchronize()
         return DecodeGraph(self, g, list(seq_ids), B)
+
+
+class PlainEngine(EngineBase):
+    """What the designs without adapters share: projections in the model's precision, buffers grown on demand, the status word
+    of kernels with bounded waits.  ``linears``: (in, out) of every projection of a pass."""
+
+    def __init__(self, model, kv: PagedCache, max_rows: int, linears, work_bytes: int = 0):
+        super().__init__(model, kv, max_rows)
+        lib, T = ops._lib.lib(), self.max_rows
+        # (some projections have more rows than the pass: scratch no longer grows beyond 128)
+        need = max([work_bytes] + [lib.mlora_linear_workspace(max(T, 128), k, n) for k, n in linears])
+        self.ws_linear = ops.new_workspace(need, model.device)
+        self.status = torch.zeros(1, dtype=torch.int32, device=model.device)
+        self._buf, self._retired = {}, []
+
+    # -- buffers that only some passes need, grown on demand (never while a graph is being captured: its warm-up run
+    # -- has the same sizes); outgrown ones stay alive for the graphs that hold their addresses -------------------
+    def _grow(self, name, numel, dtype=None):
+        t = self._buf.get(name)
+        if t is None or t.numel() < numel:
+            if t is not None:
+                self._retired.append(t)
+            t = self._buf[name] = torch.zeros(numel, dtype=dtype or self.m.dtype, device=self.m.device)
+        return t[:numel]
+
+    def check_status(self):
+        super().check_status()
+        if int(self.status.item()):
+            self.status.zero_()
+            raise RuntimeError("mlora: an attention kernel gave up a bounded wait; this pass's results are undefined")
+
+    def _linear(self, x, W, out, flags=0):
+        if self.m.dtype == torch.float32:  # (OUT_F32: what it writes anyway)
+            return ops.linear_f32(x, W, flags & ~ops.OUT_F32, out=out)
+        return ops.linear(x, W, flags=flags, out=out, work=self.ws_linear)
 
 
 class DecodeGraph:
@@ -259,7 +295,7 @@ class DecodeSession:
             return g
         e = self.eng
         state = (self.live, self.last_tok, self.gen_count, self.out_tokens, e.kv.seq_lens, self.n_live)
-        saved = [t.clone() for t in state]
+        saved, undo = [t.clone() for t in state], e.kv.snapshot(self.seq_ids)
         side = torch.cuda.Stream()
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):
@@ -271,6 +307,7 @@ class DecodeSession:
             self._step(rows)
         for t, s in zip(state, saved):
             t.copy_(s)
+        undo()
         torch.cuda.synchronize()
         self._graphs[rows] = g
         return g

@@ -127,6 +127,11 @@ class PagedCache:
         for sid in seq_ids:
             self._len_host[self._slot_of[int(sid)]] += n_steps
 
+    def snapshot(self, seq_ids):
+        """Whatever a step of these sequences changes and running it again would not put right (pages are simply written
+        again): a function that puts it back."""
+        return lambda: None
+
     # -- checks used by tests ---------------------------------------------------------------------
     def _gather_pages(self, pages, sid):
         """The first ``length(sid)`` rows of a sequence out of ``pages`` [n_pages, page_size, ...]."""
@@ -187,6 +192,44 @@ class PagedLatentCache(PagedCache):
         r = torch.arange(8, device=pages.device)
         t = pages.reshape(n, ps // 8, pitch // 64, 8, 8, 8)[:, :, :, r[:, None], r[:, None] ^ r[None, :]]
         return t.transpose(2, 3).reshape(n, ps, pitch)
+
+
+class HybridCache(PagedCache):
+    """Layers that keep keys and values per token (pages) beside layers that keep a state of fixed size per sequence.
+
+    ``attention``: entry -> (kv heads, head size as stored); ``states``: entry -> {name: (shape of one sequence, dtype)}, stored
+    as [max_batch, *shape] by the sequence's slot.  An entry is one run of a layer: a layer that runs several times has as many.
+    A state is not cleared when a slot changes hands: whoever reads it takes position 0 as a start from zero."""
+
+    def __init__(self, attention, states, max_batch, max_total_seq_len, prefill_chunk_size, page_size, device, max_seq_len=None,
+                 dtype=torch.bfloat16):
+        super().__init__(max_batch, max_total_seq_len, prefill_chunk_size, page_size, device, max_seq_len)
+        self.pages = {e: torch.zeros(2, self.n_pages, h, self.page_size, d, dtype=dtype, device=self.device)
+                      for e, (h, d) in attention.items()}
+        self.states = {e: {name: torch.zeros(self.max_batch, *shape, dtype=dt, device=self.device)
+                           for name, (shape, dt) in entry.items()} for e, entry in states.items()}
+
+    def k_pages(self, entry):
+        return self.pages[entry][0]
+
+    def v_pages(self, entry):
+        return self.pages[entry][1]
+
+    def state(self, entry, name):
+        return self.states[entry][name]
+
+    def gather(self, sid, entry):
+        """(K, V) of a sequence as dense [n, kv heads, head size] tensors."""
+        return [self._gather_pages(p.transpose(1, 2), sid) for p in self.pages[entry]]
+
+    def snapshot(self, seq_ids):
+        slots = torch.tensor([self._slot_of[int(s)] for s in seq_ids], dtype=torch.int64, device=self.device)
+        saved = [(t, t.index_select(0, slots)) for entry in self.states.values() for t in entry.values()]
+
+        def restore():
+            for t, old in saved:
+                t.index_copy_(0, slots, old)
+        return restore
 
 
 # The three global functions of the reference's runtime, same names and argument order.

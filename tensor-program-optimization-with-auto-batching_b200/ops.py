@@ -659,3 +659,122 @@ def latent_attention(qa, R, H, pages, block_table, row_slot, row_pos, scale, out
         block_table.shape[1], _ptr(row_slot), _ptr(row_pos), T, H, scale, n_splits, _ptr(out), _ptr(work),
         work.numel() if work is not None else 0, _ptr(status), _stream()), "mlora_latent_attention")
     return out
+
+
+# ---------------------------------------------------------------- hyper-connections + layer norm
+def residual_streams_layernorm(delta, src, read, w, eps, width, out, dst=None, back=None, rows=None):
+    """``src``: the streams [T, n, H], or the one row [T, H] they all are.  Mixes ``delta`` in with ``back`` (kept in ``dst`` when
+    given) and normalises the sum weighted by ``read`` into ``out``; see ``mlora_residual_streams_layernorm``."""
+    _need_cuda(src, out)
+    H = src.shape[-1]
+    check(_lib.lib().mlora_residual_streams_layernorm(
+        _ptr(delta), _ptr(src), src.stride(0), H if src.dim() == 3 else 0, _ptr(dst), _ptr(back), _ptr(read), _ptr(rows), _ptr(w),
+        eps, _ptr(out), out.shape[0], read.numel(), H, width, int(out.dtype == torch.float32), _stream()),
+        "mlora_residual_streams_layernorm")
+    return out
+
+
+# ---------------------------------------------------------------- rotated and normalised queries and keys; chunks; sinks
+def rotate_rms_append(x, bias, inv_freq, rot, dim, eps, q_scale, q_out, k_pages, v_pages, block_table, row_slot, row_pos, Hq, Hkv):
+    _need_cuda(x, k_pages)
+    check(_lib.lib().mlora_rotate_rms_append(
+        _ptr(x), x.stride(0), _ptr(bias), _ptr(inv_freq), rot, dim, k_pages.shape[3], eps, q_scale, _ptr(q_out), _ptr(k_pages),
+        _ptr(v_pages), _ptr(block_table), block_table.shape[1], _ptr(row_slot), _ptr(row_pos), x.shape[0], Hq, Hkv,
+        k_pages.shape[2], int(x.dtype == torch.float32), _stream()), "mlora_rotate_rms_append")
+    return q_out
+
+
+def paged_attention_masked(q, k_pages, v_pages, block_table, row_slot, row_pos, Hq, scale, out, chunk=0, sink=None, n_splits=0,
+                           work=None):
+    """One query row per (row, head); bf16 heads of 64 and 128 stream whole pages, everything else runs the plain kernel."""
+    _need_cuda(q, k_pages)
+    T, (Hkv, ps, D) = q.shape[0], k_pages.shape[1:]
+    if q.dtype == torch.float32 or D not in (64, 128) or ps not in (16, 32):
+        check(_lib.lib().mlora_paged_attention_any(
+            _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], _ptr(row_slot), _ptr(row_pos), T, Hq, Hkv,
+            D, ps, scale, chunk, _ptr(sink), _ptr(out), out.stride(0), int(q.dtype == torch.float32), _stream()),
+            "mlora_paged_attention_any")
+        return out
+    check(_lib.lib().mlora_paged_attention_masked(
+        _ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], _ptr(row_slot), _ptr(row_pos),
+        T, Hq, Hkv, D, ps, scale, chunk, _ptr(sink), _ptr(out), out.stride(0), n_splits, _ptr(work),
+        work.numel() if work is not None else 0, _stream()), "mlora_paged_attention_masked")
+    return out
+
+
+def paged_attention_splits(T, Hq, max_pages) -> int:
+    return int(_lib.lib().mlora_paged_attention_splits(T, Hq, max_pages))
+
+
+def paged_attention_workspace(T, Hq, D, n_splits) -> int:
+    return int(_lib.lib().mlora_paged_attention_workspace(T, Hq, D, n_splits))
+
+
+def prefill_attention_masked(q, k_pages, v_pages, block_table, tiles, n_tiles, Hq, scale, out, chunk=0, sink=None, status=None):
+    _need_cuda(q, k_pages)
+    Hkv, ps, D = k_pages.shape[1:]
+    check(_lib.lib().mlora_prefill_attention_masked(
+        _ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], _ptr(block_table), block_table.shape[1], _ptr(tiles),
+        n_tiles, Hq, Hkv, D, ps, scale, chunk, _ptr(sink), q.shape[0], _ptr(out), out.stride(0), _ptr(status), _stream()),
+        "mlora_prefill_attention_masked")
+    return out
+
+
+# ---------------------------------------------------------------- gated delta rule
+@dataclass
+class DeltaRule:
+    """Sizes (as stored: multiples of 8), column layout of a projected row, and the small fp32 tensors of one layer."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    vdim_true: int
+    taps: int
+    q_scale: float
+    g_col: int
+    b_col: int
+    a_col: int
+    conv: torch.Tensor     # [taps, channels]
+    A_log: torch.Tensor    # [heads]
+    dt_bias: torch.Tensor  # [heads]
+    norm: torch.Tensor     # [vdim]
+
+    @property
+    def channels(self):
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+
+def short_conv(x, w, ring, row_slot, row_pos, out):
+    """``x`` [T, >= C] -> silu of its causal convolution; ``w`` [taps, C] fp32, ``ring`` [slots, taps, C]."""
+    _need_cuda(x, w)
+    taps, C_ = w.shape
+    check(_lib.lib().mlora_short_conv(_ptr(x), x.stride(0), C_, taps, _ptr(w), _ptr(ring), _ptr(row_slot), _ptr(row_pos),
+                                      x.shape[0], _ptr(out), int(x.dtype == torch.float32), _stream()), "mlora_short_conv")
+    return out
+
+
+def delta_scan(xc, x, r: DeltaRule, segs, n_segs, state, ring, out):
+    _need_cuda(xc, state)
+    check(_lib.lib().mlora_delta_scan(
+        _ptr(xc), _ptr(x), x.stride(0), r.channels, r.taps, r.b_col, r.a_col, _ptr(r.A_log), _ptr(r.dt_bias), r.heads, r.kv_heads,
+        r.dim, r.vdim, r.q_scale, _ptr(segs), n_segs, _ptr(state), _ptr(ring), _ptr(out), int(x.dtype == torch.float32), _stream()),
+        "mlora_delta_scan")
+    return out
+
+
+def gated_rms(o, gate, w, heads, vdim_true, eps, out):
+    """o [T, heads * vdim] fp32, gate [T, >= heads * vdim] (a column slice is fine)."""
+    _need_cuda(o, gate)
+    T, cols = o.shape
+    check(_lib.lib().mlora_gated_rms(_ptr(o), _ptr(gate), gate.stride(0), _ptr(w), T, heads, cols // heads, vdim_true, eps, _ptr(out),
+                                     int(out.dtype == torch.float32), _stream()), "mlora_gated_rms")
+    return out
+
+
+def delta_step(x, r: DeltaRule, eps, row_slot, row_pos, state, ring, out):
+    _need_cuda(x, state)
+    check(_lib.lib().mlora_delta_step(
+        _ptr(x), x.stride(0), r.channels, r.taps, r.g_col, r.b_col, r.a_col, _ptr(r.conv), _ptr(r.A_log), _ptr(r.dt_bias), _ptr(r.norm),
+        eps, r.heads, r.kv_heads, r.dim, r.vdim, r.vdim_true, r.q_scale, _ptr(row_slot), _ptr(row_pos), x.shape[0], _ptr(state),
+        _ptr(ring), _ptr(out), int(x.dtype == torch.float32), _stream()), "mlora_delta_step")
+    return out

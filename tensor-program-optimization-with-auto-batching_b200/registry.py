@@ -12,6 +12,7 @@ import torch
 
 from . import checkpoint
 from .model import PackedLlama
+from .relidra import PackedRelidra
 from .tevudra import PackedTevudra
 
 
@@ -31,9 +32,14 @@ def _pack_tevudra(cfg, weights, adapters, scales, device, dtype):
     return PackedTevudra(cfg, weights, device=device, dtype=dtype)
 
 
+def _pack_relidra(cfg, weights, adapters, scales, device, dtype):
+    return PackedRelidra(cfg, weights, device=device, dtype=dtype)
+
+
 DESIGNS = {d.name: d for d in (
     Design("LlamaForCausalLM", _pack_llama, (torch.bfloat16,), True),
     Design("Tevudra", _pack_tevudra, PackedTevudra.dtypes, False),
+    Design("Relidra", _pack_relidra, PackedRelidra.dtypes, False),
 )}
 
 

@@ -21,13 +21,10 @@ import numpy as np
 import torch
 
 from . import ops
-from .engine import EngineBase
+from .engine import PlainEngine
 from .kv_cache import PagedLatentCache
 from .ops import ACT_GELU, ACT_RELU2, OUT_F32
-
-
-def _up(n, m):
-    return -(-n // m) * m
+from .packing import PackedDesign, up as _up
 
 
 def _head_pad(d):
@@ -105,35 +102,19 @@ class _Layer:
     """Packed weights of one layer."""
 
 
-class PackedTevudra:
+class PackedTevudra(PackedDesign):
     """Device-resident weights.  ``weights``: tensors under the checkpoint's names (``embed``, ``l<i>.mix.q``, ...)."""
 
-    dtypes = (torch.bfloat16, torch.float32)
+    name = "Tevudra"
 
     def __init__(self, cfg, weights, device="cuda", dtype=torch.bfloat16):
-        if dtype not in self.dtypes:
-            raise ValueError(f"Tevudra runs in bfloat16 or float32, not {dtype}")
         self.config = c = TevudraConfig.parse(cfg)
-        self.cfg, self.dtype, self.device = dict(cfg), dtype, torch.device(device)
-        self.V, self.L, self.width = c.vocab, len(c.layers), c.width
-        self.H = _up(c.width, 8)                       # pitch of residual and normalised rows
-        self.tp_size, self.n_adapters = 1, 0           # (no adapters on this design)
+        super().__init__(cfg, c.vocab, c.width, len(c.layers), device, dtype)
         get = lambda n: weights[n]
         self.embed = self._mat(get("embed"), (c.vocab, self.H), torch.bfloat16)
         self.norm = _Norm(get, "final.norm", self.H, self.device)
         self.head = self._weight(get("head"), (c.vocab, self.H))
         self.layers = [self._layer(i, mix, ff, get) for i, (mix, ff) in enumerate(c.layers)]
-
-    # -- packing ------------------------------------------------------------------------------------------------
-    def _mat(self, t, shape, dtype=None):
-        """``t`` in the corner of a zero matrix of ``shape``, on the device."""
-        out = torch.zeros(shape, dtype=dtype or self.dtype, device=self.device)
-        out[tuple(slice(0, n) for n in t.shape)] = t.to(self.device).to(out.dtype)
-        return out
-
-    def _weight(self, t, shape):
-        W = self._mat(t, shape)
-        return ops.PackedWeight(W) if self.dtype == torch.bfloat16 else W
 
     def _layer(self, i, mix, ff, get):
         lw, H, dev = _Layer(), self.H, self.device
@@ -183,9 +164,6 @@ class PackedTevudra:
             lw.s_up, lw.s_down = self._weight(get(p + "shared.up"), (lw.sffp, H)), self._weight(get(p + "shared.down"), (H, lw.sffp))
         return lw
 
-    def add_adapter(self, *_):
-        raise ValueError("the Tevudra design has no adapters")
-
     # -- what the model is served with ----------------------------------------------------------------------------
     def new_cache(self, max_batch, max_total_seq_len, prefill_chunk, page_size=16, max_seq_len=None):
         ranks = {i: lw.mix.rank for i, lw in enumerate(self.layers) if lw.mix.source == i}
@@ -196,14 +174,21 @@ class PackedTevudra:
         return TevudraEngine(self, kv, max_rows)
 
 
-class TevudraEngine(EngineBase):
+class TevudraEngine(PlainEngine):
     # a prompt pass expands keys and values of at most this many context rows; beyond, its rows attend in latent space
     MAX_EXPANDED_ROWS = 1 << 18
     # cost of an operation in latent space (row by row) against one of the tiled prompt attention
     LATENT_COST = 3.0
 
     def __init__(self, model: PackedTevudra, kv: PagedLatentCache, max_rows: int):
-        super().__init__(model, kv, max_rows)
+        shapes = [(model.H, model.V)]
+        for lw in model.layers:
+            shapes += [(model.H, lw.in_cols), (lw.mix.heads * lw.dv, model.H)]
+            if isinstance(lw.ff, Dense):
+                shapes += [(model.H, lw.ffp), (lw.ffp, model.H)]
+            elif lw.ff is not None:
+                shapes += [(model.H, lw.sffp), (lw.sffp, model.H)] if lw.ff.shared_ff else []
+        super().__init__(model, kv, max_rows, shapes, ops._lib.lib().mlora_grouped_linear_workspace(64))
         m, dev, T = model, model.device, self.max_rows
         act = dict(dtype=m.dtype, device=dev)
         lws, moes = m.layers, [lw for lw in m.layers if isinstance(lw.ff, MoE)]
@@ -225,33 +210,10 @@ class TevudraEngine(EngineBase):
             self.router_out = torch.zeros(T * widest(lambda lw: lw.ff.experts, moes), dtype=torch.float32, device=dev)
             self.e_act = torch.zeros(widest(lambda lw: pairs(lw) * lw.ffp, moes), **act)
             self.e_out = torch.zeros(widest(lambda lw: pairs(lw) * m.H, moes), **act)
-        lib = ops._lib.lib()
-        shapes = [(m.H, m.V)]
-        for lw in lws:
-            shapes += [(m.H, lw.in_cols), (lw.mix.heads * lw.dv, m.H)]
-            if isinstance(lw.ff, Dense):
-                shapes += [(m.H, lw.ffp), (lw.ffp, m.H)]
-            elif lw.ff is not None:
-                shapes += [(m.H, lw.sffp), (lw.sffp, m.H)] if lw.ff.shared_ff else []
-        # (the expansion of a context may have more rows than the pass: scratch no longer grows beyond 128)
-        need = max([lib.mlora_linear_workspace(max(T, 128), k, n) for k, n in shapes] + [lib.mlora_grouped_linear_workspace(64)])
-        self.ws_linear = ops.new_workspace(need, dev)
-        self.status = torch.zeros(1, dtype=torch.int32, device=dev)
         # prompt passes: query tiles of <= 128 rows, context segments (whole pages) of the expanded keys and values
         self.tiles = torch.zeros((T + 127) // 128 + kv.max_batch + 1, 4, dtype=torch.int32, device=dev)
         self.segs = torch.zeros(kv.max_batch, 4, dtype=torch.int32, device=dev)
         self._n_tiles = self._n_segs = self._ctx_rows = self._max_ctx = 0
-        self._buf, self._retired = {}, []
-
-    # -- buffers that only some passes need, grown on demand (never while a graph is being captured: its warm-up run
-    # -- has the same sizes); outgrown ones stay alive for the graphs that hold their addresses -------------------
-    def _grow(self, name, numel, dtype=None):
-        t = self._buf.get(name)
-        if t is None or t.numel() < numel:
-            if t is not None:
-                self._retired.append(t)
-            t = self._buf[name] = torch.zeros(numel, dtype=dtype or self.m.dtype, device=self.m.device)
-        return t[:numel]
 
     # -- prompt passes ------------------------------------------------------------------------------------------
     def _begin_prompt_pass(self, chunk):
@@ -284,18 +246,7 @@ class TevudraEngine(EngineBase):
     def _end_prompt_pass(self):
         self._n_tiles = 0
 
-    def check_status(self):
-        super().check_status()
-        if int(self.status.item()):
-            self.status.zero_()
-            raise RuntimeError("mlora: an attention kernel gave up a bounded wait; this pass's results are undefined")
-
     # -- pieces of a layer ----------------------------------------------------------------------------------------
-    def _linear(self, x, W, out, flags=0):
-        if self.m.dtype == torch.float32:  # (OUT_F32: what it writes anyway)
-            return ops.linear_f32(x, W, flags & ~OUT_F32, out=out)
-        return ops.linear(x, W, flags=flags, out=out, work=self.ws_linear)
-
     def _grouped(self, x, W, out, flags=0, **kw):
         if self.m.dtype == torch.float32:
             flags &= ~OUT_F32

@@ -178,7 +178,13 @@ class B200VM:
             # the reference keeps only the last token before lm_head (llama_for_causal_lm.py:130-137)
             last = (torch.arange(B, device=m.device, dtype=torch.int32) + 1) * S - 1
             eng.last_rows[:B].copy_(last)
+            passes, r = [], 0  # what the rows are: (sequence, first row, rows, position of the first row)
+            for sid, n in zip(*kv._pending):
+                passes.append((sid, r, n, kv.length(sid)))
+                r += n
+            eng._begin_prompt_pass(passes)
             logits, _ = eng.forward(T, False, use_lora, eng.last_rows, B, hidden=h2)
+            eng._end_prompt_pass()
         else:
             logits, _ = eng.forward(T, True, use_lora, hidden=h2)
         return NDArray(logits.clone().view(B, 1, m.V)), kv
