@@ -1071,7 +1071,8 @@ class KernelTimer:
 
     NAMES = ("linear", "grouped_linear", "moe_plan", "moe_route_plan", "residual_dyt", "residual_rmsnorm", "latent_append", "latent_gather",
              "latent_attention", "prefill_attention_dense", "embed", "argmax", "paged_attention", "prefill_attention",
-             "kv_append_rope")
+             "kv_append_rope", "paged_attention_masked", "prefill_attention_masked", "residual_streams_layernorm", "rotate_rms_append",
+             "short_conv", "delta_scan", "gated_rms", "delta_step")
 
     def __init__(self, ops, torch, dev, hbm_gbs, tflops):
         self.ops, self.torch, self.hbm, self.tflops = ops, torch, hbm_gbs, tflops
@@ -1110,6 +1111,27 @@ class KernelTimer:
         if name in ("paged_attention", "prefill_attention"):
             Hq, Hkv, D = (a[6], a[7], a[8]) if name == "paged_attention" else (a[6], a[7], a[8])
             return f"{sum(news)} rows, {Hq} heads", 4 * D * Hkv * sum(lens) + 4 * D * Hq * sum(news), 4.0 * Hq * D * pairs
+        if name in ("paged_attention_masked", "prefill_attention_masked"):  # (bench shapes: one chunk)
+            Hq, (Hkv, _, D) = a[6], a[1].shape[1:]
+            return f"{sum(news)} rows, {Hq} heads", 4 * D * Hkv * sum(lens) + 4 * D * Hq * sum(news), 4.0 * Hq * D * pairs
+        if name == "residual_streams_layernorm":
+            T, H, n = a[6].shape[0], a[6].shape[1], a[2].numel()
+            src = n if a[1].dim() == 3 else 1
+            return (f"{T} x {H}, {n} streams" + (" (read only)" if k.get("dst") is None else " (from the embedding)" if src < n else ""),
+                    T * H * (4 * src + 2 + (2 if a[0] is not None else 0) + (4 * n if k.get("dst") is not None else 0)), 0.0)
+        if name == "rotate_rms_append":
+            return f"{a[0].shape[0]} rows", 2 * a[0].shape[0] * (a[0].shape[1] + a[7].shape[1] + 2 * a[14] * a[8].shape[3]), 0.0
+        if name == "short_conv":
+            return f"{a[5].shape[0]} rows x {a[5].shape[1]}", 4 * a[5].numel(), 0.0
+        if name == "delta_scan":
+            r, o = a[2], a[7]
+            return (f"{o.shape[0]} rows, {r.heads} heads, {len(news)} sequences",
+                    2 * a[0].numel() + 4 * o.numel() + 8 * len(news) * r.heads * r.dim * r.vdim, 0.0)
+        if name == "gated_rms":
+            return f"{a[0].shape[0]} rows", 8 * a[0].numel(), 0.0
+        if name == "delta_step":
+            r, T = a[1], a[0].shape[0]
+            return f"{T} rows, {r.heads} heads", T * (8 * r.heads * r.dim * r.vdim + 2 * (r.taps + 1) * r.channels + 4 * r.heads * r.vdim), 0.0
         if name == "latent_append":
             return f"{a[0].shape[0]} rows", 4 * a[0].shape[0] * a[1], 0.0
         if name == "latent_gather":
@@ -1167,8 +1189,8 @@ class KernelTimer:
         return call
 
 
-def run_tevudra(args):
-    """Side measurement (its own JSON line): Tevudra at layer shapes of real models, random weights, beside the framework's
+def run_design(args, design):
+    """Side measurement (its own JSON line): a design at layer shapes of real models, random weights, beside the framework's
     Llama path (no adapters) at equal width, heads and head size.  Prefill of 16 x 512 and 2 x 4096 tokens, decode steps (CUDA
     graph) of 32 requests at contexts of 1024 and 8192; then every kernel of one pass by itself against its roofline."""
     import numpy as np
@@ -1182,18 +1204,22 @@ def run_tevudra(args):
     peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))) if src == "measured" else {}
     tflops = float(peaks.get("bf16_tflops", 1590.0))
     lines = []
-    for name in args.shapes.split(","):
-        tcfg = synth.tevudra_config(name)
-        W, heads = tcfg["width"], tcfg["layers"][0]["mixer"]["heads"]
-        lcfg = dict(synth.llama_config("llama2-7b"), hidden_size=W, num_attention_heads=heads, num_key_value_heads=heads,
+    make_config, make_weights = {"tevudra": (synth.tevudra_config, synth.tevudra_weights),
+                                 "relidra": (synth.relidra_config, synth.relidra_weights)}[design]
+    for name in (args.shapes or f"{design}-2048,{design}-4096").split(","):
+        tcfg = make_config(name)
+        mixer = tcfg["layers"][-1]["mixer"]
+        W, heads = tcfg["width"], mixer["heads"]
+        lcfg = dict(synth.llama_config("llama2-7b"), hidden_size=W, num_attention_heads=heads,
+                    num_key_value_heads=mixer.get("kv_heads", heads),
                     intermediate_size={2048: 5504, 4096: 11008}[W], num_hidden_layers=4, name=f"llama-{W}")
-        for design, cfg in (("tevudra", tcfg), ("llama", lcfg)):
-            w = (synth.tevudra_weights if design == "tevudra" else synth.base_weights)(cfg, dtype=torch.bfloat16, device=dev)
+        for make, cfg in ((make_weights, tcfg), (synth.base_weights, lcfg)):
+            w = make(cfg, dtype=torch.bfloat16, device=dev)
             model = reg.build_model(cfg, w, device=dev)
             del w
             torch.cuda.empty_cache()
             V = cfg.get("vocab", cfg.get("vocab_size"))
-            line = {"workload": "tevudra", "model": cfg["name"], "layers": 4, "peak_source": src, "dtype": "bf16", "data": "synthetic",
+            line = {"workload": design, "model": cfg["name"], "layers": 4, "peak_source": src, "dtype": "bf16", "data": "synthetic",
                     "prefill": [], "decode": [], "kernels": {}}
             timer = KernelTimer(ops, torch, dev, hbm, tflops)
             for n_req, length in ((16, 512), (2, 4096)):
@@ -1336,13 +1362,13 @@ def main():
     ap.add_argument("--kernel-case", default="", choices=["", "linear", "attention", "operator", "prefill", "prefill-lora", "prefill-attn", "expand", "chain",
                                                                "latent", "experts"],
                     help="profiling aid: launch one kernel a few times on a small case (> L2, < 1 GB) and exit")
-    ap.add_argument("--workload", default="", choices=["", "13b-shape", "13b-tp", "prefill-heavy", "tevudra"],
+    ap.add_argument("--workload", default="", choices=["", "13b-shape", "13b-tp", "prefill-heavy", "tevudra", "relidra"],
                     help="side measurements (own JSON line, not the benchmark's): 13b-shape = the 13B shape and adapter "
                          "mix on one GPU; 13b-tp = the tensor-parallel configuration, tp size = number of ranks "
                          "(launch with torch.distributed.run); prefill-heavy = 64 x 512-token prompts, 64 rank-64 adapters on "
-                         "seven projections, Zipf ids, 16 decode tokens; tevudra = the Tevudra design beside the Llama path at "
+                         "seven projections, Zipf ids, 16 decode tokens; tevudra, relidra = that design beside the Llama path at "
                          "equal layer sizes, prefill, decode and every kernel against its roofline")
-    ap.add_argument("--shapes", default="tevudra-2048,tevudra-4096", help="tevudra workload: shapes to run")
+    ap.add_argument("--shapes", default="", help="tevudra and relidra workloads: shapes to run (default: both of the design's)")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
@@ -1359,8 +1385,8 @@ def main():
         run_13b_tp(args, rank, world, local_rank)
     elif args.workload == "prefill-heavy":
         run_prefill_heavy(args)
-    elif args.workload == "tevudra":
-        run_tevudra(args)
+    elif args.workload in ("tevudra", "relidra"):
+        run_design(args, args.workload)
     elif args.kernel_case:
         run_kernel_case(args.kernel_case)
     elif args.impl == "reference":

@@ -26,59 +26,93 @@ struct RotArgs {
   int Hq, Hkv, page_size;
 };
 
-// CTA per row: sines and cosines of its position once, then a warp per head.  y = rotate(x + bias); y / rms(y): queries
-// times q_scale to q_out, keys to their page; a key as it was before rotation and norm goes to the value pages.
-template <typename A>
+// V neighbouring values as one access.
+template <typename A, int V>
+struct Pack {
+  A v[V];
+};
+template <>
+struct __align__(4) Pack<bf16, 2> {
+  bf16 v[2];
+};
+template <>
+struct __align__(8) Pack<float, 2> {
+  float v[2];
+};
+
+// CTA (row, part of the heads): sines and cosines of its position once, then a warp per head, two heads at a time.  Lane:
+// columns V (lane + 32 j).  y = rotate(x + bias); y / rms(y): queries times q_scale to q_out, keys to their page; a key as it
+// was before rotation and norm goes to the value pages.
+template <typename A, int V, int NP>
 __global__ void __launch_bounds__(256) rotate_rms_append_kernel(RotArgs<A> a) {
-  extern __shared__ float2 s_cs[];  // [rot / 2]
+  typedef Pack<A, V> P;
+  extern __shared__ float s_cs[];  // [rot / 2] cosines, then sines
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, lane = threadIdx.x & 31, half = a.rot / 2;
   const int pos = a.row_pos[t];
   const int pidx = pos / a.page_size;
   const bool store = pos >= 0 && pidx < a.max_pages;
+  const A* row = a.x + (size_t)t * a.ld;
+  const int page = store ? a.bt[(size_t)a.row_slot[t] * a.max_pages + pidx] : 0;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     float sn, cs;
     sincosf((float)pos * a.inv_freq[i], &sn, &cs);
-    s_cs[i] = make_float2(cs, sn);
+    s_cs[i] = cs;
+    s_cs[half + i] = sn;
   }
   __syncthreads();
-  const A* row = a.x + (size_t)t * a.ld;
-  const int page = store ? a.bt[(size_t)a.row_slot[t] * a.max_pages + pidx] : 0;
-  for (int h = threadIdx.x >> 5; h < a.Hq + a.Hkv; h += blockDim.x >> 5) {
-    const A* x = row + (size_t)h * a.dim;
-    const float* b = a.bias ? a.bias + (size_t)h * a.dim : nullptr;
-    float raw[kMaxPerLane], y[kMaxPerLane], ss = 0.f;
+  const int heads = a.Hq + a.Hkv, step = gridDim.y * (blockDim.x >> 5);
+  for (int h0 = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5); h0 < heads; h0 += 2 * step) {
+    P raw[2][NP], other[2][NP];
 #pragma unroll
-    for (int j = 0; j < kMaxPerLane; ++j) {
-      const int d = lane + 32 * j;
-      raw[j] = y[j] = 0.f;
-      if (d >= a.dim) continue;
-      raw[j] = to_f32(x[d]) + (b ? b[d] : 0.f);
-      y[j] = raw[j];
-      if (d < a.rot) {
-        const int o = d < half ? d + half : d - half;
-        const float other = to_f32(x[o]) + (b ? b[o] : 0.f);
-        const float2 c = s_cs[d < half ? d : o];
-        y[j] = d < half ? raw[j] * c.x - other * c.y : raw[j] * c.x + other * c.y;
+    for (int u = 0; u < 2; ++u) {
+      const int h = h0 + u * step;
+#pragma unroll
+      for (int j = 0; j < NP; ++j) {
+        const int d = V * (lane + 32 * j);
+        if (h >= heads || d >= a.dim) continue;
+        raw[u][j] = *reinterpret_cast<const P*>(row + (size_t)h * a.dim + d);
+        if (d < a.rot) other[u][j] = *reinterpret_cast<const P*>(row + (size_t)h * a.dim + (d < half ? d + half : d - half));
       }
-      ss = fmaf(y[j], y[j], ss);
     }
-    ss = warp_sum(ss);
-    const float inv = 1.f / sqrtf(ss / (float)a.dim + a.eps);
-    if (h < a.Hq) {
-      A* q = a.q_out + ((size_t)t * a.Hq + h) * a.pad;
 #pragma unroll
-      for (int j = 0; j < kMaxPerLane; ++j)
-        if (lane + 32 * j < a.pad) q[lane + 32 * j] = from_f32<A>(y[j] * inv * a.q_scale);
-    } else if (store) {
-      const size_t at = (((size_t)page * a.Hkv + (h - a.Hq)) * a.page_size + pos % a.page_size) * a.pad;
+    for (int u = 0; u < 2; ++u) {
+      const int h = h0 + u * step;
+      if (h >= heads) break;
+      const float* b = a.bias ? a.bias + (size_t)h * a.dim : nullptr;
+      float x[NP][V], y[NP][V], ss = 0.f;
 #pragma unroll
-      for (int j = 0; j < kMaxPerLane; ++j)
-        if (lane + 32 * j < a.pad) {
-          a.k_pages[at + lane + 32 * j] = from_f32<A>(y[j] * inv);
-          a.v_pages[at + lane + 32 * j] = from_f32<A>(raw[j]);
+      for (int j = 0; j < NP; ++j)
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          const int d = V * (lane + 32 * j) + e;
+          x[j][e] = y[j][e] = 0.f;
+          if (d >= a.dim) continue;
+          x[j][e] = y[j][e] = to_f32(raw[u][j].v[e]) + (b ? b[d] : 0.f);
+          if (d < a.rot) {
+            const int i = d < half ? d : d - half;
+            const float z = to_f32(other[u][j].v[e]) + (b ? b[d < half ? d + half : i] : 0.f);
+            const float cs = s_cs[i], sn = s_cs[half + i];
+            y[j][e] = d < half ? x[j][e] * cs - z * sn : x[j][e] * cs + z * sn;
+          }
+          ss = fmaf(y[j][e], y[j][e], ss);
         }
+      const float inv = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+      const bool is_q = h < a.Hq;
+      const float f = is_q ? inv * a.q_scale : inv;
+      const size_t at = is_q ? ((size_t)t * a.Hq + h) * a.pad
+                             : (((size_t)page * a.Hkv + (h - a.Hq)) * a.page_size + pos % a.page_size) * a.pad;
+#pragma unroll
+      for (int j = 0; j < NP; ++j) {
+        const int d = V * (lane + 32 * j);
+        if (d >= a.pad || (!is_q && !store)) continue;
+        P o, v;
+#pragma unroll
+        for (int e = 0; e < V; ++e) o.v[e] = from_f32<A>(y[j][e] * f), v.v[e] = from_f32<A>(x[j][e]);
+        *reinterpret_cast<P*>((is_q ? a.q_out : a.k_pages) + at + d) = o;
+        if (!is_q) *reinterpret_cast<P*>(a.v_pages + at + d) = v;
+      }
     }
   }
 }
@@ -184,11 +218,21 @@ extern "C" int mlora_rotate_rms_append(const void* d_x, int64_t ld, const float*
   MLORA_REQUIRE(d_x && d_q && d_k_pages && d_v_pages && d_block_table && d_row_slot && d_row_pos && (!rot || d_inv_freq),
                 "rotate_rms_append: null pointer");
   if (T == 0) return MLORA_OK;
+  // two columns per access where halves and heads allow it; few rows: the heads spread over more CTAs
+  const bool two = dim % 2 == 0 && rot % 4 == 0 && pad % 2 == 0 && ld % 2 == 0;
+  const int heads = Hq + Hkv, threads = T >= 1024 ? 256 : 64;
+  const int parts = T >= 1024 ? 1 : (heads + 3) / 4;
   const auto launch = [&](auto zero) {
     using A = decltype(zero);
     RotArgs<A> a{(const A*)d_x, ld, d_bias, d_inv_freq, rot, dim, pad, eps, q_scale, (A*)d_q, (A*)d_k_pages, (A*)d_v_pages,
                  d_block_table, max_pages, d_row_slot, d_row_pos, Hq, Hkv, page_size};
-    launch_pdl_if(pdl_enabled_attn(), rotate_rms_append_kernel<A>, T, 256, (size_t)rot * 4, (cudaStream_t)stream, a);
+    const auto go = [&](auto kernel) {
+      launch_pdl_if(pdl_enabled_attn(), kernel, dim3(T, parts), threads, (size_t)rot * 4, (cudaStream_t)stream, a);
+    };
+    if (two && pad <= 64) go(rotate_rms_append_kernel<A, 2, 1>);
+    else if (two && pad <= 128) go(rotate_rms_append_kernel<A, 2, 2>);
+    else if (two) go(rotate_rms_append_kernel<A, 2, kMaxPerLane / 2>);
+    else go(rotate_rms_append_kernel<A, 1, kMaxPerLane>);
   };
   if (f32)
     launch(0.f);

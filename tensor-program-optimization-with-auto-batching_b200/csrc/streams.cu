@@ -57,8 +57,15 @@ __global__ void __launch_bounds__(512) residual_streams_norm_kernel(StreamsArgs<
   for (int k = threadIdx.x * 8; k < a.H; k += blockDim.x * 8) {
     float x[kN][8], u[8];
 #pragma unroll
-    for (int s = 0; s < kN; ++s)
-      if (s < n) load8(a.src + row * a.ld_src + s * a.src_stream + k, x[s]);
+    for (int s = 0; s < kN; ++s) {
+      if (s >= n) break;
+      if (s > 0 && a.src_stream == 0) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[s][i] = x[0][i];
+      } else {
+        load8(a.src + row * a.ld_src + s * a.src_stream + k, x[s]);
+      }
+    }
 #pragma unroll
     for (int i = 0; i < 8; ++i) u[i] = 0.f;
     if (a.delta) {

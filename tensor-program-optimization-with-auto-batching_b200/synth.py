@@ -157,6 +157,53 @@ def tevudra_weights(cfg: dict, dtype=torch.bfloat16, device="cpu") -> dict:
     return p
 
 
+def relidra_config(name: str) -> dict:
+    """Relidra shapes with layers like a real model's: delta-rule and attention layers in turn, four query heads to a key head."""
+    w, heads, ff, streams = {"relidra-2048": (2048, 16, 8192, 2), "relidra-4096": (4096, 32, 16384, 4)}[name]
+    delta = {"type": "delta", "mixer": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}}
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                          "mask": {"size": 16384}, "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 1.0}}}}
+    return {"architecture": "Relidra", "name": name, "vocab": 32000, "width": w, "streams": streams, "norm": {"eps": 1e-6},
+            "layers": [dict((att if i % 2 else delta), mlp={"kind": "dense", "ff": ff}) for i in range(4)]}
+
+
+def relidra_weights(cfg: dict, dtype=torch.bfloat16, device="cpu") -> dict:
+    """Random weights of a Relidra configuration: matrices ~ N(0, 1/in), norm weights 1 + N(0, 0.02), streams that mostly stay
+    themselves."""
+    g = _gen(SEED_WEIGHTS, device)
+    rnd = lambda *s: torch.randn(*s, generator=g, device=device, dtype=torch.float32)
+    mat = lambda o, i: (rnd(o, i) / math.sqrt(i)).to(dtype)
+    W, n = cfg["width"], cfg["streams"]
+    p = {"embed": rnd(cfg["vocab"], W).to(dtype), "final.norm": (1 + 0.02 * rnd(W)).to(dtype)}
+
+    def sublayer(i, q):
+        p[f"l{i}.norm{q}"] = (1 + 0.02 * rnd(W)).to(dtype)
+        hc = f"l{i}.hc{q}."
+        p[hc + "in"], p[hc + "out"] = (1 / n + 0.1 * rnd(n)).to(dtype), (0.5 + 0.1 * rnd(n)).to(dtype)
+        p[hc + "mix"] = (torch.eye(n, device=device) + 0.1 * rnd(n, n)).to(dtype)
+
+    for i, layer in enumerate(cfg["layers"]):
+        m, x = layer["mixer"], f"l{i}.mix."
+        H, G, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        sublayer(i, 1)
+        for name, rows in (("q", G * d), ("k", G * d), ("v", H * v)) if layer["type"] == "delta" else (("q", H * d), ("k", G * d)):
+            p[x + name] = mat(rows, W)
+            if layer["type"] == "delta":
+                p[x + name + ".conv"] = (rnd(rows, m["conv"]) / math.sqrt(m["conv"])).to(dtype)
+            else:
+                p[x + name + ".b"] = (0.1 * rnd(rows)).to(dtype)
+        p[x + "o"] = mat(W, H * v)
+        if layer["type"] == "delta":
+            p[x + "g"], p[x + "b"], p[x + "a"] = mat(H * v, W), mat(H, W), mat(H, W)
+            p[x + "A_log"], p[x + "dt_bias"], p[x + "norm"] = rnd(H).to(dtype) - 2, rnd(H).to(dtype) - 2, (1 + 0.02 * rnd(v)).to(dtype)
+        else:
+            p[x + "sink"] = rnd(H).to(dtype)
+        if layer["mlp"]:
+            sublayer(i, 2)
+            p[f"l{i}.mlp.up"], p[f"l{i}.mlp.down"] = mat(layer["mlp"]["ff"], W), mat(W, layer["mlp"]["ff"])
+    return p
+
+
 def adapter_ids_uniform(n_requests: int, n_adapters: int) -> np.ndarray:
     return np.random.default_rng(SEED_IDS).integers(0, n_adapters, n_requests).astype(np.int32)
 
