@@ -58,11 +58,10 @@ __global__ void __launch_bounds__(512) residual_streams_norm_kernel(StreamsArgs<
     float x[kN][8], u[8];
 #pragma unroll
     for (int s = 0; s < kN; ++s) {
-      if (s >= n) break;
       if (s > 0 && a.src_stream == 0) {
 #pragma unroll
         for (int i = 0; i < 8; ++i) x[s][i] = x[0][i];
-      } else {
+      } else if (s < n) {
         load8(a.src + row * a.ld_src + s * a.src_stream + k, x[s]);
       }
     }
