@@ -1072,7 +1072,7 @@ class KernelTimer:
     NAMES = ("linear", "grouped_linear", "moe_plan", "moe_route_plan", "residual_dyt", "residual_rmsnorm", "latent_append", "latent_gather",
              "latent_attention", "prefill_attention_dense", "embed", "argmax", "paged_attention", "prefill_attention",
              "kv_append_rope", "paged_attention_masked", "prefill_attention_masked", "residual_streams_layernorm", "rotate_rms_append",
-             "short_conv", "delta_scan", "gated_rms", "delta_step")
+             "short_conv", "delta_scan", "delta_chunk", "gated_rms", "delta_step")
 
     def __init__(self, ops, torch, dev, hbm_gbs, tflops):
         self.ops, self.torch, self.hbm, self.tflops = ops, torch, hbm_gbs, tflops
@@ -1123,8 +1123,8 @@ class KernelTimer:
             return f"{a[0].shape[0]} rows", 2 * a[0].shape[0] * (a[0].shape[1] + a[7].shape[1] + 2 * a[14] * a[8].shape[3]), 0.0
         if name == "short_conv":
             return f"{a[5].shape[0]} rows x {a[5].shape[1]}", 4 * a[5].numel(), 0.0
-        if name == "delta_scan":
-            r, o = a[2], a[7]
+        if name in ("delta_scan", "delta_chunk"):
+            r, o = a[2], a[7 if name == "delta_scan" else 8]
             return (f"{o.shape[0]} rows, {r.heads} heads, {len(news)} sequences",
                     2 * a[0].numel() + 4 * o.numel() + 8 * len(news) * r.heads * r.dim * r.vdim, 0.0)
         if name == "gated_rms":

@@ -574,6 +574,9 @@ int mlora_paged_attention_any(const void* d_q, const void* d_k_pages, const void
  * mlora_delta_scan: the recurrence over the rows of each segment int32 [n][4] = (slot, first row, rows, position of the first
  *   row), one segment per sequence; xc from mlora_short_conv, x the projected rows with b and a from columns b_col and a_col.
  *   Leaves state and ring after the segment's last row, and o [T, heads * vdim] fp32.
+ * mlora_delta_chunk: the same on the tensor cores, 64 tokens at a time (bf16 activations, dim 64 or 128; fp32 factors in three
+ *   bf16 planes, so results agree to fp32 rounding).  T = rows of x and xc, max_rows = rows of the longest segment; d_work:
+ *   mlora_delta_chunk_workspace bytes; d_status as for mlora_prefill_attention.
  * mlora_gated_rms: out = o / sqrt(mean(o^2) + eps) * w * silu(gate) per head (mean over the first vdim_true columns).
  * mlora_delta_step: everything for one new token per row (gate from column g_col); rows with row_pos < 0 give zeros. */
 int mlora_short_conv(const void* d_x, int64_t ld, int32_t C, int32_t taps, const float* d_w, const void* d_ring,
@@ -582,6 +585,11 @@ int mlora_delta_scan(const void* d_xc, const void* d_x, int64_t ld, int32_t C, i
                      const float* d_A_log, const float* d_dt_bias, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim,
                      float q_scale, const int32_t* d_segs, int32_t n_segs, float* d_state, void* d_ring, float* d_out, int32_t f32,
                      void* stream);
+size_t mlora_delta_chunk_workspace(int32_t T, int32_t n_segs, int32_t heads);
+int mlora_delta_chunk(const void* d_xc, const void* d_x, int64_t ld, int32_t C, int32_t taps, int32_t b_col, int32_t a_col,
+                      const float* d_A_log, const float* d_dt_bias, int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim,
+                      float q_scale, const int32_t* d_segs, int32_t n_segs, int32_t T, int32_t max_rows, float* d_state, void* d_ring,
+                      float* d_out, void* d_work, size_t work_bytes, int32_t* d_status, void* stream);
 int mlora_gated_rms(const float* d_o, const void* d_gate, int64_t ld_gate, const float* d_w, int32_t T, int32_t heads, int32_t vdim,
                     int32_t vdim_true, float eps, void* d_out, int32_t f32, void* stream);
 int mlora_delta_step(const void* d_x, int64_t ld, int32_t C, int32_t taps, int32_t g_col, int32_t b_col, int32_t a_col,

@@ -107,6 +107,9 @@ PROTOTYPES = {
     "mlora_short_conv": (C.c_int, [_vp, _i64, _i32, _i32, _vp, _vp, _vp, _vp, _i32, _vp, _i32, _vp]),
     "mlora_delta_scan": (C.c_int, [_vp, _vp, _i64, _i32, _i32, _i32, _i32, _vp, _vp, _i32, _i32, _i32, _i32, _f32, _vp, _i32,
                                    _vp, _vp, _vp, _i32, _vp]),
+    "mlora_delta_chunk_workspace": (_sz, [_i32, _i32, _i32]),
+    "mlora_delta_chunk": (C.c_int, [_vp, _vp, _i64, _i32, _i32, _i32, _i32, _vp, _vp, _i32, _i32, _i32, _i32, _f32, _vp, _i32,
+                                    _i32, _i32, _vp, _vp, _vp, _vp, _sz, _vp, _vp]),
     "mlora_gated_rms": (C.c_int, [_vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _f32, _vp, _i32, _vp]),
     "mlora_delta_step": (C.c_int, [_vp, _i64, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _f32, _i32, _i32, _i32, _i32,
                                    _i32, _f32, _vp, _vp, _i32, _vp, _vp, _vp, _i32, _vp]),

@@ -37,18 +37,6 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-// Shared-memory descriptor of an MN-major operand tile with 128-byte swizzle: rows of 128 bytes hold 64 consecutive
-// M/N elements of one k; `lbo` bytes to the next 64 M/N elements, `sbo` bytes to the next 8 k.
-__device__ __forceinline__ uint64_t make_smem_desc_mn(uint32_t saddr, uint32_t lbo, uint32_t sbo) {
-  uint64_t d = 0;
-  d |= (uint64_t)((saddr & 0x3FFFFu) >> 4);
-  d |= (uint64_t)(lbo >> 4) << 16;
-  d |= (uint64_t)(sbo >> 4) << 32;
-  d |= (uint64_t)1 << 46;
-  d |= (uint64_t)2 << 61;
-  return d;
-}
-
 struct PfArgs {
   const int32_t* block_table;  // paged form
   int max_pages;

@@ -21,7 +21,7 @@
 // Products are done on pairs of rows (fma.rn.f32x2).
 #include <cmath>
 
-#include "act_io.cuh"
+#include "delta.cuh"
 
 namespace mlora {
 namespace {
@@ -47,8 +47,6 @@ template <typename A>
 __device__ __forceinline__ void load4(const A* p, float (&f)[4]) {
   widen4(*reinterpret_cast<const typename Raw4<A>::type*>(p), f);
 }
-__device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
-__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 typedef unsigned long long f32x2;  // two fp32 values in one register pair
 __device__ __forceinline__ f32x2 pack2(float a, float b) {
@@ -71,12 +69,6 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
   return r;
 }
-
-struct DeltaDims {
-  int heads, kv_heads, dim, vdim;  // sizes as stored: multiples of 8
-  int vdim_true;                   // columns the norm's mean goes over
-  float q_scale;
-};
 
 // The part of a state one warp holds: 16 columns, RJ * 32 rows.  Lane l: rows 32 j + 4 (l % 8) + {0..3}, columns
 // 4 (l / 8) + {0..3}.
@@ -179,7 +171,6 @@ struct ConvArgs {
 };
 
 constexpr int kConvRows = 16;  // rows per thread, walked with the inputs of the last tokens in registers
-constexpr int kMaxTaps = 8;
 
 // Thread: 8 channels x kConvRows rows.  K taps.
 template <typename A, int K>
@@ -243,9 +234,6 @@ struct ScanArgs {
   A* ring;              // [slot][taps][C]
   float* out;           // [T, heads * vdim]
 };
-
-__device__ __forceinline__ float step_size(float b) { return 1.f / (1.f + expf(-b)); }
-__device__ __forceinline__ float decay(float a, float A_log, float dt_bias) { return expf(-expf(A_log) * softplus(a + dt_bias)); }
 
 constexpr int kPer = 2;  // tokens a warp stages per block of tokens
 
@@ -322,7 +310,7 @@ __global__ void __launch_bounds__(NW * 32) delta_scan_kernel(ScanArgs<A> a) {
         }
       }
       if (4 * lane < kCols) *reinterpret_cast<float4*>(s_v + tok * kCols + 4 * lane) = make_float4(fv[0], fv[1], fv[2], fv[3]);
-      if (lane == 0) s_g[tok] = make_float4(decay(to_f32(pa[e]), A_log, dt_bias), step_size(to_f32(pb[e])), sx * iq * ik, 0.f);
+      if (lane == 0) s_g[tok] = make_float4(expf(log_decay(to_f32(pa[e]), A_log, dt_bias)), step_size(to_f32(pb[e])), sx * iq * ik, 0.f);
     }
   };
 
@@ -456,7 +444,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(StepArgs<A> a) {
   const A* row = a.x + (size_t)t * a.ld;
   A* ring = a.ring + (size_t)slot * a.taps * a.C;
   const int q_col = kh * d.dim, k_col = (d.kv_heads + kh) * d.dim, v_col = 2 * d.kv_heads * d.dim + h * d.vdim;
-  const float beta = step_size(to_f32(row[a.b_col + h])), g = decay(to_f32(row[a.a_col + h]), a.A_log[h], a.dt_bias[h]);
+  const float beta = step_size(to_f32(row[a.b_col + h])), g = expf(log_decay(to_f32(row[a.a_col + h]), a.A_log[h], a.dt_bias[h]));
   for (int i = tid; i < 2 * kRows + d.vdim; i += threads) {
     const int part = i < kRows ? 0 : i < 2 * kRows ? 1 : 2, e = i - part * kRows;
     float val = 0.f;
@@ -518,16 +506,6 @@ __global__ void __launch_bounds__(256) delta_step_kernel(StepArgs<A> a) {
 }
 
 // ---- host --------------------------------------------------------------------------------------------------------------------
-int check_dims(const char* who, const DeltaDims& d, int C, int taps) {
-  MLORA_REQUIRE(d.heads > 0 && d.kv_heads > 0 && d.heads % d.kv_heads == 0 && d.heads <= 65535, "%s: bad head counts", who);
-  MLORA_REQUIRE(d.dim > 0 && d.dim % 8 == 0 && d.dim <= 256, "%s: dim a multiple of 8 up to 256 (got %d)", who, d.dim);
-  MLORA_REQUIRE(d.vdim > 0 && d.vdim % 8 == 0 && d.vdim <= 4096 && d.vdim_true > 0 && d.vdim_true <= d.vdim,
-                "%s: vdim a multiple of 8 up to 4096 (got %d)", who, d.vdim);
-  MLORA_REQUIRE(C % 8 == 0 && C >= 2 * d.kv_heads * d.dim + d.heads * d.vdim, "%s: too few channels (%d)", who, C);
-  MLORA_REQUIRE(taps > 0 && taps <= kMaxTaps, "%s: 1 to %d taps (got %d)", who, kMaxTaps, taps);
-  return MLORA_OK;
-}
-
 template <typename A, int RJ, int NW>
 int launch_scan(const ScanArgs<A>& a, int n_segs, cudaStream_t st) {
   constexpr int kTok = kPer * NW;
@@ -554,6 +532,18 @@ int launch_scan_rows(const ScanArgs<A>& a, int n_segs, cudaStream_t st) {
 }
 
 }  // namespace
+}  // namespace mlora
+
+namespace mlora {
+int check_delta_dims(const char* who, const DeltaDims& d, int C, int taps) {
+  MLORA_REQUIRE(d.heads > 0 && d.kv_heads > 0 && d.heads % d.kv_heads == 0 && d.heads <= 65535, "%s: bad head counts", who);
+  MLORA_REQUIRE(d.dim > 0 && d.dim % 8 == 0 && d.dim <= 256, "%s: dim a multiple of 8 up to 256 (got %d)", who, d.dim);
+  MLORA_REQUIRE(d.vdim > 0 && d.vdim % 8 == 0 && d.vdim <= 4096 && d.vdim_true > 0 && d.vdim_true <= d.vdim,
+                "%s: vdim a multiple of 8 up to 4096 (got %d)", who, d.vdim);
+  MLORA_REQUIRE(C % 8 == 0 && C >= 2 * d.kv_heads * d.dim + d.heads * d.vdim, "%s: too few channels (%d)", who, C);
+  MLORA_REQUIRE(taps > 0 && taps <= kMaxTaps, "%s: 1 to %d taps (got %d)", who, kMaxTaps, taps);
+  return MLORA_OK;
+}
 }  // namespace mlora
 
 using namespace mlora;
@@ -597,7 +587,7 @@ extern "C" int mlora_delta_scan(const void* d_xc, const void* d_x, int64_t ld, i
                                 int32_t dim, int32_t vdim, float q_scale, const int32_t* d_segs, int32_t n_segs, float* d_state,
                                 void* d_ring, float* d_out, int32_t f32, void* stream) {
   const DeltaDims d{heads, kv_heads, dim, vdim, vdim, q_scale};
-  const int rc = check_dims("delta_scan", d, C, taps);
+  const int rc = check_delta_dims("delta_scan", d, C, taps);
   if (rc) return rc;
   MLORA_REQUIRE(n_segs >= 0 && n_segs <= 65535 && ld >= C && b_col >= 0 && a_col >= 0 && b_col + heads <= ld && a_col + heads <= ld,
                 "delta_scan: bad sizes");
@@ -642,7 +632,7 @@ extern "C" int mlora_delta_step(const void* d_x, int64_t ld, int32_t C, int32_t 
                                 const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, float* d_state, void* d_ring,
                                 void* d_out, int32_t f32, void* stream) {
   const DeltaDims d{heads, kv_heads, dim, vdim, vdim_true, q_scale};
-  const int rc = check_dims("delta_step", d, C, taps);
+  const int rc = check_delta_dims("delta_step", d, C, taps);
   if (rc) return rc;
   MLORA_REQUIRE(T >= 0 && T <= 65535 && ld >= C && g_col >= 0 && b_col >= 0 && a_col >= 0 && b_col + heads <= ld &&
                     a_col + heads <= ld && (int64_t)g_col + heads * vdim <= ld,

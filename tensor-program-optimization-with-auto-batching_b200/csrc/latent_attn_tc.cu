@@ -55,52 +55,6 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
-__device__ __forceinline__ uint64_t desc_mn(uint32_t saddr, uint32_t lbo, uint32_t sbo) {
-  uint64_t d = 0;
-  d |= (uint64_t)((saddr & 0x3FFFFu) >> 4);
-  d |= (uint64_t)(lbo >> 4) << 16;
-  d |= (uint64_t)(sbo >> 4) << 32;
-  d |= (uint64_t)1 << 46;
-  d |= (uint64_t)2 << 61;
-  return d;
-}
-
-// D [128 x N] (+)= A [128 x 16] . B^T with A in TMEM: two bf16 of the K dimension per 32-bit column.
-__device__ __forceinline__ void umma_bf16_ta(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t acc) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(acc)
-      : "memory");
-}
-
-template <int N>
-__device__ __forceinline__ void tmem_ld(uint32_t addr, float (&v)[32]) {
-  if constexpr (N == 32) tmem_ld32(addr, v); else tmem_ld16(addr, v);
-}
-template <int N>
-__device__ __forceinline__ void tmem_st(uint32_t addr, const float (&v)[32]) {
-  const uint32_t* r = reinterpret_cast<const uint32_t*>(v);
-  if constexpr (N == 32)
-    asm volatile(
-        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-        "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,"
-        "%30,%31,%32};" ::"r"(addr),
-        "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]),
-        "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]),
-        "r"(r[21]), "r"(r[22]), "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]),
-        "r"(r[31])
-        : "memory");
-  else
-    asm volatile(
-        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(addr),
-        "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]),
-        "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
-        : "memory");
-  asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
-}
-
 template <int HG>
 __global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(LtArgs a) {
   extern __shared__ uint8_t smem_raw[];
@@ -216,7 +170,7 @@ __global__ void __launch_bounds__(kLtThreads, 1) latent_attn_tc_kernel(LtArgs a)
           const uint32_t c = smem_u32(ring + s_o * slot_bytes + j * 2048);
 #pragma unroll
           for (int k = 0; k < 4; ++k)  // 16 keys = two row groups
-            umma_bf16(tmem_o + j * 32, desc_mn(c + k * 2 * group, 1024, group), pd + 2 * k, idesc_o, (b | k) ? 1u : 0u);
+            umma_bf16(tmem_o + j * 32, make_smem_desc_mn(c + k * 2 * group, 1024, group), pd + 2 * k, idesc_o, (b | k) ? 1u : 0u);
         }
         umma_commit(&empty_bar[s_o]);
         umma_commit(&o_bar[b & 1]);

@@ -762,6 +762,27 @@ def delta_scan(xc, x, r: DeltaRule, segs, n_segs, state, ring, out):
     return out
 
 
+DELTA_CHUNK_MIN_ROWS = 24  # a pass with a longer segment walks chunks of 64 tokens, a shorter one single tokens
+
+
+def delta_chunk_fits(r: DeltaRule, dtype, max_rows) -> bool:
+    return dtype == torch.bfloat16 and r.dim in (64, 128) and max_rows >= DELTA_CHUNK_MIN_ROWS
+
+
+def delta_chunk_workspace(T, n_segs, heads) -> int:
+    return int(_lib.lib().mlora_delta_chunk_workspace(T, n_segs, heads))
+
+
+def delta_chunk(xc, x, r: DeltaRule, segs, n_segs, max_rows, state, ring, out, work, status=None):
+    """:func:`delta_scan` 64 tokens at a time; ``max_rows``: rows of the longest segment."""
+    _need_cuda(xc, state)
+    check(_lib.lib().mlora_delta_chunk(
+        _ptr(xc), _ptr(x), x.stride(0), r.channels, r.taps, r.b_col, r.a_col, _ptr(r.A_log), _ptr(r.dt_bias), r.heads, r.kv_heads,
+        r.dim, r.vdim, r.q_scale, _ptr(segs), n_segs, x.shape[0], max_rows, _ptr(state), _ptr(ring), _ptr(out), _ptr(work),
+        work.numel(), _ptr(status), _stream()), "mlora_delta_chunk")
+    return out
+
+
 def gated_rms(o, gate, w, heads, vdim_true, eps, out):
     """o [T, heads * vdim] fp32, gate [T, >= heads * vdim] (a column slice is fine)."""
     _need_cuda(o, gate)

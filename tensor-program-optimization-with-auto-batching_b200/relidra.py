@@ -228,7 +228,7 @@ class RelidraEngine(PlainEngine):
         # prompt passes: segments of the recurrence, query tiles of <= 128 rows
         self.segs = torch.zeros(kv.max_batch, 4, dtype=torch.int32, device=dev)
         self.tiles = torch.zeros((T + 127) // 128 + kv.max_batch + 1, 4, dtype=torch.int32, device=dev)
-        self._n_segs = self._n_tiles = 0
+        self._n_segs = self._n_tiles = self._max_seg = 0
 
     # -- prompt passes ------------------------------------------------------------------------------------------
     def _begin_prompt_pass(self, chunk):
@@ -236,7 +236,7 @@ class RelidraEngine(PlainEngine):
         tiles = [(s, r0 + off, min(128, n - off), p0 + off) for s, r0, n, p0 in segs for off in range(0, n, 128)]
         for dst, v in ((self.segs, segs), (self.tiles, tiles)):
             self._stage(dst.view(-1), np.asarray(v, dtype=np.int32).reshape(-1), torch.int32)
-        self._n_segs, self._n_tiles = len(segs), len(tiles)
+        self._n_segs, self._n_tiles, self._max_seg = len(segs), len(tiles), max(n for _, _, n, _ in segs)
 
     def _end_prompt_pass(self):
         self._n_segs = self._n_tiles = 0
@@ -250,7 +250,11 @@ class RelidraEngine(PlainEngine):
         xc = ops.short_conv(proj, r.conv, ring, row_slot, row_pos, self._grow("conv", self.max_rows * self._conv_cols)[:T * r.channels]
                             .view(T, r.channels))
         o = self._grow("o", self.max_rows * self._o_cols, torch.float32)[:T * lw.out_cols].view(T, lw.out_cols)
-        ops.delta_scan(xc, proj, r, self.segs, self._n_segs, S, ring, o)
+        if ops.delta_chunk_fits(r, self.m.dtype, self._max_seg):
+            work = self._grow("chunks", ops.delta_chunk_workspace(T, self._n_segs, r.heads), torch.uint8)
+            ops.delta_chunk(xc, proj, r, self.segs, self._n_segs, self._max_seg, S, ring, o, work, status=self.status)
+        else:
+            ops.delta_scan(xc, proj, r, self.segs, self._n_segs, S, ring, o)
         return ops.gated_rms(o, proj[:, r.g_col:], r.norm, r.heads, r.vdim_true, eps, out)
 
     def _attention(self, T, lw, run, proj, out, decode):

@@ -221,8 +221,8 @@ class DeltaCase:
     def slot(self, s):
         return len(self.rows) - s
 
-    def scan(self, parts):
-        """parts: (sequence, rows) in the order of the pass."""
+    def scan(self, parts, chunks=False):
+        """parts: (sequence, rows) in the order of the pass.  chunks: 64 tokens at a time on the tensor cores."""
         ops, r, cuda = self.ops, self.rule, self.cuda
         segs, rows, slots, pos, first = [], [], [], [], 0
         for s, n in parts:
@@ -237,7 +237,14 @@ class DeltaCase:
         o = torch.full((T, r.heads * r.vdim), nan, device=cuda)
         out = torch.full((T, r.heads * r.vdim), nan, dtype=self.dtype, device=cuda)
         ops.short_conv(x, r.conv, self.ring, i32(slots, cuda), i32(pos, cuda), xc)
-        ops.delta_scan(xc, x, r, i32(segs, cuda), len(segs), self.state, self.ring, o)
+        if chunks:
+            work = torch.full((ops.delta_chunk_workspace(T, len(segs), r.heads),), 255, dtype=torch.uint8, device=cuda)
+            status = torch.zeros(1, dtype=torch.int32, device=cuda)
+            ops.delta_chunk(xc, x, r, i32(segs, cuda), len(segs), max(n for _, n in parts), self.state, self.ring, o, work, status)
+            assert not int(status)
+        else:
+            ops.delta_scan(xc, x, r, i32(segs, cuda), len(segs), self.state, self.ring, o)
+        self.raw = o
         ops.gated_rms(o, x[:, r.g_col:], r.norm, r.heads, r.vdim_true, 1e-4, out)
         for (s, n), (_, a, _, _) in zip(parts, segs):
             self.got[s].append(out[a:a + n])
@@ -294,6 +301,51 @@ def test_delta_portions_and_single_tokens(ops, cuda, dtype, size):
         c.step([0])
     c.scan([(1, 2)])
     c.check()
+
+
+CHUNKED = [(2, 2, 64, 64, 4), (4, 2, 64, 24, 3), (3, 1, 128, 128, 4), (2, 2, 128, 200, 2), (1, 1, 57, 33, 4), (2, 1, 121, 136, 5)]
+
+
+@pytest.mark.parametrize("size", CHUNKED)
+def test_delta_chunks_whole_sequences(ops, cuda, size):
+    c = DeltaCase(ops, cuda, BF, *size, lengths=(1, 64, 2, 63, 200, 65, 128))
+    c.scan([(1, 64), (0, 1), (4, 200), (2, 2), (3, 63), (6, 128), (5, 65)], chunks=True)
+    c.check()
+    # the same rows one token at a time: equal to fp32 rounding, before anything is rounded to 16 bits
+    one = DeltaCase(ops, cuda, BF, *size, lengths=(1, 64, 2, 63, 200, 65, 128))
+    one.scan([(1, 64), (0, 1), (4, 200), (2, 2), (3, 63), (6, 128), (5, 65)])
+    close(c.raw, one.raw, F32, f32=5e-6)
+    used = slice(1, len(c.rows) + 1)
+    close(c.state[used], one.state[used], F32, f32=5e-6)
+    assert torch.equal(c.ring.nan_to_num(), one.ring.nan_to_num())
+
+
+@pytest.mark.parametrize("size", CHUNKED[:4])
+def test_delta_chunks_portions_and_single_tokens(ops, cuda, size):
+    c = DeltaCase(ops, cuda, BF, *size, lengths=(300, 150))
+    for part in ([(0, 1)], [(0, 2), (1, 20)], [(1, 70), (0, 64)], [(0, 100)], [(1, 1), (0, 65)]):
+        c.scan(part, chunks=True)
+    for _ in range(6):
+        c.step([1, -1, 0])
+    c.scan([(0, 20), (1, 2)])
+    c.scan([(0, 40), (1, 50)], chunks=True)
+    while c.at[1] < 150:
+        c.step([1])
+    c.scan([(0, 2)], chunks=True)
+    c.check()
+
+
+def test_delta_chunks_many_tokens_and_strong_decays(ops, cuda):
+    """Long walks; decays from almost none to complete within a few tokens."""
+    for shift in (0.0, 4.0, 8.0):
+        c = DeltaCase(ops, cuda, BF, 2, 1, 64, 32, 4, lengths=(1500,))
+        c.rule.A_log += shift
+        one = DeltaCase(ops, cuda, BF, 2, 1, 64, 32, 4, lengths=(1500,))
+        one.rule.A_log += shift
+        c.scan([(0, 1500)], chunks=True)
+        one.scan([(0, 1500)])
+        close(c.raw, one.raw, F32, f32=2e-5)
+        close(c.state[1], one.state[1], F32, f32=2e-5)
 
 
 def test_delta_many_tokens_one_by_one(ops, cuda):
