@@ -39,6 +39,14 @@ template <>
 struct __align__(8) Pack<float, 2> {
   float v[2];
 };
+template <>
+struct __align__(8) Pack<bf16, 4> {
+  bf16 v[4];
+};
+template <>
+struct __align__(16) Pack<float, 4> {
+  float v[4];
+};
 
 // CTA (row, part of the heads): sines and cosines of its position once, then a warp per head, two heads at a time.  Lane:
 // columns V (lane + 32 j).  y = rotate(x + bias); y / rms(y): queries times q_scale to q_out, keys to their page; a key as it
@@ -46,7 +54,7 @@ struct __align__(8) Pack<float, 2> {
 template <typename A, int V, int NP>
 __global__ void __launch_bounds__(256) rotate_rms_append_kernel(RotArgs<A> a) {
   typedef Pack<A, V> P;
-  extern __shared__ float s_cs[];  // [rot / 2] cosines, then sines
+  extern __shared__ __align__(16) float s_cs[];  // [rot / 2] cosines, then sines
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, lane = threadIdx.x & 31, half = a.rot / 2;
@@ -80,24 +88,30 @@ __global__ void __launch_bounds__(256) rotate_rms_append_kernel(RotArgs<A> a) {
     for (int u = 0; u < 2; ++u) {
       const int h = h0 + u * step;
       if (h >= heads) break;
+      typedef Pack<float, V> F;
       const float* b = a.bias ? a.bias + (size_t)h * a.dim : nullptr;
       float x[NP][V], y[NP][V], ss = 0.f;
 #pragma unroll
-      for (int j = 0; j < NP; ++j)
+      for (int j = 0; j < NP; ++j) {  // (a lane's V columns lie on one side of the half, inside or outside of the rotated part)
+        const int d = V * (lane + 32 * j);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[j][e] = y[j][e] = 0.f;
+        if (d >= a.dim) continue;
+        F bd{}, bo{}, cs, sn;
+        const int i = d < half ? d : d - half;
+        if (b) bd = *reinterpret_cast<const F*>(b + d);
+        if (b && d < a.rot) bo = *reinterpret_cast<const F*>(b + (d < half ? d + half : i));
+        if (d < a.rot) cs = *reinterpret_cast<const F*>(s_cs + i), sn = *reinterpret_cast<const F*>(s_cs + half + i);
 #pragma unroll
         for (int e = 0; e < V; ++e) {
-          const int d = V * (lane + 32 * j) + e;
-          x[j][e] = y[j][e] = 0.f;
-          if (d >= a.dim) continue;
-          x[j][e] = y[j][e] = to_f32(raw[u][j].v[e]) + (b ? b[d] : 0.f);
+          x[j][e] = y[j][e] = to_f32(raw[u][j].v[e]) + bd.v[e];
           if (d < a.rot) {
-            const int i = d < half ? d : d - half;
-            const float z = to_f32(other[u][j].v[e]) + (b ? b[d < half ? d + half : i] : 0.f);
-            const float cs = s_cs[i], sn = s_cs[half + i];
-            y[j][e] = d < half ? x[j][e] * cs - z * sn : x[j][e] * cs + z * sn;
+            const float z = (to_f32(other[u][j].v[e]) + bo.v[e]) * (d < half ? -sn.v[e] : sn.v[e]);
+            y[j][e] = fmaf(x[j][e], cs.v[e], z);
           }
           ss = fmaf(y[j][e], y[j][e], ss);
         }
+      }
       const float inv = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
       const bool is_q = h < a.Hq;
       const float f = is_q ? inv * a.q_scale : inv;
@@ -218,8 +232,10 @@ extern "C" int mlora_rotate_rms_append(const void* d_x, int64_t ld, const float*
   MLORA_REQUIRE(d_x && d_q && d_k_pages && d_v_pages && d_block_table && d_row_slot && d_row_pos && (!rot || d_inv_freq),
                 "rotate_rms_append: null pointer");
   if (T == 0) return MLORA_OK;
-  // two columns per access where halves and heads allow it; few rows: the heads spread over more CTAs
+  // two or four columns per access where halves and heads allow it; few rows: the heads spread over more CTAs
   const bool two = dim % 2 == 0 && rot % 4 == 0 && pad % 2 == 0 && ld % 2 == 0;
+  const bool four = dim % 4 == 0 && rot % 8 == 0 && pad % 4 == 0 && ld % 4 == 0 && aligned16(d_x) && aligned16(d_bias) &&
+                    aligned16(d_q) && aligned16(d_k_pages) && aligned16(d_v_pages);
   const int heads = Hq + Hkv, threads = T >= 1024 ? 256 : 64;
   const int parts = T >= 1024 ? 1 : (heads + 3) / 4;
   const auto launch = [&](auto zero) {
@@ -229,7 +245,8 @@ extern "C" int mlora_rotate_rms_append(const void* d_x, int64_t ld, const float*
     const auto go = [&](auto kernel) {
       launch_pdl_if(pdl_enabled_attn(), kernel, dim3(T, parts), threads, (size_t)rot * 4, (cudaStream_t)stream, a);
     };
-    if (two && pad <= 64) go(rotate_rms_append_kernel<A, 2, 1>);
+    if (four && pad <= 128) go(rotate_rms_append_kernel<A, 4, 1>);
+    else if (two && pad <= 64) go(rotate_rms_append_kernel<A, 2, 1>);
     else if (two && pad <= 128) go(rotate_rms_append_kernel<A, 2, 2>);
     else if (two) go(rotate_rms_append_kernel<A, 2, kMaxPerLane / 2>);
     else go(rotate_rms_append_kernel<A, 1, kMaxPerLane>);

@@ -214,7 +214,7 @@ __global__ void __launch_bounds__(128) short_conv_kernel(ConvArgs<A> a) {
       float s = 0.f;
 #pragma unroll
       for (int j = K - 1; j >= 0; --j) s = fmaf(w[K - 1 - j][i], h[j][i], s);
-      o[i] = silu(s);
+      o[i] = silu<A>(s);
     }
     store8(a.out + (size_t)t * a.C + c, o);
   }
@@ -387,7 +387,7 @@ __global__ void __launch_bounds__(256) gated_rms_kernel(const float* __restrict_
     load4(gt + i, g);
     load4(w + i, wt);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) v[j] = v[j] * inv * wt[j] * silu(g[j]);
+    for (int j = 0; j < 4; ++j) v[j] = v[j] * inv * wt[j] * silu<A>(g[j]);
     A* dst = out + (size_t)r * vdim + i;
     if constexpr (sizeof(A) == 2) {
       __nv_bfloat162 p[2] = {__floats2bfloat162_rn(v[0], v[1]), __floats2bfloat162_rn(v[2], v[3])};
@@ -456,7 +456,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(StepArgs<A> a) {
         s = fmaf(a.conv[(size_t)(a.taps - 1 - j) * a.C + ch], to_f32(ring[(size_t)((pos - j) % a.taps) * a.C + ch]), s);
       s = fmaf(a.conv[(size_t)(a.taps - 1) * a.C + ch], to_f32(cur), s);
       if (part == 2 || h % rep == 0) ring[(size_t)(pos % a.taps) * a.C + ch] = cur;
-      val = silu(s);
+      val = silu<float>(s);
     }
     smem[i] = val;
   }
@@ -502,7 +502,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(StepArgs<A> a) {
   for (int i = lane; i < d.vdim; i += 32) ss = fmaf(s_o[i], s_o[i], ss);
   const float inv = 1.f / sqrtf(warp_sum(ss) / (float)d.vdim_true + a.eps);
   for (int i = tid; i < d.vdim; i += threads)
-    out[i] = from_f32<A>(s_o[i] * inv * a.norm_w[i] * silu(to_f32(row[a.g_col + h * d.vdim + i])));
+    out[i] = from_f32<A>(s_o[i] * inv * a.norm_w[i] * silu<A>(to_f32(row[a.g_col + h * d.vdim + i])));
 }
 
 // ---- host --------------------------------------------------------------------------------------------------------------------

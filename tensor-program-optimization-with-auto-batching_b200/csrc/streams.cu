@@ -19,12 +19,13 @@ struct StreamsArgs {
   int64_t ld_src, src_stream;
   float* dst;             // streams after [T][n][H], or NULL: not stored
   const float* back;      // [n] + [n, n]: what every stream gets of delta, then mix[from][to]; with delta
-  const float* read;      // [n] weights of the sum that is normalised
+  const float* read;      // [n_read] weights of the sum that is normalised
   const int32_t* rows;    // NULL: every row; else output row i is row rows[i]
   const bf16* w;
   float eps;
   A* out;
-  int n, H, width;        // H: pitch of all rows (a multiple of 8); width: columns that count
+  int n, n_read;          // n_read = n, or (n = 1) the weights of streams that are all the one row
+  int H, width;           // H: pitch of all rows (a multiple of 8); width: columns that count
 };
 
 __device__ __forceinline__ float cta_sum(float v, float* sm /*[33]*/) {
@@ -51,7 +52,15 @@ __global__ void __launch_bounds__(512) residual_streams_norm_kernel(StreamsArgs<
   const size_t orow = blockIdx.x, row = a.rows ? (size_t)a.rows[orow] : orow;
   if (a.delta)
     for (int i = threadIdx.x; i < n * (n + 1); i += blockDim.x) s_back[i] = a.back[i];
-  for (int i = threadIdx.x; i < n; i += blockDim.x) s_read[i] = a.read[i];
+  if constexpr (N == 1) {
+    if (threadIdx.x == 0) {
+      float r = 0.f;
+      for (int i = 0; i < a.n_read; ++i) r += a.read[i];
+      s_read[0] = r;
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) s_read[i] = a.read[i];
+  }
   __syncthreads();
   float sum = 0.f;
   for (int k = threadIdx.x * 8; k < a.H; k += blockDim.x * 8) {
@@ -137,7 +146,7 @@ int launch_streams(const StreamsArgs<A>& a, int T, cudaStream_t st) {
     MLORA_CHECK_LAUNCH("residual_streams_norm_kernel");
     return (int)MLORA_OK;
   };
-  switch (a.n) {
+  switch (!a.delta && a.src_stream == 0 ? 1 : a.n) {  // (untouched streams: one row, the sum of the weights)
     case 1: return go(residual_streams_norm_kernel<A, 1>);
     case 2: return go(residual_streams_norm_kernel<A, 2>);
     case 3: return go(residual_streams_norm_kernel<A, 3>);
@@ -166,7 +175,7 @@ extern "C" int mlora_residual_streams_layernorm(const void* d_delta, const float
   const auto launch = [&](auto zero) {
     using A = decltype(zero);
     StreamsArgs<A> a{(const A*)d_delta, d_src, ld_src, src_stream, d_dst, d_back, d_read, d_rows, (const bf16*)d_w, eps,
-                     (A*)d_out, n, H, width};
+                     (A*)d_out, n, n, H, width};
     return launch_streams(a, T, (cudaStream_t)stream);
   };
   return f32 ? launch(0.f) : launch(bf16());
