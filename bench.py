@@ -1071,8 +1071,8 @@ class KernelTimer:
 
     NAMES = ("linear", "grouped_linear", "moe_plan", "moe_route_plan", "residual_dyt", "residual_rmsnorm", "latent_append", "latent_gather",
              "latent_attention", "prefill_attention_dense", "embed", "argmax", "paged_attention", "prefill_attention",
-             "kv_append_rope", "paged_attention_masked", "prefill_attention_masked", "residual_streams_layernorm", "rotate_rms_append",
-             "short_conv", "delta_scan", "delta_chunk", "gated_rms", "delta_step")
+             "kv_append_rope", "paged_attention_masked", "paged_attention_rms", "prefill_attention_masked",
+             "residual_streams_layernorm", "rotate_rms_append", "short_conv", "delta_scan", "delta_chunk", "gated_rms", "delta_step")
 
     def __init__(self, ops, torch, dev, hbm_gbs, tflops):
         self.ops, self.torch, self.hbm, self.tflops = ops, torch, hbm_gbs, tflops
@@ -1113,6 +1113,9 @@ class KernelTimer:
             return f"{sum(news)} rows, {Hq} heads", 4 * D * Hkv * sum(lens) + 4 * D * Hq * sum(news), 4.0 * Hq * D * pairs
         if name in ("paged_attention_masked", "prefill_attention_masked"):  # (bench shapes: one chunk)
             Hq, (Hkv, _, D) = a[6], a[1].shape[1:]
+            return f"{sum(news)} rows, {Hq} heads", 4 * D * Hkv * sum(lens) + 4 * D * Hq * sum(news), 4.0 * Hq * D * pairs
+        if name == "paged_attention_rms":
+            Hq, (Hkv, _, D) = a[11], a[6].shape[1:]
             return f"{sum(news)} rows, {Hq} heads", 4 * D * Hkv * sum(lens) + 4 * D * Hq * sum(news), 4.0 * Hq * D * pairs
         if name == "residual_streams_layernorm":
             T, H, n = a[6].shape[0], a[6].shape[1], a[2].numel()

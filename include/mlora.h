@@ -541,6 +541,8 @@ int mlora_residual_streams_layernorm(const void* d_delta, const float* d_src, in
  *   mlora_prefill_attention with the scale of the scores as an argument (positive for the latter), `chunk` > 0: position i
  *   sees the positions j <= i with j / chunk == i / chunk only, and d_sink [Hq] (NULL: none): exp(sink[h]) is added to the
  *   sum of a head's softmax.  Prompt form: heads of 64 or 128, pages of a multiple of 16.
+ * mlora_paged_attention_rms: a decode step in one launch: mlora_rotate_rms_append of the rows' new tokens (bf16, dim <= D) and
+ *   mlora_paged_attention_masked over the pages and them.
  * mlora_paged_attention_any: the same for heads of up to 512, bf16 or fp32, on the CUDA cores, one query row per CTA. */
 int mlora_rotate_rms_append(const void* d_x, int64_t ld, const float* d_bias, const float* d_inv_freq, int32_t rot, int32_t dim,
                             int32_t pad, float eps, float q_scale, void* d_q, void* d_k_pages, void* d_v_pages,
@@ -551,6 +553,11 @@ int mlora_paged_attention_masked(const void* d_q, int64_t ld, const void* d_k_pa
                                  const int32_t* d_row_pos, int32_t T, int32_t Hq, int32_t Hkv, int32_t D, int32_t page_size,
                                  float scale, int32_t chunk, const float* d_sink, void* d_out, int64_t ld_out, int32_t n_splits,
                                  void* d_work, size_t work_bytes, void* stream);
+int mlora_paged_attention_rms(const void* d_x, int64_t ld, const float* d_bias, const float* d_inv_freq, int32_t rot, int32_t dim,
+                              float eps, void* d_k_pages, void* d_v_pages, const int32_t* d_block_table, int32_t max_pages,
+                              const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, int32_t Hq, int32_t Hkv, int32_t D,
+                              int32_t page_size, float scale, int32_t chunk, const float* d_sink, void* d_out, int64_t ld_out,
+                              int32_t n_splits, void* d_work, size_t work_bytes, void* stream);
 int mlora_prefill_attention_masked(const void* d_q, int64_t ld, const void* d_k_pages, const void* d_v_pages,
                                    int32_t n_pages_total, const int32_t* d_block_table, int32_t max_pages, const int32_t* d_tiles,
                                    int32_t n_tiles, int32_t Hq, int32_t Hkv, int32_t D, int32_t page_size, float scale,

@@ -100,6 +100,8 @@ PROTOTYPES = {
                                           _vp, _i32, _i32, _i32, _i32, _i32, _vp]),
     "mlora_paged_attention_masked": (C.c_int, [_vp, _i64, _vp, _vp, _vp, _i32, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _f32,
                                                _i32, _vp, _vp, _i64, _i32, _vp, _sz, _vp]),
+    "mlora_paged_attention_rms": (C.c_int, [_vp, _i64, _vp, _vp, _i32, _i32, _f32, _vp, _vp, _vp, _i32, _vp, _vp, _i32, _i32, _i32,
+                                            _i32, _i32, _f32, _i32, _vp, _vp, _i64, _i32, _vp, _sz, _vp]),
     "mlora_prefill_attention_masked": (C.c_int, [_vp, _i64, _vp, _vp, _i32, _vp, _i32, _vp, _i32, _i32, _i32, _i32, _i32,
                                                  _f32, _i32, _vp, _i32, _vp, _i64, _vp, _vp]),
     "mlora_paged_attention_any": (C.c_int, [_vp, _vp, _vp, _vp, _i32, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _f32, _i32, _vp,

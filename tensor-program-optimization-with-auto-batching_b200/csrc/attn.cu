@@ -36,6 +36,11 @@ struct AttnArgs {
   float qscale;        // of the scores, times log2(e)
   int chunk;           // > 0: a row sees only positions of its own chunk of this many (counted from position 0)
   const float* sink;   // [Hq] or NULL: a logit per head that only enters the softmax's sum
+  // instantiations with RMS: rows [q heads | k heads] of `dim` <= D columns, rotated and normalised here (mlora_rotate_rms_append)
+  const float* bias;      // [(Hq + Hkv) * dim] or NULL
+  const float* inv_freq;  // [rot / 2]
+  int rot, dim;
+  float eps;
   // optional: the LoRA shrink of the projection that reads `out` (o_proj), computed in this kernel's tail
   const bf16* sh_A;            // [N, sh_r, Hq*D] or nullptr
   const int32_t* sh_slots;     // [T]
@@ -76,8 +81,9 @@ __device__ __forceinline__ void merge_state(float& m, float& l, float (&acc)[8],
   m = mn;
 }
 
-// grid (Hq, T, n_splits), 128 threads.  IT = page_size / tokens-per-load.
-template <int D, int IT>
+// grid (Hq, T, n_splits), 128 threads.  IT = page_size / tokens-per-load.  RMS: with the new token's bias, rotation and norm in
+// the prologue, and its key before those as its value.
+template <int D, int IT, bool RMS>
 __global__ void __launch_bounds__(128) paged_attn_kernel(AttnArgs a) {
   constexpr int LPT = D / 8;    // lanes per token
   constexpr int TPW = 32 / LPT; // tokens per warp-wide load
@@ -105,7 +111,42 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(AttnArgs a) {
   const bool can_store = pos >= 0 && pos / PS < a.max_pages;
 
   // ---- prologue: rotate q (and the new k), stage the new k/v -----------------------------------
-  if (tid < D / 2) {
+  if constexpr (RMS) {
+    __shared__ float s_sum[2][4];
+    const int half = a.rot / 2, d = tid;
+    float qy = 0.f, ky = 0.f, kx = 0.f;
+    if (d < a.dim) {
+      const int o = d < half ? d + half : d - half;  // the column it is paired with, if it is rotated
+      const auto value = [&](int head, int c) {
+        return __bfloat162float(row[(size_t)head * a.dim + c]) + (a.bias ? a.bias[(size_t)head * a.dim + c] : 0.f);
+      };
+      qy = value(h, d);
+      kx = ky = value(a.Hq + kvh, d);
+      if (d < a.rot) {
+        float sn, cs;
+        sincosf((float)pos * a.inv_freq[d < half ? d : o], &sn, &cs);
+        if (d < half) sn = -sn;
+        qy = fmaf(qy, cs, value(h, o) * sn);
+        ky = fmaf(ky, cs, value(a.Hq + kvh, o) * sn);
+      }
+    }
+    const float q2 = warp_sum(qy * qy), k2 = warp_sum(ky * ky);
+    if (lane == 0) s_sum[0][warp] = q2, s_sum[1][warp] = k2;
+    __syncthreads();
+    const float nq = (s_sum[0][0] + s_sum[0][1]) + (s_sum[0][2] + s_sum[0][3]);
+    const float nk = (s_sum[1][0] + s_sum[1][1]) + (s_sum[1][2] + s_sum[1][3]);
+    if (d < D) {
+      const bf16 kr = __float2bfloat16_rn(ky * (1.f / sqrtf(nk / (float)a.dim + a.eps))), vr = __float2bfloat16_rn(kx);
+      sq[d] = qy * (1.f / sqrtf(nq / (float)a.dim + a.eps)) * qscale;
+      sk[d] = __bfloat162float(kr);
+      sv[d] = __bfloat162float(vr);
+      if (has_new && h % rep == 0 && can_store) {
+        const size_t at = (((size_t)bt[pos / PS] * a.Hkv + kvh) * PS + pos % PS) * D + d;
+        a.k_pages[at] = kr;
+        a.v_pages[at] = vr;
+      }
+    }
+  } else if (tid < D / 2) {
     const int i = tid;
     float q1 = __bfloat162float(row[h * D + i]), q2 = __bfloat162float(row[h * D + i + D / 2]);
     if (a.fused) {
@@ -132,7 +173,7 @@ __global__ void __launch_bounds__(128) paged_attn_kernel(AttnArgs a) {
       dst[i + D / 2] = r2;
     }
   }
-  if (has_new && tid < D) {
+  if (!RMS && has_new && tid < D) {
     const bf16 v = row[(size_t)(a.Hq + a.Hkv + kvh) * D + tid];
     sv[tid] = __bfloat162float(v);
     if (h % rep == 0 && can_store) {
@@ -445,13 +486,20 @@ struct Softmax {
   int chunk = 0;
   const float* sink = nullptr;
 };
+// Bias, rotation and norm of the new tokens (see mlora_paged_attention_rms); dim 0: none of it.
+struct NewToken {
+  const float* bias = nullptr;
+  const float* inv_freq = nullptr;
+  int rot = 0, dim = 0;
+  float eps = 0.f;
+};
 
 static int attention_impl(const void* d_qkv, int64_t ld, void* d_k_pages, void* d_v_pages,
                           const int32_t* d_block_table, int32_t max_pages, const int32_t* d_row_slot,
                           const int32_t* d_row_pos, int32_t T, int32_t Hq, int32_t Hkv, int32_t D,
                           int32_t page_size, float rope_theta, int32_t fused_append, void* d_out,
                           int64_t ld_out, int32_t n_splits, void* d_work, size_t work_bytes,
-                          void* stream, const ShrinkTail& sh, const Softmax& sm) {
+                          void* stream, const ShrinkTail& sh, const Softmax& sm, const NewToken& nt = NewToken{}) {
   int rc = check_kv_common("paged_attention", T, Hq, Hkv, D, page_size);
   if (rc) return rc;
   MLORA_REQUIRE(d_qkv && d_k_pages && d_v_pages && d_block_table && d_row_slot && d_row_pos && d_out && max_pages > 0,
@@ -471,17 +519,18 @@ static int attention_impl(const void* d_qkv, int64_t ld, void* d_k_pages, void* 
   }
   AttnArgs a{(const bf16*)d_qkv, ld, (bf16*)d_k_pages, (bf16*)d_v_pages, d_block_table, max_pages, d_row_slot,
              d_row_pos, T, Hq, Hkv, page_size, rope_theta, fused_append ? 1 : 0, (bf16*)d_out, ld_out, n_splits,
-             (float*)d_work, sm.scale * kLog2e, sm.chunk, sm.sink, (const bf16*)sh.A, sh.slots, sh.n_adapters, sh.r, sh.u, sh.part, sh.tickets};
+             (float*)d_work, sm.scale * kLog2e, sm.chunk, sm.sink, nt.bias, nt.inv_freq, nt.rot, nt.dim, nt.eps, (const bf16*)sh.A, sh.slots, sh.n_adapters, sh.r, sh.u, sh.part, sh.tickets};
   dim3 grid(Hq, T, n_splits);
   cudaStream_t st = (cudaStream_t)stream;
+  const auto go = [&](auto plain, auto rms) { launch_pdl_if(pdl_enabled_attn(), nt.dim ? rms : plain, grid, 128, 0, st, a); };
   if (D == 128 && page_size == 16)
-    launch_pdl_if(pdl_enabled_attn(), paged_attn_kernel<128, 8>, grid, 128, 0, st, a);
+    go(paged_attn_kernel<128, 8, false>, paged_attn_kernel<128, 8, true>);
   else if (D == 128 && page_size == 32)
-    launch_pdl_if(pdl_enabled_attn(), paged_attn_kernel<128, 16>, grid, 128, 0, st, a);
+    go(paged_attn_kernel<128, 16, false>, paged_attn_kernel<128, 16, true>);
   else if (D == 64 && page_size == 16)
-    launch_pdl_if(pdl_enabled_attn(), paged_attn_kernel<64, 4>, grid, 128, 0, st, a);
+    go(paged_attn_kernel<64, 4, false>, paged_attn_kernel<64, 4, true>);
   else
-    launch_pdl_if(pdl_enabled_attn(), paged_attn_kernel<64, 8>, grid, 128, 0, st, a);
+    go(paged_attn_kernel<64, 8, false>, paged_attn_kernel<64, 8, true>);
   count_launch();
   if (n_splits > 1) {
     launch_pdl_if(pdl_enabled_attn(), attn_merge_kernel, dim3(Hq, T), D, 0, st, (const float*)d_work, Hq, D, n_splits, (bf16*)d_out, ld_out);
@@ -511,6 +560,20 @@ extern "C" int mlora_paged_attention_masked(const void* d_q, int64_t ld, const v
   return attention_impl(d_q, ld, (void*)d_k_pages, (void*)d_v_pages, d_block_table, max_pages, d_row_slot, d_row_pos, T, Hq,
                         Hkv, D, page_size, 1.f, 0, d_out, ld_out, n_splits, d_work, work_bytes, stream, ShrinkTail{},
                         Softmax{scale, chunk, d_sink});
+}
+
+extern "C" int mlora_paged_attention_rms(const void* d_x, int64_t ld, const float* d_bias, const float* d_inv_freq, int32_t rot,
+                                         int32_t dim, float eps, void* d_k_pages, void* d_v_pages, const int32_t* d_block_table,
+                                         int32_t max_pages, const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T,
+                                         int32_t Hq, int32_t Hkv, int32_t D, int32_t page_size, float scale, int32_t chunk,
+                                         const float* d_sink, void* d_out, int64_t ld_out, int32_t n_splits, void* d_work,
+                                         size_t work_bytes, void* stream) {
+  MLORA_REQUIRE(chunk >= 0 && dim > 0 && dim <= D && rot >= 0 && rot % 2 == 0 && rot <= dim && (!rot || d_inv_freq) &&
+                    ld >= (int64_t)(Hq + Hkv) * dim,
+                "paged_attention_rms: bad chunk, head size or rotation");
+  return attention_impl(d_x, ld, d_k_pages, d_v_pages, d_block_table, max_pages, d_row_slot, d_row_pos, T, Hq, Hkv, D, page_size,
+                        1.f, 1, d_out, ld_out, n_splits, d_work, work_bytes, stream, ShrinkTail{}, Softmax{scale, chunk, d_sink},
+                        NewToken{d_bias, d_inv_freq, rot, dim, eps});
 }
 
 extern "C" uint32_t mlora_paged_attention_splits(int32_t T, int32_t Hq, int32_t max_pages) {

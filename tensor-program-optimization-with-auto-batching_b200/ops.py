@@ -684,12 +684,29 @@ def rotate_rms_append(x, bias, inv_freq, rot, dim, eps, q_scale, q_out, k_pages,
     return q_out
 
 
+def paged_attention_streams(dtype, D, page_size) -> bool:
+    """Heads and pages the streaming kernel takes; the plain one takes everything."""
+    return dtype == torch.bfloat16 and D in (64, 128) and page_size in (16, 32)
+
+
+def paged_attention_rms(x, bias, inv_freq, rot, dim, eps, k_pages, v_pages, block_table, row_slot, row_pos, Hq, scale, out, chunk=0,
+                        sink=None, n_splits=0, work=None):
+    """:func:`rotate_rms_append` of one new token per row and the attention over its context in one launch."""
+    _need_cuda(x, k_pages)
+    Hkv, ps, D = k_pages.shape[1:]
+    check(_lib.lib().mlora_paged_attention_rms(
+        _ptr(x), x.stride(0), _ptr(bias), _ptr(inv_freq), rot, dim, eps, _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
+        block_table.shape[1], _ptr(row_slot), _ptr(row_pos), x.shape[0], Hq, Hkv, D, ps, scale, chunk, _ptr(sink), _ptr(out),
+        out.stride(0), n_splits, _ptr(work), work.numel() if work is not None else 0, _stream()), "mlora_paged_attention_rms")
+    return out
+
+
 def paged_attention_masked(q, k_pages, v_pages, block_table, row_slot, row_pos, Hq, scale, out, chunk=0, sink=None, n_splits=0,
                            work=None):
     """One query row per (row, head); bf16 heads of 64 and 128 stream whole pages, everything else runs the plain kernel."""
     _need_cuda(q, k_pages)
     T, (Hkv, ps, D) = q.shape[0], k_pages.shape[1:]
-    if q.dtype == torch.float32 or D not in (64, 128) or ps not in (16, 32):
+    if not paged_attention_streams(q.dtype, D, ps):
         check(_lib.lib().mlora_paged_attention_any(
             _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], _ptr(row_slot), _ptr(row_pos), T, Hq, Hkv,
             D, ps, scale, chunk, _ptr(sink), _ptr(out), out.stride(0), int(q.dtype == torch.float32), _stream()),

@@ -260,6 +260,13 @@ class RelidraEngine(PlainEngine):
     def _attention(self, T, lw, run, proj, out, decode):
         kv, mix, eps = self.kv, lw.mix, self.m.config.eps
         row_slot, row_pos, K, V = self.row_slot[:T], self.row_pos[:T], kv.k_pages(run), kv.v_pages(run)
+        if decode and ops.paged_attention_streams(self.m.dtype, lw.pad, kv.page_size):
+            keys = min(self.max_keys, mix.chunk) if mix.chunk else self.max_keys
+            splits = ops.paged_attention_splits(T, mix.heads, -(-keys // kv.page_size) + 1)
+            nb = ops.paged_attention_workspace(T, mix.heads, lw.pad, splits) if splits > 1 else 0
+            return ops.paged_attention_rms(proj, lw.bias, lw.inv_freq, mix.rot, mix.dim, eps, K, V, kv.block_table, row_slot, row_pos,
+                                           mix.heads, mix.scale, out, chunk=mix.chunk, sink=lw.sink, n_splits=splits,
+                                           work=self._grow("merge", nb, torch.uint8) if nb else None)
         q = ops.rotate_rms_append(proj, lw.bias, lw.inv_freq, mix.rot, mix.dim, eps, mix.scale,
                                   self.q[:T * lw.out_cols].view(T, lw.out_cols), K, V, kv.block_table, row_slot, row_pos, mix.heads,
                                   mix.kv_heads)
@@ -267,11 +274,8 @@ class RelidraEngine(PlainEngine):
             return ops.prefill_attention_masked(q, K, V, kv.block_table, self.tiles, self._n_tiles, mix.heads, 1.0, out,
                                                 chunk=mix.chunk, sink=lw.sink, status=self.status)
         # (the scale is in the queries)
-        keys = min(self.max_keys, mix.chunk) if mix.chunk else self.max_keys
-        splits = ops.paged_attention_splits(T, mix.heads, -(-keys // kv.page_size) + 1)
-        nb = ops.paged_attention_workspace(T, mix.heads, lw.pad, splits) if splits > 1 else 0
         return ops.paged_attention_masked(q, K, V, kv.block_table, row_slot, row_pos, mix.heads, 1.0, out, chunk=mix.chunk,
-                                          sink=lw.sink, n_splits=splits, work=self._grow("merge", nb, torch.uint8) if nb else None)
+                                          sink=lw.sink)
 
     def _norm(self, T, w, read, src, add, rows=None):
         """Hands ``add`` = (rows, connection of the sublayer they come from) back to the streams and normalises the sum that

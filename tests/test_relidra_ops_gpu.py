@@ -158,6 +158,32 @@ def test_chunked_attention_with_sinks(ops, cuda, Hq, Hkv, D, page, chunk, n):
             close(out.view(n, Hq, D), want, BF)
 
 
+@pytest.mark.parametrize("Hq,Hkv,dim,rot,pad,page,chunk", [(4, 2, 36, 20, 64, 16, 23), (5, 1, 72, 72, 128, 32, 40), (8, 2, 128, 64, 128, 16, 0),
+                                                           (2, 2, 64, 0, 64, 32, 64), (1, 1, 64, 64, 64, 16, 7)])
+@pytest.mark.parametrize("splits", [1, 4])
+def test_decode_attention_in_one_launch(ops, cuda, Hq, Hkv, dim, rot, pad, page, chunk, splits):
+    """Token by token: rotation, norm, append and attention in one launch against the oracle over the whole sequence."""
+    n, g = 90, gen(dim + chunk)
+    x = torch.randn(n, (Hq + Hkv) * dim, generator=g).to(BF)
+    bias, sink = torch.randn((Hq + Hkv) * dim, generator=g), torch.randn(Hq, generator=g) + 2
+    freq = torch.tensor([500.0 ** (-2.0 * i / max(rot, 1)) / 2.0 for i in range(rot // 2)], dtype=torch.float64)
+    bt, n_pages = _table(g, 2, 10, cuda)
+    K, V = (torch.full((n_pages, Hkv, page, pad), float("nan"), dtype=BF, device=cuda) for _ in range(2))
+    scale = 3.0 / dim ** 0.5
+    work = torch.zeros(max(ops.paged_attention_workspace(2, Hq, pad, splits), 16), dtype=torch.uint8, device=cuda)
+    got = []
+    for t in range(n):  # (a second row is padding: it stores nothing)
+        out = torch.full((2, Hq * pad), float("nan"), dtype=BF, device=cuda)
+        ops.paged_attention_rms(x[[t, t]].to(cuda), bias.to(cuda), freq.float().to(cuda), rot, dim, 1e-3, K, V, bt, i32([1, 0], cuda),
+                                i32([t, -1], cuda), Hq, scale, out, chunk=chunk, sink=sink.to(cuda), n_splits=splits, work=work)
+        got.append(out[0].view(Hq, pad))
+    assert not torch.stack(got)[..., dim:].any()
+    xb = (x.double() + bias.double()).view(n, Hq + Hkv, dim)
+    y = orl.rms(orl.rotate(xb, torch.arange(n), rot, 500.0, 2.0), 1e-3)
+    close(torch.stack(got)[..., :dim], _attention_want(y[:, :Hq], y[:, Hq:], xb[:, Hq:], chunk, sink, scale), BF)
+    assert K[bt[0].long()].isnan().all()
+
+
 @pytest.mark.parametrize("dtype", [BF, F32])
 @pytest.mark.parametrize("Hq,Hkv,D,page,chunk,n", [(4, 2, 40, 16, 23, 90), (2, 1, 144, 32, 70, 150), (1, 1, 512, 16, 0, 40), (3, 3, 8, 16, 5, 60)])
 def test_plain_attention_kernel(ops, cuda, dtype, Hq, Hkv, D, page, chunk, n):
