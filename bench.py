@@ -803,6 +803,8 @@ def run_kernel_case(which):
         return run_operator_case(ops, synth, dev, torch)
     if which in ("latent", "experts"):
         return run_tevudra_kernel_case(which, ops, dev, torch)
+    if which in ("delta-step", "delta-chunk"):
+        return run_delta_kernel_case(which, ops, dev, torch)
     if which == "linear":
         # the q/k/v projection of one layer with its LoRA stack: 4 weight copies = 403 MB
         c = synth.operator_case(T, 4096, 12288, N_ADAPTERS, RANK, device=dev)
@@ -1317,6 +1319,37 @@ def run_tevudra_kernel_case(which, ops, dev, torch):
         fn = lambda: ops.grouped_linear(x, weight, y, plan=plan, gather=True, flags=ops.ACT_GELU, work=work)
         used = len(set(plan.expert[:T * top].tolist()))
         by = 2 * (used * W * ff + x.numel() + y.numel())
+    time_kernel_case(which, fn, by, ops, torch)
+
+
+def run_delta_kernel_case(which, ops, dev, torch):
+    """32 heads of 128 x 128 over 16 key heads, 4 taps.  delta-step: one token of 64 rows (134 MB of states); delta-chunk: 4
+    sequences of 1024 tokens.  A few launches, then CUDA-event time."""
+    heads, kv, d, taps = 32, 16, 128, 4
+    n_seq, n = (64, 1) if which == "delta-step" else (4, 1024)
+    T, C, g = n_seq * n, 2 * kv * d + heads * d, torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *s: torch.randn(*s, generator=g, device=dev)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    r = ops.DeltaRule(heads, kv, d, d, d, taps, d ** -0.5, C, C + heads * d, C + heads * d + heads, rnd(taps, C) / 2,
+                      rnd(heads) - 2, rnd(heads) - 2, torch.ones(d, device=dev))
+    x, ring = rnd(T, C + heads * d + 2 * heads).to(torch.bfloat16), rnd(n_seq, taps, C).to(torch.bfloat16)
+    S, status = rnd(n_seq, heads, d, d) / 100, i32([0])
+    slots, pos = i32([s for s in range(n_seq) for _ in range(n)]), i32([100 + t for _ in range(n_seq) for t in range(n)])
+    if which == "delta-step":
+        out = torch.empty(T, heads * d, dtype=torch.bfloat16, device=dev)
+        fn = lambda: ops.delta_step(x, r, 1e-6, slots, pos, S, ring, out)
+        by = T * (8 * heads * d * d + 2 * (taps + 1) * C + 4 * heads * d)
+    else:
+        segs, o = i32([[s, s * n, n, 100] for s in range(n_seq)]), torch.empty(T, heads * d, device=dev)
+        xc = ops.short_conv(x, r.conv, ring, slots, pos, torch.empty(T, C, dtype=torch.bfloat16, device=dev))
+        work = ops.new_workspace(ops.delta_chunk_workspace(T, n_seq, heads), dev)
+        fn = lambda: ops.delta_chunk(xc, x, r, segs, n_seq, n, S, ring, o, work, status)
+        by = 2 * xc.numel() + 4 * o.numel() + 8 * S.numel()
+    time_kernel_case(which, fn, by, ops, torch)
+    assert not int(status)
+
+
+def time_kernel_case(which, fn, by, ops, torch):
     for _ in range(5):
         fn()
     e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
@@ -1363,7 +1396,7 @@ def main():
                     help="profiling aid: fill the KV cache with seeded random values instead of running prefill "
                          "(the number is then not a bench value)")
     ap.add_argument("--kernel-case", default="", choices=["", "linear", "attention", "operator", "prefill", "prefill-lora", "prefill-attn", "expand", "chain",
-                                                               "latent", "experts"],
+                                                               "latent", "experts", "delta-step", "delta-chunk"],
                     help="profiling aid: launch one kernel a few times on a small case (> L2, < 1 GB) and exit")
     ap.add_argument("--workload", default="", choices=["", "13b-shape", "13b-tp", "prefill-heavy", "tevudra", "relidra"],
                     help="side measurements (own JSON line, not the benchmark's): 13b-shape = the 13B shape and adapter "

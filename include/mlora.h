@@ -585,7 +585,8 @@ int mlora_paged_attention_any(const void* d_q, const void* d_k_pages, const void
  *   bf16 planes, so results agree to fp32 rounding).  T = rows of x and xc, max_rows = rows of the longest segment; d_work:
  *   mlora_delta_chunk_workspace bytes; d_status as for mlora_prefill_attention.
  * mlora_gated_rms: out = o / sqrt(mean(o^2) + eps) * w * silu(gate) per head (mean over the first vdim_true columns).
- * mlora_delta_step: everything for one new token per row (gate from column g_col); rows with row_pos < 0 give zeros. */
+ * mlora_delta_step: everything for one new token per row (gate from column g_col); rows with row_pos < 0 give zeros.
+ *   d_status as above. */
 int mlora_short_conv(const void* d_x, int64_t ld, int32_t C, int32_t taps, const float* d_w, const void* d_ring,
                      const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, void* d_out, int32_t f32, void* stream);
 int mlora_delta_scan(const void* d_xc, const void* d_x, int64_t ld, int32_t C, int32_t taps, int32_t b_col, int32_t a_col,
@@ -603,7 +604,7 @@ int mlora_delta_step(const void* d_x, int64_t ld, int32_t C, int32_t taps, int32
                      const float* d_conv, const float* d_A_log, const float* d_dt_bias, const float* d_norm_w, float eps,
                      int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t vdim_true, float q_scale,
                      const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, float* d_state, void* d_ring, void* d_out,
-                     int32_t f32, void* stream);
+                     int32_t* d_status, int32_t f32, void* stream);
 
 #ifdef __cplusplus
 }

@@ -114,7 +114,7 @@ PROTOTYPES = {
                                     _i32, _i32, _vp, _vp, _vp, _vp, _sz, _vp, _vp]),
     "mlora_gated_rms": (C.c_int, [_vp, _vp, _i64, _vp, _i32, _i32, _i32, _i32, _f32, _vp, _i32, _vp]),
     "mlora_delta_step": (C.c_int, [_vp, _i64, _i32, _i32, _i32, _i32, _i32, _vp, _vp, _vp, _vp, _f32, _i32, _i32, _i32, _i32,
-                                   _i32, _f32, _vp, _vp, _i32, _vp, _vp, _vp, _i32, _vp]),
+                                   _i32, _f32, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _vp]),
     "mlora_decode_step_begin": (C.c_int, [_vp, _vp, _vp, _vp, _i32, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),
     "mlora_decode_step_end": (C.c_int, [_vp, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _vp, _vp]),
 }

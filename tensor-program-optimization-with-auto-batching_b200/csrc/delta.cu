@@ -22,6 +22,7 @@
 #include <cmath>
 
 #include "delta.cuh"
+#include "tc_ptx.cuh"
 
 namespace mlora {
 namespace {
@@ -412,9 +413,172 @@ struct StepArgs {
   float* state;
   A* ring;
   A* out;            // [T, heads * vdim]
+  int32_t* status;
 };
 
-// CTA (head, row): eight warps = 128 columns at a time.
+// Convolution and silu of one head's channels of a new token: out = q [rows] | k [rows] | v [vdim], zero past dim; the token's
+// inputs go to the ring (those of q and k by the first head that uses them).
+template <typename A>
+__device__ __forceinline__ void step_conv(const StepArgs<A>& a, const A* row, A* ring, int h, int pos, int rows, float* out) {
+  const int tid = threadIdx.x, threads = blockDim.x, rep = a.d.heads / a.d.kv_heads, kh = h / rep;
+  const int q_col = kh * a.d.dim, k_col = (a.d.kv_heads + kh) * a.d.dim, v_col = 2 * a.d.kv_heads * a.d.dim + h * a.d.vdim;
+  // convolutions: everything two channels need is requested before the first use
+  const int total = 2 * rows + a.d.vdim, back = min(a.taps - 1, pos), now = pos % a.taps;
+  for (int i0 = tid; i0 < total; i0 += 2 * threads) {
+    float w[2][kMaxTaps], x[2][kMaxTaps];
+    A cur[2];
+    int chan[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = i0 + u * threads, part = i < rows ? 0 : i < 2 * rows ? 1 : 2, e = i - part * rows;
+      const bool there = i < total && (part == 2 || e < a.d.dim);
+      chan[u] = there ? (part == 0 ? q_col : part == 1 ? k_col : v_col) + e : -1;
+#pragma unroll
+      for (int j = 0; j < kMaxTaps; ++j) {
+        w[u][j] = x[u][j] = 0.f;
+        if (!there || j > back) continue;
+        const int at = now - j < 0 ? now - j + a.taps : now - j;
+        w[u][j] = a.conv[(size_t)(a.taps - 1 - j) * a.C + chan[u]];
+        if (j == 0)
+          cur[u] = row[chan[u]];
+        else
+          x[u][j] = to_f32(ring[(size_t)at * a.C + chan[u]]);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = i0 + u * threads;
+      if (i >= total) break;
+      float val = 0.f;
+      if (chan[u] >= 0) {
+        float sum = 0.f;
+#pragma unroll
+        for (int j = kMaxTaps - 1; j > 0; --j) sum = fmaf(w[u][j], x[u][j], sum);
+        val = silu<float>(fmaf(w[u][0], to_f32(cur[u]), sum));
+        if (i >= 2 * rows || h % rep == 0) ring[(size_t)now * a.C + chan[u]] = cur[u];
+      }
+      out[i] = val;
+    }
+  }
+}
+
+// CTA (head, row), the state in shared memory: one bulk copy in, one out.  Threads over the columns, several parts of the rows.
+template <typename A>
+__global__ void __launch_bounds__(256, 3) delta_step_bulk_kernel(StepArgs<A> a) {
+  extern __shared__ __align__(16) float smem[];
+  const DeltaDims d = a.d;
+  float* s_S = smem;                   // [dim][vdim]
+  float* s_q = s_S + d.dim * d.vdim;   // [dim]
+  float* s_k = s_q + d.dim;            // [dim]
+  float* s_v = s_k + d.dim;            // [vdim], then the outputs
+  float2* s_part = reinterpret_cast<float2*>(s_v + d.vdim);  // [256]
+  __shared__ uint64_t bar;
+  __shared__ float s_kq;
+  __shared__ int s_abort;
+  pdl_launch_dependents();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int h = blockIdx.x, t = blockIdx.y;
+  if (tid == 0) {
+    s_abort = 0;
+    mbar_init(&bar, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  pdl_wait();
+  const int slot = a.row_slot[t], pos = a.row_pos[t];
+  A* out = a.out + ((size_t)t * d.heads + h) * d.vdim;
+  if (pos < 0) {  // padding row
+    for (int i = tid; i < d.vdim; i += 256) out[i] = from_f32<A>(0.f);
+    return;
+  }
+  float* S = a.state + ((size_t)slot * d.heads + h) * d.dim * d.vdim;
+  const uint32_t bytes = (uint32_t)(d.dim * d.vdim) * 4;
+  if (pos > 0) {
+    if (tid == 0) {
+      mbar_expect_tx(&bar, bytes);
+      bulk_load(s_S, S, bytes, &bar);
+    }
+  } else {
+    for (int i = tid; i < d.dim * d.vdim; i += 256) s_S[i] = 0.f;
+  }
+  const A* row = a.x + (size_t)t * a.ld;
+  const float beta = step_size(to_f32(row[a.b_col + h])), g = expf(log_decay(to_f32(row[a.a_col + h]), a.A_log[h], a.dt_bias[h]));
+  step_conv(a, row, a.ring + (size_t)slot * a.taps * a.C, h, pos, d.dim, s_q);
+  __syncthreads();
+  if (warp == 0) {  // unit vectors, their product
+    float sq = 0.f, sk = 0.f, sx = 0.f;
+    for (int i = lane; i < d.dim; i += 32) {
+      const float q = s_q[i], k = s_k[i];
+      sq = fmaf(q, q, sq), sk = fmaf(k, k, sk), sx = fmaf(q, k, sx);
+    }
+    sq = warp_sum(sq), sk = warp_sum(sk), sx = warp_sum(sx);
+    const float iq = d.q_scale / sqrtf(sq + 1e-6f), ik = 1.f / sqrtf(sk + 1e-6f);
+    for (int i = lane; i < d.dim; i += 32) s_q[i] *= iq, s_k[i] *= ik;
+    if (lane == 0) s_kq = sx * iq * ik;
+  }
+  const bool ok = pos == 0 || mbar_wait(&bar, 0, &s_abort);
+  if (__syncthreads_or(!ok)) {  // gave up: nothing is written, the copy gets another bounded chance to land
+    if (tid == 0) {
+      if (a.status) atomicOr(a.status, 1);
+      mbar_wait(&bar, 0, &s_abort);
+    }
+    __syncthreads();
+    return;
+  }
+  const int width = min((d.vdim + 31) / 32 * 32, 256), parts = 256 / width, col = tid % width, part = tid / width;
+  const int per = (d.dim / 4 + parts - 1) / parts * 4, r0 = min(part * per, d.dim), r1 = min(r0 + per, d.dim);
+  const bool works = part < parts;
+  for (int c0 = 0; c0 < d.vdim; c0 += width) {
+    const int v = c0 + col;
+    float dk = 0.f, dq = 0.f, o = 0.f;
+    if (works && v < d.vdim) {
+#pragma unroll 4
+      for (int r = r0; r < r1; r += 4) {
+        const float4 k = *reinterpret_cast<const float4*>(s_k + r), q = *reinterpret_cast<const float4*>(s_q + r);
+        const float a0 = s_S[r * d.vdim + v], a1 = s_S[(r + 1) * d.vdim + v], a2 = s_S[(r + 2) * d.vdim + v], a3 = s_S[(r + 3) * d.vdim + v];
+        dk = fmaf(a0, k.x, dk), dq = fmaf(a0, q.x, dq);
+        dk = fmaf(a1, k.y, dk), dq = fmaf(a1, q.y, dq);
+        dk = fmaf(a2, k.z, dk), dq = fmaf(a2, q.z, dq);
+        dk = fmaf(a3, k.w, dk), dq = fmaf(a3, q.w, dq);
+      }
+    }
+    s_part[tid] = make_float2(dk, dq);
+    __syncthreads();
+    if (works && v < d.vdim) {
+      dk = dq = 0.f;
+      for (int p = 0; p < parts; ++p) {
+        const float2 x = s_part[p * width + col];
+        dk += x.x, dq += x.y;
+      }
+      const float u = beta * (s_v[v] - g * dk);
+      o = fmaf(u, s_kq, g * dq);
+#pragma unroll 4
+      for (int r = r0; r < r1; r += 4) {
+        const float4 k = *reinterpret_cast<const float4*>(s_k + r);
+        float* x = s_S + r * d.vdim + v;
+        x[0] = fmaf(k.x, u, g * x[0]);
+        x[d.vdim] = fmaf(k.y, u, g * x[d.vdim]);
+        x[2 * d.vdim] = fmaf(k.z, u, g * x[2 * d.vdim]);
+        x[3 * d.vdim] = fmaf(k.w, u, g * x[3 * d.vdim]);
+      }
+    }
+    __syncthreads();  // (everybody has read the value and the partial sums)
+    if (part == 0 && v < d.vdim) s_v[v] = o;
+  }
+  asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+  __syncthreads();
+  if (tid == 0) {
+    asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(S), "r"(smem_u32(s_S)), "r"(bytes) : "memory");
+    asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+  }
+  float ss = 0.f;
+  for (int i = lane; i < d.vdim; i += 32) ss = fmaf(s_v[i], s_v[i], ss);
+  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)d.vdim_true + a.eps);
+  for (int i = tid; i < d.vdim; i += 256)
+    out[i] = from_f32<A>(s_v[i] * inv * a.norm_w[i] * silu<A>(to_f32(row[a.g_col + h * d.vdim + i])));
+  if (tid == 0) bulk_wait_all0();
+}
+
+// CTA (head, row), for states beyond shared memory: the tile in registers, eight warps = 128 columns at a time.
 template <typename A, int RJ>
 __global__ void __launch_bounds__(256) delta_step_kernel(StepArgs<A> a) {
   constexpr int kRows = 32 * RJ;
@@ -443,23 +607,8 @@ __global__ void __launch_bounds__(256) delta_step_kernel(StepArgs<A> a) {
     tile.zero();
   const A* row = a.x + (size_t)t * a.ld;
   A* ring = a.ring + (size_t)slot * a.taps * a.C;
-  const int q_col = kh * d.dim, k_col = (d.kv_heads + kh) * d.dim, v_col = 2 * d.kv_heads * d.dim + h * d.vdim;
   const float beta = step_size(to_f32(row[a.b_col + h])), g = expf(log_decay(to_f32(row[a.a_col + h]), a.A_log[h], a.dt_bias[h]));
-  for (int i = tid; i < 2 * kRows + d.vdim; i += threads) {
-    const int part = i < kRows ? 0 : i < 2 * kRows ? 1 : 2, e = i - part * kRows;
-    float val = 0.f;
-    if (part == 2 || e < d.dim) {
-      const int ch = (part == 0 ? q_col : part == 1 ? k_col : v_col) + e;
-      const A cur = row[ch];
-      float s = 0.f;
-      for (int j = min(a.taps - 1, pos); j > 0; --j)
-        s = fmaf(a.conv[(size_t)(a.taps - 1 - j) * a.C + ch], to_f32(ring[(size_t)((pos - j) % a.taps) * a.C + ch]), s);
-      s = fmaf(a.conv[(size_t)(a.taps - 1) * a.C + ch], to_f32(cur), s);
-      if (part == 2 || h % rep == 0) ring[(size_t)(pos % a.taps) * a.C + ch] = cur;
-      val = silu<float>(s);
-    }
-    smem[i] = val;
-  }
+  step_conv(a, row, ring, h, pos, kRows, smem);
   __syncthreads();
   ulonglong2 k[RJ], q[RJ];
   float sq = 0.f, sk = 0.f, sx = 0.f;
@@ -630,7 +779,7 @@ extern "C" int mlora_delta_step(const void* d_x, int64_t ld, int32_t C, int32_t 
                                 const float* d_conv, const float* d_A_log, const float* d_dt_bias, const float* d_norm_w, float eps,
                                 int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t vdim_true, float q_scale,
                                 const int32_t* d_row_slot, const int32_t* d_row_pos, int32_t T, float* d_state, void* d_ring,
-                                void* d_out, int32_t f32, void* stream) {
+                                void* d_out, int32_t* d_status, int32_t f32, void* stream) {
   const DeltaDims d{heads, kv_heads, dim, vdim, vdim_true, q_scale};
   const int rc = check_delta_dims("delta_step", d, C, taps);
   if (rc) return rc;
@@ -645,10 +794,16 @@ extern "C" int mlora_delta_step(const void* d_x, int64_t ld, int32_t C, int32_t 
   const auto launch = [&](auto zero) {
     using A = decltype(zero);
     StepArgs<A> a{(const A*)d_x, ld, C, taps, g_col, b_col, a_col, d_conv, d_A_log, d_dt_bias, d_norm_w, eps, d, d_row_slot,
-                  d_row_pos, d_state, (A*)d_ring, (A*)d_out};
+                  d_row_pos, d_state, (A*)d_ring, (A*)d_out, d_status};
     const auto go = [&](auto kernel, int rj) {
       launch_pdl_if(pdl_enabled_attn(), kernel, dim3(heads, T), warps * 32, (size_t)(64 * rj + 2 * vdim) * 4, (cudaStream_t)stream, a);
     };
+    const size_t bulk = ((size_t)dim * vdim + 2 * dim + vdim + 512) * 4;
+    if (bulk <= 200 * 1024) {
+      if (bulk > 48 * 1024) cudaFuncSetAttribute(delta_step_bulk_kernel<A>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bulk);
+      launch_pdl_if(pdl_enabled_attn(), delta_step_bulk_kernel<A>, dim3(heads, T), 256, bulk, (cudaStream_t)stream, a);
+      return;
+    }
     if (dim <= 32) go(delta_step_kernel<A, 1>, 1);
     else if (dim <= 64) go(delta_step_kernel<A, 2>, 2);
     else if (dim <= 128) go(delta_step_kernel<A, 4>, 4);

@@ -809,10 +809,10 @@ def gated_rms(o, gate, w, heads, vdim_true, eps, out):
     return out
 
 
-def delta_step(x, r: DeltaRule, eps, row_slot, row_pos, state, ring, out):
+def delta_step(x, r: DeltaRule, eps, row_slot, row_pos, state, ring, out, status=None):
     _need_cuda(x, state)
     check(_lib.lib().mlora_delta_step(
         _ptr(x), x.stride(0), r.channels, r.taps, r.g_col, r.b_col, r.a_col, _ptr(r.conv), _ptr(r.A_log), _ptr(r.dt_bias), _ptr(r.norm),
         eps, r.heads, r.kv_heads, r.dim, r.vdim, r.vdim_true, r.q_scale, _ptr(row_slot), _ptr(row_pos), x.shape[0], _ptr(state),
-        _ptr(ring), _ptr(out), int(x.dtype == torch.float32), _stream()), "mlora_delta_step")
+        _ptr(ring), _ptr(out), _ptr(status), int(x.dtype == torch.float32), _stream()), "mlora_delta_step")
     return out

@@ -246,7 +246,7 @@ class RelidraEngine(PlainEngine):
         kv, r, eps = self.kv, lw.rule, self.m.config.eps
         S, ring, row_slot, row_pos = kv.state(run, "S"), kv.state(run, "conv"), self.row_slot[:T], self.row_pos[:T]
         if decode:
-            return ops.delta_step(proj, r, eps, row_slot, row_pos, S, ring, out)
+            return ops.delta_step(proj, r, eps, row_slot, row_pos, S, ring, out, status=self.status)
         xc = ops.short_conv(proj, r.conv, ring, row_slot, row_pos, self._grow("conv", self.max_rows * self._conv_cols)[:T * r.channels]
                             .view(T, r.channels))
         o = self._grow("o", self.max_rows * self._o_cols, torch.float32)[:T * lw.out_cols].view(T, lw.out_cols)

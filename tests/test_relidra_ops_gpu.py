@@ -302,7 +302,7 @@ class DeltaCase:
         assert self.state[-1].isnan().all() and self.state[0].isnan().all()  # other slots untouched
 
 
-SIZES = [(6, 2, 20, 12, 3), (3, 3, 33, 41, 5), (1, 1, 8, 8, 1), (2, 1, 200, 8, 2), (4, 4, 128, 136, 4), (2, 2, 64, 64, 8), (2, 1, 96, 264, 4), (3, 1, 256, 48, 6)]
+SIZES = [(6, 2, 20, 12, 3), (3, 3, 33, 41, 5), (1, 1, 8, 8, 1), (2, 1, 200, 8, 2), (4, 4, 128, 136, 4), (2, 2, 64, 64, 8), (2, 1, 96, 264, 4), (3, 1, 256, 48, 6), (1, 1, 256, 208, 3)]
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
