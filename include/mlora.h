@@ -522,7 +522,7 @@ int mlora_latent_attention_simt(const void* d_qa, int64_t q_pitch, const void* d
 
 /* ---- hyper-connections + layer norm ---------------------------------------------------------------------------
  * The residual as n streams of H columns per row.  With delta (the result of the sublayer before): stream t becomes
- * sum_s mix[s, t] stream_s + back[t] * delta, all of them from the old ones (d_back = back[n], then mix[n, n], [from, to]).
+ * sum_s mix[s, t] stream_s + back[t] * delta, all of them from the old ones (d_back = back[n], then mix[n, n], a row per old stream).
  * Then u = sum_s read[s] stream_s and out = (u - mean) / sqrt(variance + eps) * w over the first `width` columns (the others
  * are zero; w [H] bf16).  d_src: streams before, row r at d_src + r * ld_src, stream s src_stream further (0: all streams are
  * the same row).  d_dst [T][n][H] (may be d_src with ld_src = n * H, src_stream = H; NULL: the new streams are not kept).
@@ -534,7 +534,7 @@ int mlora_residual_streams_layernorm(const void* d_delta, const float* d_src, in
 
 /* ---- attention with rotated, normalised keys that are their own values; chunks; sinks -----------------------------
  * mlora_rotate_rms_append: x rows [q heads | k heads] of `dim` columns; x += bias; the first `rot` columns of a head rotated
- *   by position * inv_freq[i] (column i paired with i + rot / 2), then the head divided by sqrt(mean(x^2) + eps).  Queries,
+ *   by position * inv_freq[i] (columns i and i + rot / 2 turn together), then the head divided by sqrt(mean(x^2) + eps).  Queries,
  *   times q_scale, to d_q [T, Hq, pad]; keys to their place in d_k_pages, and x + bias as it was before to d_v_pages
  *   (pages [page][Hkv][page_size][pad]; columns from dim to pad are zero; rows with row_pos < 0 store nothing).  dim <= 512.
  * mlora_paged_attention_masked, mlora_prefill_attention_masked: mlora_paged_attention (fused_append = 0) and
@@ -576,8 +576,8 @@ int mlora_paged_attention_any(const void* d_q, const void* d_k_pages, const void
  * h / (heads / kv_heads).  dim <= 256 and vdim multiples of 8 (pad with zero weights).
  * State [slot][heads][dim][vdim]; ring [slot][taps][C]: the convolution's inputs, token p at place p % taps.  Neither is read
  * for a sequence's position 0, so neither needs clearing.  Activations are bf16, or fp32 with f32 != 0.
- * mlora_short_conv: convolution and silu of all rows of a pass (rows of one sequence are consecutive; w [taps][C] fp32, the
- *   last row is the current token's).
+ * mlora_short_conv: convolution and silu of all rows of a pass (rows of one sequence are consecutive; w [taps][C] fp32, row
+ *   taps - 1 for the token itself).
  * mlora_delta_scan: the recurrence over the rows of each segment int32 [n][4] = (slot, first row, rows, position of the first
  *   row), one segment per sequence; xc from mlora_short_conv, x the projected rows with b and a from columns b_col and a_col.
  *   Leaves state and ring after the segment's last row, and o [T, heads * vdim] fp32.

@@ -1,6 +1,6 @@
 """Plain Relidra decoder in PyTorch on the CPU: one function per mechanism, no cache, no batching.
 
-The checker of the CUDA path.  It shares no code with the package: every function below restates its equation on
+What the CUDA path is compared with.  It shares no code with the package: every function below restates its equation on
 whole sequences in the dtype of its inputs (float64 or float32).  ``params`` is a dict of tensors under the names of
 the checkpoint format.
 """
@@ -40,7 +40,7 @@ def hyper_connect(streams, w_in, w_mix, w_out, sublayer):
 
 
 def short_conv(x, taps):
-    """x [n, channels], taps [channels, K]: causal, the last tap is the current token's, zeros before the start."""
+    """x [n, channels], taps [channels, K]: a channel's own row weighs its last K inputs, taps[:, K - 1] the newest."""
     n, K = x.shape[0], taps.shape[1]
     out = torch.zeros_like(x)
     for i in range(n):
@@ -88,7 +88,7 @@ def delta_mixer(h, p, pre, heads, kv_heads, dim, vdim, eps):
 
 
 def rotate(x, pos, dims, base, factor):
-    """x [n, heads, dim]: the first ``dims`` values of a head, value i paired with i + dims / 2."""
+    """x [n, heads, dim]: values i and i + dims / 2 of a head turn together, for i below dims / 2."""
     half = dims // 2
     f = torch.tensor([base ** (-2.0 * i / dims) / factor for i in range(half)], dtype=x.dtype)
     a = (pos.to(x.dtype)[:, None] * f)[:, None, :]

@@ -164,7 +164,7 @@ struct ConvArgs {
   const A* x;        // [T, >= C]
   int64_t ld;
   int C, taps;       // channels (a multiple of 8)
-  const float* w;    // [taps][C], the last row is the current token's
+  const float* w;    // [taps][C], row taps - 1 for the token itself
   const A* ring;     // [slot][taps][C]
   const int32_t *row_slot, *row_pos;
   A* out;            // [T, C]

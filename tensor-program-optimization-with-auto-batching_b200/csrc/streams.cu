@@ -18,7 +18,7 @@ struct StreamsArgs {
   const float* src;       // streams before: row pitch ld_src, stream s at + s * src_stream (0: all streams are one row)
   int64_t ld_src, src_stream;
   float* dst;             // streams after [T][n][H], or NULL: not stored
-  const float* back;      // [n] + [n, n]: what every stream gets of delta, then mix[from][to]; with delta
+  const float* back;      // with delta: [n] what every stream gets of it, then [n, n] the mix, a row per old stream
   const float* read;      // [n_read] weights of the sum that is normalised
   const int32_t* rows;    // NULL: every row; else output row i is row rows[i]
   const bf16* w;
